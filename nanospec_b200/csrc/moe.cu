@@ -5,15 +5,19 @@
 //   ns_router_logits   the router's float product for a few tokens (longer steps: ns_cast_f32 and the float GEMM)
 //   ns_moe_route       scores = sigmoid(logits) (or softmax); consecutive experts form `groups` groups of equal size, ranked by
 //                      the top-2 sum of their scores; all but the `keep` highest-ranked groups are barred; then the `top`
-//                      highest-scoring experts that are not barred; weights = score / (sum of the chosen + 1e-20) * scale.
-//                      Ties go to the lower index.
+//                      highest-scoring experts that are not barred; weights = score / (sum of the chosen + 1e-20) * scale,
+//                      or score * scale.  An optional correction per expert is added to the scores that choose (groups
+//                      and experts) and not to the weights.  Ties go to the lower index.
 //   ns_moe_plan        counts per expert, their running offsets, and for every (token, choice) its row in the
-//                      order that has each expert's tokens side by side
+//                      order that has each expert's tokens side by side; a choice beyond the experts that have weights (an
+//                      expert that returns its input) has no row: -1
 //   ns_moe_pad_rows    the same rows in a layout where every expert owns a fixed number of rows (for one batched product)
-//   ns_moe_gather      x rows into that order;  ns_moe_combine   out[n] = sum_k weight[n, k] * y[row(n, k)] in float
+//   ns_moe_gather      x rows into that order
+//   ns_moe_combine     out[n] = sum_k weight[n, k] * y[row(n, k)] in float (x[n] in place of y for a choice without a row),
+//                      or the same sum added to a float stream
 //   ns_moe_expert_rows the experts themselves for a few tokens, no host round trip: one block row per (token,
 //                      choice) streams the chosen expert's gate and up rows, then its down rows
-//   ns_activation      out = act(x) elementwise: exact (erf) gelu, tanh gelu, silu, squared relu
+//   ns_activation      out = act(x) elementwise: exact (erf) gelu, tanh gelu, silu, squared relu, xielu
 #include "common.cuh"
 
 namespace {
@@ -62,15 +66,17 @@ router_logits_kernel(const T* __restrict__ x, long long ldx, const float* __rest
 // one warp per token
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, int n_tokens, int E, int groups, int keep, int top, float scale,
-                 int softmax, int* __restrict__ ids, float* __restrict__ weights) {
+                 int softmax, const float* __restrict__ correction, int renormalize, int* __restrict__ ids,
+                 float* __restrict__ weights) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     extern __shared__ float rs[];
     const int lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
     const int n = blockIdx.x * 4 + wib;
     if (n >= n_tokens) return;
-    float* sc = rs + (size_t)wib * 2 * E;  // scores, then group scores (at most E of them)
-    float* gs = sc + E;
+    float* sc = rs + (size_t)wib * 3 * E;  // scores, the scores that choose, then group scores (at most E of them)
+    float* cs = sc + E;
+    float* gs = cs + E;
     const float* z = logits + (size_t)n * E;
     if (softmax) {
         float mx = -INFINITY;
@@ -87,14 +93,15 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int E, int grou
     } else {
         for (int e = lane; e < E; e += 32) sc[e] = 1.f / (1.f + expf(-z[e]));
     }
+    for (int e = lane; e < E; e += 32) cs[e] = sc[e] + (correction ? correction[e] : 0.f);
     __syncwarp();
-    const float taken = -1.f;  // scores are positive; a taken or barred entry is marked below every score
+    const float taken = -INFINITY;  // a taken or barred entry
     if (groups > 1) {
         const int per = E / groups;
         for (int g = lane; g < groups; g += 32) {
             float a = -INFINITY, b = -INFINITY;  // the two largest
             for (int e = g * per; e < (g + 1) * per; ++e) {
-                const float v = sc[e];
+                const float v = cs[e];
                 if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
             }
             gs[g] = per > 1 ? a + b : a;
@@ -106,27 +113,27 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int E, int grou
             int wi = -1;
             for (int g = lane; g < groups; g += 32) {
                 const float v = gs[g];
-                if (v >= 0.f && (v < worst || (v == worst && g > wi))) { worst = v; wi = g; }
+                if (v > taken && (v < worst || (v == worst && g > wi))) { worst = v; wi = g; }
             }
             for (int o = 16; o > 0; o >>= 1) {
                 const float ov = __shfl_xor_sync(0xffffffffu, worst, o);
                 const int oi = __shfl_xor_sync(0xffffffffu, wi, o);
                 if (oi >= 0 && (wi < 0 || ov < worst || (ov == worst && oi > wi))) { worst = ov; wi = oi; }
             }
-            if (lane == 0) gs[wi] = taken;
+            if (lane == 0 && wi >= 0) gs[wi] = taken;
             __syncwarp();
         }
         for (int e = lane; e < E; e += 32)
-            if (gs[e / per] < 0.f) sc[e] = taken;
+            if (gs[e / per] == taken) cs[e] = taken;
         __syncwarp();
     }
     float total = 0.f, mine = 0.f;
     int mine_id = 0;
     for (int k = 0; k < top; ++k) {
-        float best = -INFINITY;
+        float best = taken;
         int bi = -1;
         for (int e = lane; e < E; e += 32) {
-            const float v = sc[e];
+            const float v = cs[e];
             if (v > best) { best = v; bi = e; }  // ascending e: the lower index wins a tie
         }
         for (int o = 16; o > 0; o >>= 1) {
@@ -134,16 +141,18 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int E, int grou
             const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (oi >= 0 && (bi < 0 || ov > best || (ov == best && oi < bi))) { best = ov; bi = oi; }
         }
-        total += best;
-        if (lane == k % 32 && k < 32) { mine = best; mine_id = bi; }
+        bi = max(bi, 0);  // (no score above the marker is left only when the logits are not numbers)
+        const float w = sc[bi];
+        total += w;
+        if (lane == k % 32 && k < 32) { mine = w; mine_id = bi; }
         if (k >= 32 && lane == 0) {  // more than 32 choices: written unnormalised, fixed up below
             ids[(size_t)n * top + k] = bi;
-            weights[(size_t)n * top + k] = best;
+            weights[(size_t)n * top + k] = w;
         }
-        if (lane == 0) sc[bi] = taken;
+        if (lane == 0) cs[bi] = taken;
         __syncwarp();
     }
-    const float f = scale / (total + 1e-20f);
+    const float f = renormalize ? scale / (total + 1e-20f) : scale;
     if (lane < top && lane < 32) {
         ids[(size_t)n * top + lane] = mine_id;
         weights[(size_t)n * top + lane] = mine * f;
@@ -162,7 +171,8 @@ moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int E, int* __restrict
     const int tid = threadIdx.x;
     for (int e = tid; e < E; e += blockDim.x) count[e] = 0;
     __syncthreads();
-    for (int i = tid; i < n_pairs; i += blockDim.x) atomicAdd(&count[ids[i]], 1);
+    for (int i = tid; i < n_pairs; i += blockDim.x)
+        if (ids[i] < E) atomicAdd(&count[ids[i]], 1);
     __syncthreads();
     if (tid == 0) {
         int at = 0;
@@ -176,9 +186,10 @@ moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int E, int* __restrict
     __syncthreads();
     // which row of its expert's run a pair gets does not matter to any result: rows are computed alone
     for (int i = tid; i < n_pairs; i += blockDim.x) {
-        const int row = atomicAdd(&cursor[ids[i]], 1);
+        const int e = ids[i];
+        const int row = e < E ? atomicAdd(&cursor[e], 1) : -1;
         row_of[i] = row;
-        if (pair_of) pair_of[row] = i;
+        if (pair_of && row >= 0) pair_of[row] = i;
     }
 }
 
@@ -189,6 +200,7 @@ __global__ void moe_pad_rows_kernel(const int* __restrict__ ids, const int* __re
     ns_pdl_wait();
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n_pairs) return;
+    if (row_of[i] < 0) return;  // a choice without a row
     const int e = ids[i];
     row_of[i] = e * capacity + (row_of[i] - offsets[e]);
 }
@@ -199,22 +211,51 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, const int* __restrict
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     const int pair = blockIdx.x;
+    if (row_of[pair] < 0) return;
     const T* src = x + (size_t)(pair / top) * width;
     T* dst = xs + (size_t)row_of[pair] * width;
     for (int h = threadIdx.x; h < width; h += blockDim.x) dst[h] = src[h];
 }
 
-template <typename T>
+// out[n] = sum_k weight[n, k] * (row >= 0 ? ys[row] : x[n]), float sums in the order of the choice, rounded once; with `resid`
+// the sum is added to that float row instead.  VEC = 8: eight features to a thread with 16-byte accesses.
+template <typename T, int VEC>
 __global__ void moe_combine_kernel(const T* __restrict__ ys, const int* __restrict__ row_of, const float* __restrict__ weights,
-                                   T* __restrict__ out, int top, int width) {
+                                   const T* __restrict__ x, T* __restrict__ out, float* __restrict__ resid, int top, int width) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     const int n = blockIdx.x;
-    for (int h = threadIdx.x; h < width; h += blockDim.x) {
-        float a = 0.f;
-        for (int k = 0; k < top; ++k)
-            a = fmaf(weights[(size_t)n * top + k], ns_ld(ys, (size_t)row_of[(size_t)n * top + k] * width + h), a);
-        ns_st(out, (size_t)n * width + h, a);
+    const int* rows = row_of + (size_t)n * top;
+    const float* w = weights + (size_t)n * top;
+    for (int h = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; h < width; h += gridDim.y * blockDim.x * VEC) {
+        const size_t at = (size_t)n * width + h;
+        if constexpr (VEC == 8) {
+            float a[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) a[i] = 0.f;
+            for (int k = 0; k < top; ++k) {
+                const int row = rows[k];
+                const float wk = w[k];
+                float v[8];
+                ld8(row >= 0 ? ys + (size_t)row * width + h : x + at, v);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) a[i] = fmaf(wk, v[i], a[i]);
+            }
+            if (resid) {
+                float v[8];
+                ld8(resid + at, v);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) a[i] += v[i];
+                st8(resid + at, a);
+            } else {
+                st8(out + at, a);
+            }
+        } else {
+            float a = 0.f;
+            for (int k = 0; k < top; ++k) a = fmaf(w[k], rows[k] >= 0 ? ns_ld(ys, (size_t)rows[k] * width + h) : ns_ld(x, at), a);
+            if (resid) resid[at] += a;
+            else ns_st(out, at, a);
+        }
     }
 }
 
@@ -238,12 +279,13 @@ __device__ __forceinline__ float dot_row(const T* __restrict__ w, const float* _
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_gate_up_rows_kernel(const T* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ w_gate,
-                        const T* __restrict__ w_up, T* __restrict__ act, int top, int width, int ff, int per_block) {
+                        const T* __restrict__ w_up, T* __restrict__ act, int E, int top, int width, int ff, int per_block) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     extern __shared__ float xs[];
     const int pair = blockIdx.x, lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
     const int e = ids[pair];
+    if (e >= E) return;  // returns its input: nothing to compute here
     const T* xr = x + (size_t)(pair / top) * width;
     for (int k = threadIdx.x; k < width; k += blockDim.x) xs[k] = ns_ld(xr, k);
     __syncthreads();
@@ -257,16 +299,18 @@ moe_gate_up_rows_kernel(const T* __restrict__ x, const int* __restrict__ ids, co
     }
 }
 
-// out[n, i] = sum_k weight[n, k] * (down_e(k)[i] . act[n, k]); grid (tokens, feature chunks)
+// out[n, i] = sum_k weight[n, k] * (down_e(k)[i] . act[n, k]), x[n, i] in place of the product for e(k) >= E; grid (tokens, feature chunks)
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_down_rows_kernel(const T* __restrict__ act, const int* __restrict__ ids, const float* __restrict__ weights,
-                     const T* __restrict__ w_down, T* __restrict__ out, int top, int width, int ff, int per_block) {
+                     const T* __restrict__ w_down, const T* __restrict__ x, T* __restrict__ out, int E, int top, int width, int ff,
+                     int per_block) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     extern __shared__ float as[];  // [top][ff]
     const int n = blockIdx.x, lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
-    for (int i = threadIdx.x; i < top * ff; i += blockDim.x) as[i] = ns_ld(act, (size_t)n * top * ff + i);
+    for (int i = threadIdx.x; i < top * ff; i += blockDim.x)
+        as[i] = ids[(size_t)n * top + i / ff] < E ? ns_ld(act, (size_t)n * top * ff + i) : 0.f;
     __syncthreads();
     const bool vec = ff % 8 == 0 && ((uintptr_t)w_down % 16 == 0);
     const int i0 = blockIdx.y * per_block, i1 = min(width, i0 + per_block);
@@ -274,36 +318,46 @@ moe_down_rows_kernel(const T* __restrict__ act, const int* __restrict__ ids, con
         float a = 0.f;
         for (int k = 0; k < top; ++k) {
             const int e = ids[(size_t)n * top + k];
+            if (e >= E) {
+                a = fmaf(weights[(size_t)n * top + k], ns_ld(x, (size_t)n * width + i), a);
+                continue;
+            }
             a = fmaf(weights[(size_t)n * top + k], dot_row(w_down + ((size_t)e * width + i) * ff, as + (size_t)k * ff, ff, lane, vec), a);
         }
         if (lane == 0) ns_st(out, (size_t)n * width + i, a);
     }
 }
 
-__device__ __forceinline__ float act_value(float z, int kind) {
+// xielu's coefficients, taken by the kinds that have none as well: a of the quadratic branch, b of the exponential one
+struct ActCoef { float a, b; };
+__device__ __forceinline__ ActCoef act_coef(const float* coef) { return coef ? ActCoef{coef[0], coef[1]} : ActCoef{0.f, 0.f}; }
+
+__device__ __forceinline__ float act_value(float z, int kind, ActCoef c) {
     if (kind == 0) return 0.5f * z * (1.f + erff(z * 0.70710678118654752440f));
     if (kind == 1) return 0.5f * z * (1.f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
     if (kind == 3) { const float p = fmaxf(z, 0.f); return p * p; }
+    if (kind == 4) return (z > 0.f ? c.a * z * z : c.b * (expm1f(z) - z)) + 0.5f * z;
     return z / (1.f + expf(-z));
 }
 
 template <typename T>
-__global__ void activation_vec_kernel(const T* __restrict__ x, T* __restrict__ out, int kind, size_t total8) {
+__global__ void activation_vec_kernel(const T* __restrict__ x, T* __restrict__ out, int kind, const float* __restrict__ coef, size_t total8) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total8) return;
     float v[8];
     ld8(x + i * 8, v);
+    const ActCoef c = act_coef(coef);
 #pragma unroll
-    for (int k = 0; k < 8; ++k) v[k] = act_value(v[k], kind);
+    for (int k = 0; k < 8; ++k) v[k] = act_value(v[k], kind, c);
     st8(out + i * 8, v);
 }
 
 // rows of `cols` features with strides of their own (column ranges of wider buffers); VEC = 8 needs both rows on 16 bytes
 template <typename T, int VEC>
 __global__ void activation_rows_kernel(const T* __restrict__ x, long long ldx, T* __restrict__ out, long long ldo, int cols, int kind,
-                                       size_t total) {
+                                       const float* __restrict__ coef, size_t total) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -311,24 +365,25 @@ __global__ void activation_rows_kernel(const T* __restrict__ x, long long ldx, T
     const int per_row = cols / VEC;
     const size_t row = i / per_row;
     const int c = (int)(i - row * per_row) * VEC;
+    const ActCoef co = act_coef(coef);
     if constexpr (VEC == 8) {
         float v[8];
         ld8(x + row * ldx + c, v);
 #pragma unroll
-        for (int k = 0; k < 8; ++k) v[k] = act_value(v[k], kind);
+        for (int k = 0; k < 8; ++k) v[k] = act_value(v[k], kind, co);
         st8(out + row * ldo + c, v);
     } else {
-        ns_st(out, row * ldo + c, act_value(ns_ld(x, row * ldx + c), kind));
+        ns_st(out, row * ldo + c, act_value(ns_ld(x, row * ldx + c), kind, co));
     }
 }
 
 template <typename T>
-__global__ void activation_kernel(const T* __restrict__ x, T* __restrict__ out, int kind, size_t total) {
+__global__ void activation_kernel(const T* __restrict__ x, T* __restrict__ out, int kind, const float* __restrict__ coef, size_t total) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
-    ns_st(out, i, act_value(ns_ld(x, i), kind));
+    ns_st(out, i, act_value(ns_ld(x, i), kind, act_coef(coef)));
 }
 
 }  // namespace
@@ -364,13 +419,14 @@ NS_API int ns_router_logits(const void* x, long long ldx, const float* w, float*
 }
 
 NS_API int ns_moe_route(const float* logits, int n_tokens, int E, int groups, int keep, int top, float scale, int softmax,
-                        int* ids, float* weights, cudaStream_t stream) {
+                        const float* correction, int renormalize, int* ids, float* weights, cudaStream_t stream) {
     if (n_tokens <= 0) return NS_OK;
     if (E < 1 || E > kMaxExperts || top < 1 || top > E) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_moe_route: %d experts, %d chosen (at most %d experts)", E, top, kMaxExperts);
     if (groups > 1 && (E % groups || keep < 1 || keep > groups || keep * (E / groups) < top))
         NS_FAIL(NS_ERR_ARGUMENT, "ns_moe_route: %d groups over %d experts, %d kept, %d chosen", groups, E, keep, top);
-    const size_t smem = (size_t)4 * 2 * E * sizeof(float);
-    NS_LAUNCH(moe_route_kernel, (n_tokens + 3) / 4, 128, smem, stream, logits, n_tokens, E, groups, keep, top, scale, softmax, ids, weights);
+    const size_t smem = (size_t)4 * 3 * E * sizeof(float);
+    NS_LAUNCH(moe_route_kernel, (n_tokens + 3) / 4, 128, smem, stream, logits, n_tokens, E, groups, keep, top, scale, softmax,
+              correction, renormalize, ids, weights);
     NS_CHECK_LAUNCH("ns_moe_route");
     return NS_OK;
 }
@@ -399,21 +455,29 @@ NS_API int ns_moe_gather(const void* x, const int* row_of, void* xs, int n_token
     return NS_OK;
 }
 
-NS_API int ns_moe_combine(const void* ys, const int* row_of, const float* weights, void* out, int n_tokens, int top, int width,
-                          int dtype, cudaStream_t stream) {
+// x [n, width] (only read for choices without a row); resid (float) or out receives the sum
+NS_API int ns_moe_combine(const void* ys, const int* row_of, const float* weights, const void* x, void* out, float* resid, int n_tokens,
+                          int top, int width, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return NS_OK;
-    if (dtype == NS_F32) NS_LAUNCH((moe_combine_kernel<float>), n_tokens, 256, 0, stream, (const float*)ys, row_of, weights, (float*)out, top, width);
-    else if (dtype == NS_BF16) NS_LAUNCH((moe_combine_kernel<__nv_bfloat16>), n_tokens, 256, 0, stream, (const __nv_bfloat16*)ys, row_of, weights, (__nv_bfloat16*)out, top, width);
-    else NS_FAIL(NS_ERR_ARGUMENT, "ns_moe_combine: unknown dtype %d", dtype);
+    if (dtype != NS_F32 && dtype != NS_BF16) NS_FAIL(NS_ERR_ARGUMENT, "ns_moe_combine: unknown dtype %d", dtype);
+    if (!out && !resid) NS_FAIL(NS_ERR_ARGUMENT, "ns_moe_combine: nowhere to put the sum");
+    const bool vec = width % 8 == 0 && (((uintptr_t)ys | (uintptr_t)x | (uintptr_t)out | (uintptr_t)resid) % 16 == 0);
+    const int per_row = vec ? width / 8 : width;
+    const int threads = per_row >= 256 ? 256 : (per_row + 31) / 32 * 32;
+    const dim3 grid(n_tokens, vec ? (per_row + threads - 1) / threads : 1);
+#define NS_COMBINE(T, V) NS_LAUNCH((moe_combine_kernel<T, V>), grid, threads, 0, stream, (const T*)ys, row_of, weights, (const T*)x, (T*)out, resid, top, width)
+    if (dtype == NS_F32) { if (vec) NS_COMBINE(float, 8); else NS_COMBINE(float, 1); }
+    else { if (vec) NS_COMBINE(__nv_bfloat16, 8); else NS_COMBINE(__nv_bfloat16, 1); }
+#undef NS_COMBINE
     NS_CHECK_LAUNCH("ns_moe_combine");
     return NS_OK;
 }
 
 // x [n, width]; ids, weights [n, top]; w_gate, w_up [E, ff, width]; w_down [E, width, ff]; act [n * top, ff] scratch;
-// out [n, width]
+// out [n, width]; ids from n_experts on return their input
 NS_API int ns_moe_expert_rows(const void* x, const int* ids, const float* weights, const void* w_gate, const void* w_up,
-                              const void* w_down, void* act, void* out, int n_tokens, int top, int width, int ff, int dtype,
-                              cudaStream_t stream) {
+                              const void* w_down, void* act, void* out, int n_experts, int n_tokens, int top, int width,
+                              int ff, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return NS_OK;
     const size_t smem_a = (size_t)width * sizeof(float), smem_b = (size_t)top * ff * sizeof(float);
     if (smem_a > 200 * 1024 || smem_b > 200 * 1024)
@@ -425,10 +489,10 @@ NS_API int ns_moe_expert_rows(const void* x, const int* ids, const float* weight
         if (smem_a > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(moe_gate_up_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
         if (smem_b > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(moe_down_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));    \
         NS_LAUNCH((moe_gate_up_rows_kernel<T>), grid_a, 256, smem_a, stream, (const T*)x, ids, (const T*)w_gate, (const T*)w_up,      \
-                  (T*)act, top, width, ff, per_a);                                                                            \
+                  (T*)act, n_experts, top, width, ff, per_a);                                                                            \
         NS_CHECK_LAUNCH("ns_moe_expert_rows");                                                                                \
-        NS_LAUNCH((moe_down_rows_kernel<T>), grid_b, 256, smem_b, stream, (const T*)act, ids, weights, (const T*)w_down, (T*)out,     \
-                  top, width, ff, per_b);                                                                                     \
+        NS_LAUNCH((moe_down_rows_kernel<T>), grid_b, 256, smem_b, stream, (const T*)act, ids, weights, (const T*)w_down, (const T*)x, (T*)out,     \
+                  n_experts, top, width, ff, per_b);                                                                                     \
     }
     if (dtype == NS_F32) NS_MOE_ROWS(float)
     else if (dtype == NS_BF16) NS_MOE_ROWS(__nv_bfloat16)
@@ -439,42 +503,43 @@ NS_API int ns_moe_expert_rows(const void* x, const int* ids, const float* weight
 }
 
 // the same over rows that lie in wider buffers: x[r * ldx + c] -> out[r * ldo + c], c < cols
-NS_API int ns_activation_rows(const void* x, long long ldx, void* out, long long ldo, int n_rows, int cols, int kind, int dtype,
-                              cudaStream_t stream) {
+NS_API int ns_activation_rows(const void* x, long long ldx, void* out, long long ldo, int n_rows, int cols, int kind,
+                              const float* coef, int dtype, cudaStream_t stream) {
     if (n_rows <= 0 || cols <= 0) return NS_OK;
-    if (kind < 0 || kind > 3) NS_FAIL(NS_ERR_ARGUMENT, "ns_activation_rows: unknown kind %d", kind);
+    if (kind < 0 || kind > 4 || (kind == 4 && !coef)) NS_FAIL(NS_ERR_ARGUMENT, "ns_activation_rows: unknown kind %d", kind);
     if (dtype != NS_F32 && dtype != NS_BF16) NS_FAIL(NS_ERR_ARGUMENT, "ns_activation_rows: unknown dtype %d", dtype);
     const size_t esz = dtype == NS_F32 ? 4 : 2;
     const bool vec = cols % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) % 16 == 0) && (ldx * esz) % 16 == 0 && (ldo * esz) % 16 == 0;
     const size_t total = (size_t)n_rows * (vec ? cols / 8 : cols);
     const unsigned blocks = (unsigned)((total + 255) / 256);
     if (dtype == NS_F32) {
-        if (vec) NS_LAUNCH((activation_rows_kernel<float, 8>), blocks, 256, 0, stream, (const float*)x, ldx, (float*)out, ldo, cols, kind, total);
-        else NS_LAUNCH((activation_rows_kernel<float, 1>), blocks, 256, 0, stream, (const float*)x, ldx, (float*)out, ldo, cols, kind, total);
+        if (vec) NS_LAUNCH((activation_rows_kernel<float, 8>), blocks, 256, 0, stream, (const float*)x, ldx, (float*)out, ldo, cols, kind, coef, total);
+        else NS_LAUNCH((activation_rows_kernel<float, 1>), blocks, 256, 0, stream, (const float*)x, ldx, (float*)out, ldo, cols, kind, coef, total);
     } else {
-        if (vec) NS_LAUNCH((activation_rows_kernel<__nv_bfloat16, 8>), blocks, 256, 0, stream, (const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)out, ldo, cols, kind, total);
-        else NS_LAUNCH((activation_rows_kernel<__nv_bfloat16, 1>), blocks, 256, 0, stream, (const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)out, ldo, cols, kind, total);
+        if (vec) NS_LAUNCH((activation_rows_kernel<__nv_bfloat16, 8>), blocks, 256, 0, stream, (const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)out, ldo, cols, kind, coef, total);
+        else NS_LAUNCH((activation_rows_kernel<__nv_bfloat16, 1>), blocks, 256, 0, stream, (const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)out, ldo, cols, kind, coef, total);
     }
     NS_CHECK_LAUNCH("ns_activation_rows");
     return NS_OK;
 }
 
-// kind 0: 0.5 z (1 + erf(z / sqrt 2));  1: 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)));  2: z sigmoid(z);  3: max(z, 0)^2
-NS_API int ns_activation(const void* x, void* out, long long total, int kind, int dtype, cudaStream_t stream) {
+// kind 0: 0.5 z (1 + erf(z / sqrt 2));  1: 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)));  2: z sigmoid(z);  3: max(z, 0)^2;
+// 4: (z > 0 ? a z^2 : b (exp(z) - 1 - z)) + z / 2 with a, b = coef[0], coef[1] (float, on the device)
+NS_API int ns_activation(const void* x, void* out, long long total, int kind, const float* coef, int dtype, cudaStream_t stream) {
     if (total <= 0) return NS_OK;
-    if (kind < 0 || kind > 3) NS_FAIL(NS_ERR_ARGUMENT, "ns_activation: unknown kind %d", kind);
+    if (kind < 0 || kind > 4 || (kind == 4 && !coef)) NS_FAIL(NS_ERR_ARGUMENT, "ns_activation: unknown kind %d", kind);
     if (total % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) % 16 == 0)) {  // eight elements to a thread
         const size_t total8 = (size_t)total / 8;
         const unsigned vblocks = (unsigned)((total8 + 255) / 256);
-        if (dtype == NS_F32) NS_LAUNCH((activation_vec_kernel<float>), vblocks, 256, 0, stream, (const float*)x, (float*)out, kind, total8);
-        else if (dtype == NS_BF16) NS_LAUNCH((activation_vec_kernel<__nv_bfloat16>), vblocks, 256, 0, stream, (const __nv_bfloat16*)x, (__nv_bfloat16*)out, kind, total8);
+        if (dtype == NS_F32) NS_LAUNCH((activation_vec_kernel<float>), vblocks, 256, 0, stream, (const float*)x, (float*)out, kind, coef, total8);
+        else if (dtype == NS_BF16) NS_LAUNCH((activation_vec_kernel<__nv_bfloat16>), vblocks, 256, 0, stream, (const __nv_bfloat16*)x, (__nv_bfloat16*)out, kind, coef, total8);
         else NS_FAIL(NS_ERR_ARGUMENT, "ns_activation: unknown dtype %d", dtype);
         NS_CHECK_LAUNCH("ns_activation");
         return NS_OK;
     }
     const unsigned blocks = (unsigned)((total + 255) / 256);
-    if (dtype == NS_F32) NS_LAUNCH((activation_kernel<float>), blocks, 256, 0, stream, (const float*)x, (float*)out, kind, (size_t)total);
-    else if (dtype == NS_BF16) NS_LAUNCH((activation_kernel<__nv_bfloat16>), blocks, 256, 0, stream, (const __nv_bfloat16*)x, (__nv_bfloat16*)out, kind, (size_t)total);
+    if (dtype == NS_F32) NS_LAUNCH((activation_kernel<float>), blocks, 256, 0, stream, (const float*)x, (float*)out, kind, coef, (size_t)total);
+    else if (dtype == NS_BF16) NS_LAUNCH((activation_kernel<__nv_bfloat16>), blocks, 256, 0, stream, (const __nv_bfloat16*)x, (__nv_bfloat16*)out, kind, coef, (size_t)total);
     else NS_FAIL(NS_ERR_ARGUMENT, "ns_activation: unknown dtype %d", dtype);
     NS_CHECK_LAUNCH("ns_activation");
     return NS_OK;

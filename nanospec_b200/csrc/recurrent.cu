@@ -1,11 +1,12 @@
-// Mixers with a fixed-size state per request: linear attention with a decay (retention) and the gated
-// delta rule, for portions of prompts and single decoded tokens alike.
+// Mixers with a fixed-size state per request: linear attention with a decay (retention), the gated
+// delta rule and the selective state space of Mamba-2, for portions of prompts and single decoded tokens alike.
 //
 // Per head the state is a matrix S [D, V] of floats.  For every token, in order:
 //     plain:  S = g S + k v^T                      o = S^T q
+//     step:   S = g S + k (beta v)^T               o = S^T q      (state space: k = B, q = C, v = x, beta the step size)
 //     delta:  S = g S;  u = beta (v - S^T k);  S = S + k u^T;   o = S^T q
 // The read-out is taken from the state before the token's write, which is the same number:
-//     o = S_new^T q = g (S_old^T q) + w (k . q)      with w = v (plain) or u (delta),
+//     o = S_new^T q = g (S_old^T q) + w (k . q)      with w = v (plain), beta v (step) or u (delta),
 // so that the two sums over a column, S_old^T k and S_old^T q, run side by side and the write to S is off the path
 // from one token to the next; k . q per token and key head comes from the preparation.
 // The columns of S never meet: column e needs only v[e], so the scan runs one column per group of four
@@ -168,7 +169,7 @@ rotary_prepare_kernel(const T* __restrict__ proj, int ld_proj, const int* __rest
 // walk over the tokens waits for memory once per stage and not once per token; a row of q or k lies there in LPC
 // segments of R + 4 floats (the parts' 16-byte reads then fall into different banks).
 // q and k heads are shared by H / G heads each.  gate: per token and head (row stride ld) or null, then `decay[h]` is
-// used; beta: null selects the plain rule.
+// used; beta: null selects the plain rule; with it `delta` selects the delta rule, otherwise the step rule.
 // ---------------------------------------------------------------------------------------
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
@@ -224,7 +225,7 @@ linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, con
                    const float* __restrict__ gate, const float* __restrict__ beta, const float* __restrict__ kq,
                    const float* __restrict__ decay, int ld, float* __restrict__ state, long long state_floats,
                    const int* __restrict__ qo_indptr, const int* __restrict__ state_slot, float* __restrict__ out, int ld_out,
-                   int H, int G, int D, int V) {
+                   int H, int G, int D, int V, int delta) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     using Sh = ScanShape<R, LPC, C, ONE>;
@@ -320,19 +321,20 @@ linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, con
             for (int c = 0; c < C; ++c) {
                 w[c] = sv[t * Sh::kCols + col + c * CB];
                 dq[c] = dot_part<R>(S[c], qc);
-                dk[c] = beta ? dot_part<R>(S[c], kc) : 0.f;
+                dk[c] = delta ? dot_part<R>(S[c], kc) : 0.f;
             }
 #pragma unroll
             for (int off = 32 / LPC; off < 32; off <<= 1) {
 #pragma unroll
                 for (int c = 0; c < C; ++c) {
-                    if (beta) dk[c] += __shfl_xor_sync(0xffffffffu, dk[c], off);
+                    if (delta) dk[c] += __shfl_xor_sync(0xffffffffu, dk[c], off);
                     dq[c] += __shfl_xor_sync(0xffffffffu, dq[c], off);
                 }
             }
 #pragma unroll
             for (int c = 0; c < C; ++c) {
-                if (beta) w[c] = bc * (w[c] - gc * dk[c]);
+                if (delta) w[c] = bc * (w[c] - gc * dk[c]);
+                else if (beta) w[c] *= bc;
 #pragma unroll
                 for (int r = 0; r < R; ++r) S[c][r] = fmaf(kc[r], w[c], gc * S[c][r]);
                 const float o = fmaf(w[c], kqc, gc * dq[c]);
@@ -371,6 +373,181 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, int ld_o, con
         if (gain) y *= gain[e];
         if (gate) y *= silu_f(ns_ld(gate, (size_t)n * ld_gate + (size_t)h * V + e));
         ns_st(out, (size_t)n * ld_out + (size_t)h * V + e, y);
+    }
+}
+
+// ---------------------------------------------------------------------------------------
+// state space, preparation.  proj row: [z: H*V | x: H*V | B: G*D | C: G*D | dt: H | ...].  x, B and C (the C_ch = H*V + 2*G*D
+// channels from column H*V on) pass a causal convolution over time per channel (taps [n_taps, channels], one row per tap, the
+// last row the current token's; plus conv_bias; inputs before this step's first token come from the request's tail
+// [(n_taps - 1), channels] in its state) and silu, rounded to the activations' type; then
+//     step = softplus(dt + dt_bias[h]),   g = exp(-exp(A_log[h]) * step).
+// rec row (floats): [C: G*Dp | B: G*Dp | x: H*V | g: H | step: H | B . C: G], heads of B and C padded with zeros to Dp.
+// One block per token; VEC = 8: eight channels to a thread with 16-byte accesses.
+// ---------------------------------------------------------------------------------------
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+ssm_prepare_kernel(const T* __restrict__ proj, int ld_proj, const float* __restrict__ taps, const float* __restrict__ conv_bias,
+                   int n_taps, const float* __restrict__ a_log, const float* __restrict__ dt_bias, const float* __restrict__ state,
+                   long long state_floats, long long tail_off, const int* __restrict__ token_req, const int* __restrict__ qo_indptr,
+                   const int* __restrict__ state_slot, float* __restrict__ rec, int ld_rec, int G, int H, int D, int Dp, int V) {
+    ns_pdl_launch_dependents();
+    ns_pdl_wait();
+    extern __shared__ __align__(16) float bc[];  // B then C of the token, unpadded: the operands of B . C
+    const int n = blockIdx.x;
+    const int req = token_req[n];
+    if (req < 0) return;
+    const int inner = H * V, gd = G * D, C = inner + 2 * gd;
+    const int start = qo_indptr[req], t = n - start;
+    const float* tail = state + (long long)state_slot[req] * state_floats + tail_off;
+    float* out = rec + (size_t)n * ld_rec;
+    const T* x0 = proj + (size_t)start * ld_proj + inner;
+    for (int c = threadIdx.x * VEC; c < C; c += blockDim.x * VEC) {
+        float a[VEC], v[VEC], w[VEC];
+        if constexpr (VEC == 8) {
+            ld8(conv_bias + c, a);
+            for (int j = 0; j < n_taps; ++j) {
+                const int i = t - (n_taps - 1) + j;
+                if (i >= 0) ld8(x0 + (size_t)i * ld_proj + c, v);
+                else ld8(tail + (size_t)(i + n_taps - 1) * C + c, v);
+                ld8(taps + (size_t)j * C + c, w);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) a[k] = fmaf(w[k], v[k], a[k]);
+            }
+        } else {
+            a[0] = conv_bias[c];
+            for (int j = 0; j < n_taps; ++j) {
+                const int i = t - (n_taps - 1) + j;
+                v[0] = i >= 0 ? ns_ld(x0, (size_t)i * ld_proj + c) : tail[(size_t)(i + n_taps - 1) * C + c];
+                a[0] = fmaf(taps[(size_t)j * C + c], v[0], a[0]);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) a[k] = round_to<T>(silu_f(a[k]));
+        float* dst;
+        if (c < inner) {
+            dst = out + 2 * G * Dp + c;
+        } else {
+            const int b = c - inner;                       // feature of [B | C]
+            const int hd = b / D, e = b - hd * D;          // B heads 0 .. G - 1, then C heads
+            dst = out + (size_t)(hd < G ? G + hd : hd - G) * Dp + e;
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) bc[b + k] = a[k];
+        }
+        if constexpr (VEC == 8) st8(dst, a);
+        else dst[0] = a[0];
+    }
+    float* og = out + (size_t)2 * G * Dp + inner;
+    for (int h = threadIdx.x; h < H; h += blockDim.x) {
+        const float step = softplus_f(ns_ld(proj, (size_t)n * ld_proj + inner + C + h) + dt_bias[h]);
+        og[h] = expf(-expf(a_log[h]) * step);
+        og[H + h] = step;
+    }
+    for (int i = threadIdx.x; i < 2 * G * (Dp - D); i += blockDim.x) {
+        const int hd = i / (Dp - D);
+        out[(size_t)hd * Dp + D + (i - hd * (Dp - D))] = 0.f;
+    }
+    __syncthreads();
+    const int lane = threadIdx.x & 31;
+    for (int hd = threadIdx.x >> 5; hd < G; hd += blockDim.x >> 5) {
+        float s = 0.f;
+        for (int e = lane; e < D; e += 32) s = fmaf(bc[hd * D + e], bc[gd + hd * D + e], s);
+        s = ns_warp_sum(s);
+        if (lane == 0) og[2 * H + hd] = s;
+    }
+}
+
+// ---------------------------------------------------------------------------------------
+// state space, read-out to mixer output: u = (o + skip[h] * x) * silu(z) over the H*V features of a token, then each of `parts`
+// equal runs of features divided by its own root mean square (eps inside the root) and multiplied by gain; rounded once.
+// x lies in the preparation's rows (float), z in the projection.  One block per token, u in shared memory.  A request's last
+// block of the step also moves the convolution's tail on (nothing reads it any more in this step): conv_in is the first of the
+// C channels in the projection, see conv_tail_kernel.
+// ---------------------------------------------------------------------------------------
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+ssm_gate_norm_kernel(const float* __restrict__ o, int ld_o, const float* __restrict__ x, int ld_x, const T* __restrict__ z, int ld_z,
+                     const float* __restrict__ skip, const float* __restrict__ gain, float eps, int parts, T* __restrict__ out,
+                     int ld_out, const int* __restrict__ token_req, const int* __restrict__ qo_indptr, const int* __restrict__ state_slot,
+                     const T* __restrict__ conv_in, float* __restrict__ state, long long state_floats, long long tail_off, int C,
+                     int n_taps, int H, int V) {
+    ns_pdl_launch_dependents();
+    ns_pdl_wait();
+    extern __shared__ __align__(16) float u[];  // [H * V], then one partial sum per warp, then one scale per part
+    const int n = blockIdx.x;
+    const int req = token_req[n];
+    if (req < 0) return;
+    const int inner = H * V, L = inner / parts;
+    float* part_sum = u + inner;
+    float* part_inv = part_sum + 8;
+    for (int c = threadIdx.x * VEC; c < inner; c += blockDim.x * VEC) {
+        const float d = skip[c / V];  // (VEC features lie in one head)
+        if constexpr (VEC == 8) {
+            float a[8], b[8], g[8];
+            ld8(o + (size_t)n * ld_o + c, a);
+            ld8(x + (size_t)n * ld_x + c, b);
+            ld8(z + (size_t)n * ld_z + c, g);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) a[k] = fmaf(d, b[k], a[k]) * silu_f(g[k]);
+            st8(u + c, a);
+        } else {
+            u[c] = fmaf(d, x[(size_t)n * ld_x + c], o[(size_t)n * ld_o + c]) * silu_f(ns_ld(z, (size_t)n * ld_z + c));
+        }
+    }
+    __syncthreads();
+    // the 8 warps share the parts: one or several warps to a part, in passes when there are more parts than warps
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    int wpp = 1;  // warps per part, a power of two
+    while (wpp * 2 * parts <= 8) wpp *= 2;
+    const int at_once = 8 / wpp;
+    for (int p0 = 0; p0 < parts; p0 += at_once) {
+        const int p = p0 + warp / wpp;
+        float ss = 0.f;
+        if (p < parts)
+            for (int e = (warp % wpp) * 32 + lane; e < L; e += 32 * wpp) { const float v = u[p * L + e]; ss += v * v; }
+        ss = ns_warp_sum(ss);
+        if (wpp == 1) {
+            if (p < parts && lane == 0) part_inv[p] = rsqrtf(ss / (float)L + eps);
+        } else {
+            if (lane == 0) part_sum[warp] = ss;
+            __syncthreads();
+            if (p < parts && warp % wpp == 0 && lane == 0) {
+                float total = 0.f;
+                for (int k = 0; k < wpp; ++k) total += part_sum[warp + k];
+                part_inv[p] = rsqrtf(total / (float)L + eps);
+            }
+            __syncthreads();
+        }
+    }
+    __syncthreads();
+    for (int c = threadIdx.x * VEC; c < inner; c += blockDim.x * VEC) {
+        if constexpr (VEC == 8) {
+            float a[8], g[8];
+            ld8(u + c, a);
+            ld8(gain + c, g);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) a[k] = a[k] * part_inv[(c + k) / L] * g[k];
+            st8(out + (size_t)n * ld_out + c, a);
+        } else {
+            ns_st(out, (size_t)n * ld_out + c, u[c] * part_inv[c / L] * gain[c]);
+        }
+    }
+    const int start = qo_indptr[req], len = qo_indptr[req + 1] - start;
+    if (n_taps > 1 && n == start + len - 1) {
+        float* tail = state + (long long)state_slot[req] * state_floats + tail_off;
+        for (int c = threadIdx.x * VEC; c < C; c += blockDim.x * VEC) {
+            for (int j = 0; j < n_taps - 1; ++j) {  // ascending: entry j + len is read before it is written
+                const int i = len - (n_taps - 1) + j;
+                if constexpr (VEC == 8) {
+                    float a[8];
+                    if (i >= 0) ld8(conv_in + (size_t)(start + i) * ld_z + c, a);
+                    else ld8(tail + (size_t)(j + len) * C + c, a);
+                    st8(tail + (size_t)j * C + c, a);
+                } else {
+                    tail[(size_t)j * C + c] = i >= 0 ? ns_ld(conv_in, (size_t)(start + i) * ld_z + c) : tail[(size_t)(j + len) * C + c];
+                }
+            }
+        }
     }
 }
 
@@ -455,7 +632,7 @@ namespace {
 template <int R, int LPC, int C, bool ONE>
 int launch_scan_as(const float* q, const float* k, const float* v, const float* gate, const float* beta, const float* kq,
                 const float* decay, int ld, float* state, long long state_floats, const int* qo_indptr, const int* state_slot, float* out, int ld_out,
-                int n_requests, int H, int G, int D, int V, cudaStream_t stream) {
+                int n_requests, int H, int G, int D, int V, int delta, cudaStream_t stream) {
     using Sh = ScanShape<R, LPC, C, ONE>;
     static bool configured = false;
     if (!configured && Sh::kBytes > 48 * 1024) {
@@ -465,7 +642,7 @@ int launch_scan_as(const float* q, const float* k, const float* v, const float* 
     const int col_blocks = (V + Sh::kCols - 1) / Sh::kCols;
     if (H > 65535 || col_blocks > 65535) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_linear_scan: %d heads of %d columns exceed the grid", H, V);
     NS_LAUNCH((linear_scan_kernel<R, LPC, C, ONE>), dim3(n_requests, H, col_blocks), 128, Sh::kBytes, stream, q, k, v, gate, beta, kq, decay, ld,
-              state, state_floats, qo_indptr, state_slot, out, ld_out, H, G, D, V);
+              state, state_floats, qo_indptr, state_slot, out, ld_out, H, G, D, V, delta);
     NS_CHECK_LAUNCH("ns_linear_scan");
     return NS_OK;
 }
@@ -473,12 +650,12 @@ int launch_scan_as(const float* q, const float* k, const float* v, const float* 
 template <int R, int LPC, int C>
 int launch_scan(const float* q, const float* k, const float* v, const float* gate, const float* beta, const float* kq,
                 const float* decay, int ld, float* state, long long state_floats, const int* qo_indptr, const int* state_slot,
-                float* out, int ld_out, int n_requests, int H, int G, int D, int V, cudaStream_t stream, int longest) {
+                float* out, int ld_out, int n_requests, int H, int G, int D, int V, int delta, cudaStream_t stream, int longest) {
     if (longest <= 1)
         return launch_scan_as<R, LPC, C, true>(q, k, v, gate, beta, kq, decay, ld, state, state_floats, qo_indptr, state_slot, out,
-                                               ld_out, n_requests, H, G, D, V, stream);
+                                               ld_out, n_requests, H, G, D, V, delta, stream);
     return launch_scan_as<R, LPC, C, false>(q, k, v, gate, beta, kq, decay, ld, state, state_floats, qo_indptr, state_slot, out,
-                                            ld_out, n_requests, H, G, D, V, stream);
+                                            ld_out, n_requests, H, G, D, V, delta, stream);
 }
 }  // namespace
 
@@ -493,12 +670,13 @@ NS_API int ns_linear_scan_lanes(int lanes) {
 // per column instead of four: twice the blocks and half the work per token and lane.
 NS_API int ns_linear_scan(const float* q, const float* k, const float* v, const float* gate, const float* beta, const float* kq,
                           const float* decay, int ld, float* state, long long state_floats, const int* qo_indptr, const int* state_slot, float* out,
-                          int ld_out, int n_requests, int H, int G, int D, int V, int longest, int n_sms, cudaStream_t stream) {
+                          int ld_out, int n_requests, int H, int G, int D, int V, int delta, int longest, int n_sms, cudaStream_t stream) {
     if (n_requests <= 0) return NS_OK;
     const int R4 = ns_linear_scan_rows(D);
     if (!R4) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_linear_scan: a head of %d features (at most 256)", D);
     if (G < 1 || H % G) NS_FAIL(NS_ERR_ARGUMENT, "ns_linear_scan: %d heads over %d key heads", H, G);
     if (!gate && !decay) NS_FAIL(NS_ERR_ARGUMENT, "ns_linear_scan: neither a gate per token nor a decay per head");
+    if (delta && !beta) NS_FAIL(NS_ERR_ARGUMENT, "ns_linear_scan: the delta rule needs a write strength per token");
     if (!kq) NS_FAIL(NS_ERR_ARGUMENT, "ns_linear_scan: no k . q per token");
     if (ld % 4 || ((uintptr_t)q | (uintptr_t)k) % 16) NS_FAIL(NS_ERR_ARGUMENT, "ns_linear_scan: q and k rows must be 16-byte aligned");
     // Many tokens to walk and few columns to walk them on: eight lanes per column, whose sums per lane are half as long
@@ -508,7 +686,7 @@ NS_API int ns_linear_scan(const float* q, const float* k, const float* v, const 
     const long long blocks4 = (long long)n_requests * H * ((V + 31) / 32);
     const int sms = n_sms > 0 ? n_sms : 148;
     const int lanes = g_scan_lanes == 4 || g_scan_lanes == 8 ? g_scan_lanes : (longest >= 64 && R4 >= 8 && blocks4 < 4ll * sms ? 8 : 4);
-#define NS_SCAN_ARGS q, k, v, gate, beta, kq, decay, ld, state, state_floats, qo_indptr, state_slot, out, ld_out, n_requests, H, G, D, V, stream, longest
+#define NS_SCAN_ARGS q, k, v, gate, beta, kq, decay, ld, state, state_floats, qo_indptr, state_slot, out, ld_out, n_requests, H, G, D, V, delta, stream, longest
     switch (R4) {
         case 4: return launch_scan<4, 4, 1>(NS_SCAN_ARGS);
         case 8: return lanes == 8 ? launch_scan<4, 8, 1>(NS_SCAN_ARGS) : launch_scan<8, 4, 1>(NS_SCAN_ARGS);
@@ -534,5 +712,56 @@ NS_API int ns_head_norm_gate(const float* o, int ld_o, const void* gate, int ld_
     else
         NS_FAIL(NS_ERR_ARGUMENT, "ns_head_norm_gate: unknown dtype %d", dtype);
     NS_CHECK_LAUNCH("ns_head_norm_gate");
+    return NS_OK;
+}
+
+NS_API int ns_ssm_prepare(const void* proj, int ld_proj, const float* taps, const float* conv_bias, int n_taps, const float* a_log,
+                          const float* dt_bias, const float* state, long long state_floats, long long tail_off, const int* token_req,
+                          const int* qo_indptr, const int* state_slot, float* rec, int ld_rec, int n_tokens, int G, int H, int D, int Dp,
+                          int V, int dtype, cudaStream_t stream) {
+    if (n_tokens <= 0) return NS_OK;
+    if (n_taps < 1 || G < 1 || H % G || Dp < D || Dp % 4) NS_FAIL(NS_ERR_ARGUMENT, "ns_ssm_prepare: taps=%d heads=%d/%d D=%d Dp=%d", n_taps, H, G, D, Dp);
+    if (dtype != NS_F32 && dtype != NS_BF16) NS_FAIL(NS_ERR_ARGUMENT, "ns_ssm_prepare: unknown dtype %d", dtype);
+    const size_t smem = (size_t)2 * G * D * sizeof(float);
+    if (smem > 48 * 1024) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_ssm_prepare: %d groups of %d features do not fit shared memory", G, D);
+    const size_t esz = dtype == NS_F32 ? 4 : 2;
+    const bool vec = (H * V) % 8 == 0 && D % 8 == 0 && (ld_proj * esz) % 16 == 0 && ld_rec % 4 == 0 && state_floats % 4 == 0 && tail_off % 4 == 0 &&
+                     (((uintptr_t)proj | (uintptr_t)taps | (uintptr_t)conv_bias | (uintptr_t)state | (uintptr_t)rec) % 16 == 0);
+#define NS_SSM_PREPARE(T, VC)                                                                                                         \
+    NS_LAUNCH((ssm_prepare_kernel<T, VC>), n_tokens, 256, smem, stream, (const T*)proj, ld_proj, taps, conv_bias, n_taps, a_log, dt_bias, \
+              state, state_floats, tail_off, token_req, qo_indptr, state_slot, rec, ld_rec, G, H, D, Dp, V)
+    if (dtype == NS_F32) { if (vec) NS_SSM_PREPARE(float, 8); else NS_SSM_PREPARE(float, 1); }
+    else { if (vec) NS_SSM_PREPARE(__nv_bfloat16, 8); else NS_SSM_PREPARE(__nv_bfloat16, 1); }
+#undef NS_SSM_PREPARE
+    NS_CHECK_LAUNCH("ns_ssm_prepare");
+    return NS_OK;
+}
+
+// proj [n, ld_proj]: z at column 0, the convolution's C inputs from column H * V on; x: the preparation's rows
+NS_API int ns_ssm_gate_norm(const float* o, int ld_o, const float* x, int ld_x, const void* proj, int ld_proj, const float* skip,
+                            const float* gain, float eps, int parts, void* out, int ld_out, const int* token_req, const int* qo_indptr,
+                            const int* state_slot, float* state, long long state_floats, long long tail_off, int C, int n_taps,
+                            int n_tokens, int H, int V, int dtype, cudaStream_t stream) {
+    if (n_tokens <= 0) return NS_OK;
+    const int inner = H * V;
+    if (parts < 1 || inner % parts) NS_FAIL(NS_ERR_ARGUMENT, "ns_ssm_gate_norm: %d features in %d parts", inner, parts);
+    if (dtype != NS_F32 && dtype != NS_BF16) NS_FAIL(NS_ERR_ARGUMENT, "ns_ssm_gate_norm: unknown dtype %d", dtype);
+    const size_t smem = (size_t)(inner + 8 + parts) * sizeof(float);
+    if (smem > 200 * 1024) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_ssm_gate_norm: a row of %d features in %d parts does not fit shared memory", inner, parts);
+    const size_t esz = dtype == NS_F32 ? 4 : 2;
+    const bool vec = V % 8 == 0 && C % 8 == 0 && ld_o % 4 == 0 && ld_x % 4 == 0 && (ld_proj * esz) % 16 == 0 && (ld_out * esz) % 16 == 0 &&
+                     state_floats % 4 == 0 && tail_off % 4 == 0 &&
+                     (((uintptr_t)o | (uintptr_t)x | (uintptr_t)proj | (uintptr_t)gain | (uintptr_t)out | (uintptr_t)state) % 16 == 0);
+#define NS_SSM_GATE(T, VC)                                                                                                               \
+    {                                                                                                                                    \
+        if (smem > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(ssm_gate_norm_kernel<T, VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
+        NS_LAUNCH((ssm_gate_norm_kernel<T, VC>), n_tokens, 256, smem, stream, o, ld_o, x, ld_x, (const T*)proj, ld_proj, skip, gain, eps,  \
+                  parts, (T*)out, ld_out, token_req, qo_indptr, state_slot, (const T*)proj + inner, state, state_floats, tail_off, C,     \
+                  n_taps, H, V);                                                                                                         \
+    }
+    if (dtype == NS_F32) { if (vec) NS_SSM_GATE(float, 8) else NS_SSM_GATE(float, 1) }
+    else { if (vec) NS_SSM_GATE(__nv_bfloat16, 8) else NS_SSM_GATE(__nv_bfloat16, 1) }
+#undef NS_SSM_GATE
+    NS_CHECK_LAUNCH("ns_ssm_gate_norm");
     return NS_OK;
 }

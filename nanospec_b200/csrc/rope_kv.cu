@@ -222,8 +222,10 @@ NS_API int ns_rope_kv_write(void* qkv, const int* positions, const int* token_re
 //   angle = float(position) * inv_freq[i]; cos and sin are multiplied by `magnitude`
 // A row of `qkv` is [q: nq*d | k: nkv*d | v: nkv*dv]; q and k are rewritten in place, k and v go to
 // cache[page, kv head, offset, :] (keys d wide, values dv wide) when write_kv.  `bias` (optional, float, laid out like
-// the row) is the projections' bias: it is added before the norm, and v is stored with it.  One block per token;
-// everything is computed in float and rounded once.
+// the row) is the projections' bias: it is added before the norm, and v is stored with it.  `v_norm`: every head's value
+// is divided by its root mean square over its dv features (eps inside the root, no gain) before it is stored.  One block
+// per token; everything is computed in float and rounded once; the token's sines and cosines are computed once, into
+// shared memory, for all of its heads.
 // ---------------------------------------------------------------------------------------
 namespace {
 
@@ -234,15 +236,24 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, int row_stride, const int* __rest
                           const float* __restrict__ inv_freq, float magnitude, int interleaved, int rot_pairs,
                           const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
                           T* __restrict__ k_cache, T* __restrict__ v_cache, int page_size, int nq, int nkv, int d, int dv,
-                          int write_kv, const float* __restrict__ bias) {
+                          int write_kv, const float* __restrict__ bias, int v_norm) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
+    extern __shared__ float rot_sn[];      // sines of the rotated pairs, then their cosines
+    float* rot_cs = rot_sn + rot_pairs;
     const int n = blockIdx.x;
     const int req = token_req[n];
     if (req < 0) return;
     const int pos = positions[n];
     T* row = qkv + (size_t)n * row_stride;
     const int q_size = nq * d, k_size = nkv * d;
+    for (int i = threadIdx.x; i < rot_pairs; i += blockDim.x) {
+        float sn, cs;
+        sincosf((float)pos * inv_freq[i], &sn, &cs);
+        rot_sn[i] = sn * magnitude;
+        rot_cs[i] = cs * magnitude;
+    }
+    __syncthreads();
     float inv_q = 1.f, inv_k = 1.f;
     if (q_gain || k_gain) {
         // both sums of squares in one pass over the row (16-byte reads when the row allows), one exchange for the two
@@ -284,10 +295,9 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, int row_stride, const int* __rest
         const int page = block_table[(size_t)req * table_stride + pos / page_size];
         slot = (size_t)page * nkv * page_size + (size_t)(pos % page_size);  // + kv head * page_size
     }
-    const float fpos = (float)pos;
     // 16-byte accesses: eight features at a time, when heads, the rotated part and the rows allow it
     const bool vec = d % 8 == 0 && (2 * rot_pairs) % 8 == 0 && (interleaved || rot_pairs % 8 == 0) && row_stride % 8 == 0 &&
-                     (uintptr_t)qkv % 16 == 0 && (!write_kv || (((uintptr_t)k_cache | (uintptr_t)v_cache) % 16 == 0 && dv % 8 == 0)) &&
+                     (uintptr_t)qkv % 16 == 0 && (!write_kv || (((uintptr_t)k_cache | (uintptr_t)v_cache) % 16 == 0 && dv % 8 == 0 && (!v_norm || dv <= 256))) &&
                      (!q_gain || (uintptr_t)q_gain % 16 == 0) && (!k_gain || (uintptr_t)k_gain % 16 == 0) &&
                      (!bias || (uintptr_t)bias % 16 == 0);
     if (vec) {
@@ -338,9 +348,7 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, int row_stride, const int* __rest
                 }
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    float sn, cs;
-                    sincosf(fpos * inv_freq[it * 4 + i], &sn, &cs);
-                    sn *= magnitude; cs *= magnitude;
+                    const float sn = rot_sn[it * 4 + i], cs = rot_cs[it * 4 + i];
                     const float a = x[2 * i], b = x[2 * i + 1];
                     x[2 * i] = a * cs - b * sn;
                     x[2 * i + 1] = b * cs + a * sn;
@@ -372,9 +380,7 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, int row_stride, const int* __rest
                 }
 #pragma unroll
                 for (int i = 0; i < 8; ++i) {
-                    float sn, cs;
-                    sincosf(fpos * inv_freq[e + i], &sn, &cs);
-                    sn *= magnitude; cs *= magnitude;
+                    const float sn = rot_sn[e + i], cs = rot_cs[e + i];
                     const float a = lo[i], b = hi[i];
                     lo[i] = a * cs - b * sn;
                     hi[i] = b * cs + a * sn;
@@ -386,6 +392,36 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, int row_stride, const int* __rest
         }
         if (write_kv) {
             const T* v = row + q_size + k_size;
+            if (v_norm) {
+                // a head to `lanes` lanes of a warp, eight features to a lane
+                int lanes = 1;
+                while (lanes * 8 < dv) lanes <<= 1;
+                const int per_pass = blockDim.x / lanes;
+                for (int h0 = 0; h0 < nkv; h0 += per_pass) {
+                    const int h = h0 + threadIdx.x / lanes, e = (threadIdx.x % lanes) * 8;
+                    const bool mine = h < nkv && e < dv;
+                    float x[8], ss = 0.f;
+                    if (mine) {
+                        ld8(v + h * dv + e, x);
+                        if (bias) {
+                            float b[8];
+                            ld8(bias + q_size + k_size + h * dv + e, b);
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) x[i] += b[i];
+                        }
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) ss += x[i] * x[i];
+                    }
+                    for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+                    if (mine) {
+                        const float inv = rsqrtf(ss / (float)dv + eps);
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) x[i] *= inv;
+                        st8(v_cache + (slot + (size_t)h * page_size) * dv + e, x);
+                    }
+                }
+                return;
+            }
             for (int w = threadIdx.x; w < nkv * dv / 8; w += blockDim.x) {
                 const int h = (w * 8) / dv, e = w * 8 - h * dv;
                 float x[8];
@@ -415,9 +451,7 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, int row_stride, const int* __rest
             float a = ns_ld(row, base + e0), b = ns_ld(row, base + e1);
             if (bias) { a += bias[base + e0]; b += bias[base + e1]; }
             if (gain) { a = a * inv * gain[goff + e0]; b = b * inv * gain[goff + e1]; }
-            float sn, cs;
-            sincosf(fpos * inv_freq[u], &sn, &cs);
-            sn *= magnitude; cs *= magnitude;
+            const float sn = rot_sn[u], cs = rot_cs[u];
             const float ra = a * cs - b * sn, rb = b * cs + a * sn;
             ns_st(row, base + e0, ra); ns_st(row, base + e1, rb);
             if (kc) { ns_st(kc, e0, ra); ns_st(kc, e1, rb); }
@@ -432,6 +466,22 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, int row_stride, const int* __rest
     }
     if (write_kv) {
         const T* v = row + q_size + k_size;
+        if (v_norm) {  // a warp per head
+            const int lane = threadIdx.x & 31;
+            for (int h = threadIdx.x >> 5; h < nkv; h += blockDim.x >> 5) {
+                float ss = 0.f;
+                for (int e = lane; e < dv; e += 32) {
+                    const float x = ns_ld(v, h * dv + e) + (bias ? bias[q_size + k_size + h * dv + e] : 0.f);
+                    ss += x * x;
+                }
+                const float inv = rsqrtf(ns_warp_sum(ss) / (float)dv + eps);
+                for (int e = lane; e < dv; e += 32) {
+                    const float x = ns_ld(v, h * dv + e) + (bias ? bias[q_size + k_size + h * dv + e] : 0.f);
+                    ns_st(v_cache, (slot + (size_t)h * page_size) * dv + e, x * inv);
+                }
+            }
+            return;
+        }
         for (int w = threadIdx.x; w < nkv * dv; w += blockDim.x) {
             const int h = w / dv, e = w - h * dv;
             ns_st(v_cache, (slot + (size_t)h * page_size) * dv + e, ns_ld(v, w) + (bias ? bias[q_size + k_size + w] : 0.f));
@@ -445,19 +495,21 @@ NS_API int ns_qk_norm_rope_store(void* qkv, int row_stride, const int* positions
                                  int table_stride, const float* inv_freq, float magnitude, int interleaved, int rot_pairs,
                                  const float* q_gain, const float* k_gain, float eps, void* k_cache, void* v_cache,
                                  int page_size, int nq, int nkv, int d, int dv, int n_tokens, int write_kv, int dtype,
-                                 const float* bias, cudaStream_t stream) {
+                                 const float* bias, int v_norm, cudaStream_t stream) {
     if (n_tokens <= 0) return NS_OK;
     if (rot_pairs < 0 || 2 * rot_pairs > d) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_qk_norm_rope_store: %d pairs in a head of %d", rot_pairs, d);
     if (rot_pairs > 0 && !inv_freq) NS_FAIL(NS_ERR_ARGUMENT, "ns_qk_norm_rope_store: no frequencies");
     if (write_kv && (!k_cache || !v_cache || !block_table)) NS_FAIL(NS_ERR_ARGUMENT, "ns_qk_norm_rope_store: no cache to write");
+    const size_t smem = 2 * (size_t)rot_pairs * sizeof(float);
+    if (smem > 48 * 1024) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_qk_norm_rope_store: %d rotated pairs do not fit shared memory", rot_pairs);
     if (dtype == NS_F32)
-        NS_LAUNCH((qk_norm_rope_store_kernel<float>), n_tokens, 256, 0, stream, (float*)qkv, row_stride, positions, token_req,
+        NS_LAUNCH((qk_norm_rope_store_kernel<float>), n_tokens, 256, smem, stream, (float*)qkv, row_stride, positions, token_req,
                   block_table, table_stride, inv_freq, magnitude, interleaved, rot_pairs, q_gain, k_gain, eps, (float*)k_cache,
-                  (float*)v_cache, page_size, nq, nkv, d, dv, write_kv, bias);
+                  (float*)v_cache, page_size, nq, nkv, d, dv, write_kv, bias, v_norm);
     else if (dtype == NS_BF16)
-        NS_LAUNCH((qk_norm_rope_store_kernel<__nv_bfloat16>), n_tokens, 256, 0, stream, (__nv_bfloat16*)qkv, row_stride, positions,
+        NS_LAUNCH((qk_norm_rope_store_kernel<__nv_bfloat16>), n_tokens, 256, smem, stream, (__nv_bfloat16*)qkv, row_stride, positions,
                   token_req, block_table, table_stride, inv_freq, magnitude, interleaved, rot_pairs, q_gain, k_gain, eps,
-                  (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, page_size, nq, nkv, d, dv, write_kv, bias);
+                  (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, page_size, nq, nkv, d, dv, write_kv, bias, v_norm);
     else
         NS_FAIL(NS_ERR_ARGUMENT, "ns_qk_norm_rope_store: unknown dtype %d", dtype);
     NS_CHECK_LAUNCH("ns_qk_norm_rope_store");

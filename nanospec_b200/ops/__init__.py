@@ -114,8 +114,12 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0) -> torch.Te
     runs of `block` features instead (gate j at (j // block) * 2 * block + j % block, up `block` further)."""
     _cuda(gate_up, out)
     n, inter = out.shape
-    if gate_up.shape != (n, 2 * inter) or gate_up.dtype != out.dtype or not (gate_up.is_contiguous() and out.is_contiguous()):
-        raise KernelError("swiglu: gate_up must be [N, 2I] and out [N, I], same dtype, contiguous")
+    if gate_up.shape != (n, 2 * inter) or gate_up.dtype != out.dtype or gate_up.stride(1) != 1 or out.stride(1) != 1:
+        raise KernelError("swiglu: gate_up must be [N, 2I] and out [N, I], same dtype, rows with unit inner stride")
+    if not (gate_up.is_contiguous() and out.is_contiguous()):  # column ranges of wider buffers
+        lib.call("ns_swiglu_rows", gate_up.data_ptr(), gate_up.stride(0), out.data_ptr(), out.stride(0), n, inter, int(block),
+                 dtype_code(out.dtype), _stream())
+        return out
     lib.call("ns_swiglu", gate_up.data_ptr(), out.data_ptr(), n, inter, int(block), dtype_code(out.dtype), _stream())
     return out
 
@@ -807,12 +811,13 @@ def scale_softcap(logits: torch.Tensor, scale: float = 1.0, cap: float = 0.0) ->
 def qk_norm_rope_store(qkv: torch.Tensor, ctx, lane, inv_freq: torch.Tensor | None, magnitude: float, interleaved: bool,
                        nq: int, nkv: int, head_dim: int, v_dim: int, q_gain: torch.Tensor | None = None,
                        k_gain: torch.Tensor | None = None, eps: float = 0.0, write_kv: bool = True,
-                       bias: torch.Tensor | None = None) -> None:
+                       bias: torch.Tensor | None = None, v_norm: bool = False) -> None:
     """Rows [q: nq*head_dim | k: nkv*head_dim | v: nkv*v_dim]: an RMS norm of the whole q and of the whole k projection
     (when gains are given), a rotation of the first 2 * len(inv_freq) features of each head (pairs (2i, 2i+1) when
     `interleaved`, (i, i + len) otherwise; cos and sin times `magnitude`), q and k rewritten in place, k and v stored at
     the tokens' cache slots when `write_kv` (csrc/rope_kv.cu).  `bias` (float32, one entry per feature of the row): the
-    projections' bias, added before the norm.  `nkv` 0: rows of q alone (a mixer that reads another's keys and values)."""
+    projections' bias, added before the norm.  `nkv` 0: rows of q alone (a mixer that reads another's keys and values).
+    `v_norm`: each head's value is divided by its root mean square (`eps` inside the root) before it is stored."""
     _cuda(qkv, inv_freq, q_gain, k_gain, bias)
     if bias is not None and (bias.dtype != torch.float32 or not bias.is_contiguous() or bias.numel() != nq * head_dim + nkv * (head_dim + v_dim)):
         raise KernelError("qk_norm_rope_store: a contiguous float32 bias with one entry per feature of [q | k | v]")
@@ -832,7 +837,7 @@ def qk_norm_rope_store(qkv: torch.Tensor, ctx, lane, inv_freq: torch.Tensor | No
              _ptr(bt), bt.stride(0) if bt is not None else 0, _ptr(inv_freq), float(magnitude), int(bool(interleaved)),
              inv_freq.numel() if inv_freq is not None else 0, _ptr(q_gain), _ptr(k_gain), float(eps),
              _ptr(lane.k) if write_kv else None, _ptr(lane.v) if write_kv else None, lane.page_size, nq, nkv, head_dim, v_dim, n,
-             int(bool(write_kv)), dtype_code(qkv.dtype), _ptr(bias), _stream())
+             int(bool(write_kv)), dtype_code(qkv.dtype), _ptr(bias), int(bool(v_norm)), _stream())
 
 
 def scan_padded_dim(head_dim: int) -> int:
@@ -872,10 +877,10 @@ def rotary_prepare(proj: torch.Tensor, ctx, inv_freq: torch.Tensor | None, magni
 
 
 def linear_scan(rec: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, heads: int, kv_heads: int, head_dim: int, v_dim: int,
-                decay: torch.Tensor | None = None, gated: bool = False) -> torch.Tensor:
+                decay: torch.Tensor | None = None, gated: bool = False, delta: bool = True) -> torch.Tensor:
     """The recurrence over each request's tokens of this step (csrc/recurrent.cu).  `rec` rows, as the preparation kernels write
-    them: [q: kv_heads*Dp | k: kv_heads*Dp | v: heads*v_dim], then, when `gated` (the delta rule), [g: heads | beta: heads], then
-    [k . q: kv_heads]; without `gated`, `decay` [heads] float32.
+    them: [q: kv_heads*Dp | k: kv_heads*Dp | v: heads*v_dim], then, when `gated`, [g: heads | beta: heads] (the delta rule, or with
+    `delta` False the state space, whose write is beta * v), then [k . q: kv_heads]; without `gated`, `decay` [heads] float32.
     `state` [slots, floats] holds S [heads, head_dim, v_dim] at the start of each slot's row; `out` [N, heads*v_dim] float32."""
     _cuda(rec, state, out, decay)
     dp = scan_padded_dim(head_dim)
@@ -893,7 +898,52 @@ def linear_scan(rec: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, 
     lib.call("ns_linear_scan", base, base + 4 * kv_heads * dp, base + 4 * off_v, g_ptr, b_ptr, base + 4 * off_kq,
              None if gated else decay.data_ptr(),
              rec.stride(0), state.data_ptr(), state.stride(0), ctx.qo_indptr.data_ptr(), ctx.state_slot.data_ptr(), out.data_ptr(),
-             out.stride(0), ctx.n_requests, heads, kv_heads, head_dim, v_dim, int(ctx.max_q_len or 1), sm_count(), _stream())
+             out.stride(0), ctx.n_requests, heads, kv_heads, head_dim, v_dim, int(bool(gated and delta)), int(ctx.max_q_len or 1), sm_count(), _stream())
+    return out
+
+
+def ssm_prepare(proj: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                state: torch.Tensor, tail_off: int, ctx, rec: torch.Tensor, groups: int, heads: int, state_dim: int, v_dim: int) -> None:
+    """Rows [z: heads*v_dim | x: heads*v_dim | B: groups*state_dim | C: groups*state_dim | dt: heads | ...] of `proj`: x, B and C
+    through a short convolution per channel (`taps` [n, channels], one row per tap, the last the current token's; `conv_bias`) and
+    silu, step sizes softplus(dt + dt_bias), decays exp(-exp(a_log) step), into the float32 rows [C | B | x | decay | step | B . C]
+    of `rec` that `linear_scan(..., gated=True, delta=False)` reads.  The last n - 1 inputs of every request lie in `state` at
+    `tail_off`; `ssm_gate_norm` moves them on."""
+    _cuda(proj, taps, conv_bias, a_log, dt_bias, state, rec)
+    channels = heads * v_dim + 2 * groups * state_dim
+    for t, size, name in ((taps, None, "taps"), (conv_bias, channels, "conv_bias"), (a_log, heads, "a_log"), (dt_bias, heads, "dt_bias")):
+        if t.dtype != torch.float32 or not t.is_contiguous() or (size is not None and t.numel() != size):
+            raise KernelError(f"ssm_prepare: {name} must be contiguous float32" + (f" of {size} entries" if size else ""))
+    dp = scan_padded_dim(state_dim)
+    if taps.dim() != 2 or taps.shape[1] != channels or proj.stride(1) != 1 or proj.shape[1] < heads * v_dim + channels + heads \
+            or rec.dtype != torch.float32 or rec.stride(1) != 1 or rec.shape[1] < 2 * groups * dp + heads * v_dim + 2 * heads + groups \
+            or state.dtype != torch.float32 or not state.is_contiguous() or state.shape[1] < tail_off + (taps.shape[0] - 1) * channels:
+        raise KernelError("ssm_prepare: operands do not have the sizes that the heads, groups and taps need")
+    lib.call("ns_ssm_prepare", proj.data_ptr(), proj.stride(0), taps.data_ptr(), conv_bias.data_ptr(), taps.shape[0], a_log.data_ptr(),
+             dt_bias.data_ptr(), state.data_ptr(), state.stride(0), int(tail_off), ctx.token_req.data_ptr(), ctx.qo_indptr.data_ptr(),
+             ctx.state_slot.data_ptr(), rec.data_ptr(), rec.stride(0), proj.shape[0], groups, heads, state_dim, dp, v_dim,
+             dtype_code(proj.dtype), _stream())
+
+
+def ssm_gate_norm(o: torch.Tensor, x: torch.Tensor, proj: torch.Tensor, skip: torch.Tensor, gain: torch.Tensor, eps: float, parts: int,
+                  out: torch.Tensor, state: torch.Tensor, tail_off: int, channels: int, n_taps: int, ctx, heads: int, v_dim: int) -> torch.Tensor:
+    """out = norm((o + skip[h] * x) * silu(z)) * gain: `o` the scan's read-out and `x` its input (float32), z the leading columns of
+    `proj`, the norm an RMS norm of each of `parts` equal runs of the heads' features.  Afterwards every request's convolution
+    tail holds its last n_taps - 1 inputs (the `channels` columns of `proj` behind z)."""
+    _cuda(o, x, proj, skip, gain, out, state)
+    inner = heads * v_dim
+    if o.dtype != torch.float32 or x.dtype != torch.float32 or o.shape[1] < inner or x.shape[1] < inner or o.stride(1) != 1 or x.stride(1) != 1 \
+            or proj.stride(1) != 1 or out.stride(1) != 1 or out.dtype != proj.dtype or out.shape != (proj.shape[0], inner) \
+            or proj.shape[1] < inner + channels or state.dtype != torch.float32 or not state.is_contiguous() \
+            or state.shape[1] < tail_off + (n_taps - 1) * channels:
+        raise KernelError("ssm_gate_norm: operands do not have the sizes that the heads and taps need")
+    for t, size, name in ((skip, heads, "skip"), (gain, inner, "gain")):
+        if t.dtype != torch.float32 or not t.is_contiguous() or t.numel() != size:
+            raise KernelError(f"ssm_gate_norm: {name} must be contiguous float32 of {size} entries")
+    lib.call("ns_ssm_gate_norm", o.data_ptr(), o.stride(0), x.data_ptr(), x.stride(0), proj.data_ptr(), proj.stride(0), skip.data_ptr(),
+             gain.data_ptr(), float(eps), int(parts), out.data_ptr(), out.stride(0), ctx.token_req.data_ptr(), ctx.qo_indptr.data_ptr(),
+             ctx.state_slot.data_ptr(), state.data_ptr(), state.stride(0), int(tail_off), int(channels), int(n_taps), proj.shape[0], heads,
+             v_dim, dtype_code(proj.dtype), _stream())
     return out
 
 
@@ -1032,23 +1082,26 @@ def attention_latent(q_lat: torch.Tensor, q_rot: torch.Tensor, lane, ctx, out: t
     return out
 
 
-ACTIVATIONS = {"gelu_erf": 0, "gelu_tanh": 1, "silu": 2, "relu2": 3}
+ACTIVATIONS = {"gelu_erf": 0, "gelu_tanh": 1, "silu": 2, "relu2": 3, "xielu": 4}
 
 
-def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> torch.Tensor:
-    """out = act(x) elementwise in float, rounded once: "gelu_erf" (the exact gelu), "gelu_tanh", "silu", "relu2" (the square of relu)."""
-    _cuda(x, out)
+def activation(x: torch.Tensor, out: torch.Tensor, kind: str, coef: torch.Tensor | None = None) -> torch.Tensor:
+    """out = act(x) elementwise in float, rounded once: "gelu_erf" (the exact gelu), "gelu_tanh", "silu", "relu2" (the square of relu),
+    "xielu" (x > 0: a x^2 + x / 2; x <= 0: b (exp(x) - 1 - x) + x / 2, with a, b = `coef`, two float32 on the device)."""
+    _cuda(x, out, coef)
+    if kind == "xielu" and (coef is None or coef.dtype != torch.float32 or coef.numel() != 2 or not coef.is_contiguous()):
+        raise KernelError("activation: xielu takes two contiguous float32 coefficients")
     if kind not in ACTIVATIONS:
         raise KernelError(f"activation: unknown kind {kind!r} (known: {', '.join(ACTIVATIONS)})")
     if x.shape == out.shape and x.dtype == out.dtype and x.dim() == 2 and x.stride(1) == 1 and out.stride(1) == 1 \
             and not (x.is_contiguous() and out.is_contiguous()):
         # column ranges of wider buffers: rows with strides of their own
         lib.call("ns_activation_rows", x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), x.shape[0], x.shape[1], ACTIVATIONS[kind],
-                 dtype_code(x.dtype), _stream())
+                 _ptr(coef), dtype_code(x.dtype), _stream())
         return out
     if x.shape != out.shape or x.dtype != out.dtype or not (x.is_contiguous() and out.is_contiguous()):
         raise KernelError("activation: operands of one shape and dtype, contiguous or rows with unit inner stride")
-    lib.call("ns_activation", x.data_ptr(), out.data_ptr(), x.numel(), ACTIVATIONS[kind], dtype_code(x.dtype), _stream())
+    lib.call("ns_activation", x.data_ptr(), out.data_ptr(), x.numel(), ACTIVATIONS[kind], _ptr(coef), dtype_code(x.dtype), _stream())
     return out
 
 
@@ -1082,21 +1135,24 @@ def router_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch=N
 
 
 def moe_route(logits: torch.Tensor, groups: int, keep: int, top: int, scale: float, ids: torch.Tensor, weights: torch.Tensor,
-              softmax: bool = False) -> None:
+              softmax: bool = False, correction: torch.Tensor | None = None, renormalize: bool = True) -> None:
     """Per row of float32 logits [N, E]: the chosen experts (int32 [N, top], largest score first) and their weights
-    (float32 [N, top]); see csrc/moe.cu for the rule."""
-    _cuda(logits, ids, weights)
+    (float32 [N, top]); see csrc/moe.cu for the rule.  `correction` [E] float32 is added to the scores that choose, not to the
+    weights; `renormalize`: the weights are divided by the sum of the chosen scores before they are scaled."""
+    _cuda(logits, ids, weights, correction)
+    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != logits.shape[1] or not correction.is_contiguous()):
+        raise KernelError("moe_route: one contiguous float32 correction per expert")
     n, E = logits.shape
     if logits.dtype != torch.float32 or not logits.is_contiguous() or ids.dtype != torch.int32 or weights.dtype != torch.float32 \
             or ids.shape != (n, top) or weights.shape != (n, top) or not (ids.is_contiguous() and weights.is_contiguous()):
         raise KernelError("moe_route: float32 logits [N, E], int32 ids and float32 weights [N, top], contiguous")
     lib.call("ns_moe_route", logits.data_ptr(), n, E, int(groups), int(keep), int(top), float(scale), int(bool(softmax)),
-             ids.data_ptr(), weights.data_ptr(), _stream())
+             _ptr(correction), int(bool(renormalize)), ids.data_ptr(), weights.data_ptr(), _stream())
 
 
 def moe_plan(ids: torch.Tensor, n_experts: int, offsets: torch.Tensor, row_of: torch.Tensor, pair_of: torch.Tensor | None = None) -> None:
     """offsets [E + 1] (running counts per expert), row_of [N, top] (each pair's row where every expert's tokens lie
-    side by side) and, when given, pair_of (the pair at each row), all int32."""
+    side by side; -1 for an id of `n_experts` or more, which has no row) and, when given, pair_of (the pair at each row), all int32."""
     _cuda(ids, offsets, row_of, pair_of)
     for t, name in ((ids, "ids"), (offsets, "offsets"), (row_of, "row_of"), (pair_of, "pair_of")):
         _i32(t, name)
@@ -1143,19 +1199,27 @@ def moe_gather(x: torch.Tensor, row_of: torch.Tensor, xs: torch.Tensor, top: int
     return xs
 
 
-def moe_combine(ys: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor, out: torch.Tensor, top: int) -> torch.Tensor:
-    _cuda(ys, row_of, weights, out)
-    n, width = out.shape
-    if ys.shape[0] < n * top or ys.shape[1] != width or ys.dtype != out.dtype or not (ys.is_contiguous() and out.is_contiguous()):
-        raise KernelError("moe_combine: ys [at least N * top, width] of out's dtype, contiguous")
-    lib.call("ns_moe_combine", ys.data_ptr(), row_of.data_ptr(), weights.data_ptr(), out.data_ptr(), n, int(top), width,
-             dtype_code(out.dtype), _stream())
-    return out
+def moe_combine(ys: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor, out: torch.Tensor | None, top: int,
+                x: torch.Tensor | None = None, resid: torch.Tensor | None = None) -> torch.Tensor:
+    """out[n] = sum_k weights[n, k] * ys[row_of[n, k]]; a choice without a row (-1) takes x[n].  With `resid` (float32 [N, width])
+    the sum is added to it in place of `out`."""
+    _cuda(ys, row_of, weights, out, x, resid)
+    dst = resid if resid is not None else out
+    n, width = dst.shape
+    if ys.shape[0] < n * top or ys.shape[1] != width or not (ys.is_contiguous() and dst.is_contiguous()) \
+            or (resid is not None and resid.dtype != torch.float32) or (resid is None and ys.dtype != out.dtype):
+        raise KernelError("moe_combine: contiguous ys [at least N * top, width] and an output of its dtype, or a float32 stream")
+    if x is not None and (x.shape != dst.shape or x.dtype != ys.dtype or not x.is_contiguous()):
+        raise KernelError("moe_combine: x must be contiguous [N, width] of ys's dtype")
+    lib.call("ns_moe_combine", ys.data_ptr(), row_of.data_ptr(), weights.data_ptr(), _ptr(x), _ptr(out) if resid is None else None,
+             _ptr(resid), n, int(top), width, dtype_code(ys.dtype), _stream())
+    return dst
 
 
 def moe_expert_rows(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate: torch.Tensor, w_up: torch.Tensor,
                     w_down: torch.Tensor, act: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """The chosen experts of a few tokens without a host round trip: w_gate, w_up [E, ff, width], w_down [E, width, ff]."""
+    """The chosen experts of a few tokens without a host round trip: w_gate, w_up [E, ff, width], w_down [E, width, ff]; ids
+    from E on return their input."""
     _cuda(x, ids, weights, w_gate, w_up, w_down, act, out)
     n, width = x.shape
     top, ff = ids.shape[1], w_gate.shape[1]
@@ -1163,7 +1227,7 @@ def moe_expert_rows(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w
             or out.shape != (n, width) or w_down.shape[1:] != (width, ff) or len({x.dtype, w_gate.dtype, w_up.dtype, w_down.dtype, act.dtype, out.dtype}) != 1:
         raise KernelError("moe_expert_rows: contiguous operands of one dtype and the sizes the experts have")
     lib.call("ns_moe_expert_rows", x.data_ptr(), ids.data_ptr(), weights.data_ptr(), w_gate.data_ptr(), w_up.data_ptr(),
-             w_down.data_ptr(), act.data_ptr(), out.data_ptr(), n, top, width, ff, dtype_code(x.dtype), _stream())
+             w_down.data_ptr(), act.data_ptr(), out.data_ptr(), w_gate.shape[0], n, top, width, ff, dtype_code(x.dtype), _stream())
     return out
 
 

@@ -27,15 +27,18 @@ _SIGNATURES: dict[str, list] = {
     "ns_add_rmsnorm": [_P, _P, _P, _P, _P, _I, _I, _F, _I, _I, _P],
     "ns_residual_add": [_P, _P, _I, _I, _I, _P],
     "ns_swiglu": [_P, _P, _I, _I, _I, _I, _P],
+    "ns_swiglu_rows": [_P, _L, _P, _L, _I, _I, _I, _I, _P],
     "ns_gemm_f32": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "ns_rope_kv_write": [_P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "ns_attention_generic": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _I, _P],
     "ns_add_layernorm": [_P, _P, _P, _P, _P, _I, _I, _F, _I, _I, _P],
     "ns_scale_softcap": [_P, _I, _I, _L, _F, _F, _P],
-    "ns_qk_norm_rope_store": [_P, _I, _P, _P, _P, _I, _P, _F, _I, _I, _P, _P, _F, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "ns_qk_norm_rope_store": [_P, _I, _P, _P, _P, _I, _P, _F, _I, _I, _P, _P, _F, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
     "ns_delta_prepare": [_P, _I, _P, _I, _P, _P, _P, _L, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P],
     "ns_rotary_prepare": [_P, _I, _P, _P, _P, _F, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P],
-    "ns_linear_scan": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+    "ns_linear_scan": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+    "ns_ssm_prepare": [_P, _I, _P, _P, _I, _P, _P, _P, _L, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+    "ns_ssm_gate_norm": [_P, _I, _P, _I, _P, _I, _P, _P, _F, _I, _P, _I, _P, _P, _P, _P, _L, _L, _I, _I, _I, _I, _I, _I, _P],
     "ns_head_norm_gate": [_P, _I, _P, _I, _P, _F, _P, _I, _P, _I, _I, _I, _I, _P],
     "ns_sample_rows": [_P, _L, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _P],
     "ns_attention_decode": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
@@ -68,15 +71,15 @@ _SIGNATURES: dict[str, list] = {
     "ns_attention_latent_tc": [_P, _L, _L, _P, _L, _L, _P, _P, _I, _P, _P, _P, _P, _L, _P, _L, _L, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
     "ns_cast_f32": [_P, _L, _P, _I, _I, _I, _P],
     "ns_router_logits": [_P, _L, _P, _P, _I, _I, _I, _I, _P],
-    "ns_moe_route": [_P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P],
+    "ns_moe_route": [_P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P, _P],
     "ns_moe_plan": [_P, _I, _I, _P, _P, _P, _P],
     "ns_moe_grouped": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "ns_moe_pad_rows": [_P, _P, _P, _I, _I, _P],
     "ns_moe_gather": [_P, _P, _P, _I, _I, _I, _I, _P],
-    "ns_moe_combine": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
-    "ns_moe_expert_rows": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
-    "ns_activation": [_P, _P, _L, _I, _I, _P],
-    "ns_activation_rows": [_P, _L, _P, _L, _I, _I, _I, _I, _P],
+    "ns_moe_combine": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
+    "ns_moe_expert_rows": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "ns_activation": [_P, _P, _L, _I, _P, _I, _P],
+    "ns_activation_rows": [_P, _L, _P, _L, _I, _I, _I, _P, _I, _P],
     "ns_norm_add": [_P, _P, _P, _P, _P, _I, _I, _F, _I, _P],
     "ns_token_gate": [_P, _L, _P, _L, _P, _I, _I, _P, _I, _I, _I, _P],
     "ns_sigmoid_mul": [_P, _L, _P, _L, _I, _I, _I, _P],

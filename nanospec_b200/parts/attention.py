@@ -37,7 +37,9 @@ class GQAAttention(Part):
                  keys of its own chunk (at or before its position)
     softcap      c > 0: a scaled score s becomes c * tanh(s / c) before the softmax
     bias         True: q, k, v and o have biases (float32 in every mode; names "q_bias", "k_bias", "v_bias", "o_bias",
-                 default the weight's name + ".b"); the q/k/v biases are added before the q/k norm
+                 default the weight's name + ".b"); the q/k/v biases are added before the q/k norm.  "qkv": q, k and v alone
+    v_norm       {"eps": e}: every head's value is divided by its root mean square over v_dim (no gain) before it is cached; e is
+                 the q/k norm's when both are set
     own_kv       False: the mixer has no k and v projections (nor their norm and biases): it reads the lane that another
                  layer's mixer of the same head counts, sizes and rotation writes (the recipe gives it a run with
                  `writes=False` on that lane), with queries, mask and output projection of its own
@@ -74,6 +76,12 @@ class GQAAttention(Part):
         self.chunk = int(p.get("chunk") or 0)
         self.softcap = float(p.get("softcap") or 0.0)
         self.has_bias = bool(p.get("bias"))
+        if p.get("bias") not in (None, False, True, "qkv"):
+            raise ValueError(f"gqa_attention: bias {p['bias']!r} (True, 'qkv' or none)")
+        self.has_o_bias = self.has_bias and p["bias"] != "qkv"
+        self.v_norm = dict(p["v_norm"]) if p.get("v_norm") else None
+        if self.v_norm and self.qk_norm and float(self.v_norm["eps"]) != float(self.qk_norm["eps"]):
+            raise ValueError("gqa_attention: v_norm and qk_norm share one eps")
         self.own_kv = bool(p.get("own_kv", True))
         self.sink_kind = p.get("sink")
         if self.sink_kind not in (None, "zero", "learned"):
@@ -84,8 +92,8 @@ class GQAAttention(Part):
         self.v_from_k = bool(p.get("v_from_k"))
         self.taps = int(p.get("conv") or 0)
         self.per_head = bool(self.head_norm or self.q_temp or self.head_gate or self.v_from_k or self.taps)
-        if self.per_head and (self.qk_norm is not None or self.has_bias or not self.own_kv):
-            raise ValueError("gqa_attention: head_norm, q_temp, head_gate, v_from_k and conv do not go with qk_norm, bias or borrowed keys")
+        if self.per_head and (self.qk_norm is not None or self.has_bias or not self.own_kv or self.v_norm is not None):
+            raise ValueError("gqa_attention: head_norm, q_temp, head_gate, v_from_k and conv do not go with qk_norm, v_norm, bias or borrowed keys")
         if self.head_norm and self.head_norm.get("when", "before") not in ("before", "after"):
             raise ValueError(f"gqa_attention: head_norm.when {self.head_norm.get('when')!r} ('before' or 'after' the rotation)")
         if self.v_from_k and self.v_dim != self.head_dim:
@@ -105,7 +113,8 @@ class GQAAttention(Part):
         self.v_size = self.kv_heads * self.v_dim
         self.o_in = self.heads * self.v_dim
         # what the llama-shaped fast paths (a projection with the rotation in its epilogue) do not know of
-        self.general = self.v_dim != self.head_dim or self.qk_norm is not None or self.has_bias or not self.own_kv
+        self.general = self.v_dim != self.head_dim or self.qk_norm is not None or self.has_bias or not self.own_kv \
+            or self.v_norm is not None
         # the packed projection's columns on the per-head path: [q | k | v (unless the keys double as values) | g (the heads' gates)]
         self.channels = self.q_size + self.kv_size + (0 if self.v_from_k else self.v_size)
         self.sink: torch.Tensor | None = None
@@ -144,7 +153,7 @@ class GQAAttention(Part):
                 specs[n["k_norm"]] = WeightSpec((self.kv_size,), rule="float32", init="gain")
         if self.has_bias:
             sizes = {"q": self.q_size, "k": self.kv_size, "v": self.v_size, "o": self.hidden}
-            for k in ("q", "k", "v", "o") if self.own_kv else ("q", "o"):
+            for k in (("q", "k", "v") if self.own_kv else ("q",)) + (("o",) if self.has_o_bias else ()):
                 specs[n[k + "_bias"]] = WeightSpec((sizes[k],), rule="float32", init="normal")
         return specs
 
@@ -153,7 +162,7 @@ class GQAAttention(Part):
         kinds = (("q", "k") if self.v_from_k else ("q", "k", "v")) if self.own_kv else ("q",)
         # one packed projection [q | k | v]: one matrix product instead of three
         self.w_qkv = torch.cat([tensors[n[k]] for k in kinds + (("g",) if self.head_gate else ())], dim=0).contiguous()
-        if self.per_head and self.w_qkv.shape[0] % 8:  # rows of the product start on 16 bytes in bfloat16
+        if (self.per_head or self.general) and self.w_qkv.shape[0] % 8:  # rows of the product start on 16 bytes in bfloat16
             pad = torch.zeros((-self.w_qkv.shape[0] % 8, self.hidden), dtype=self.w_qkv.dtype, device=self.w_qkv.device)
             self.w_qkv = torch.cat([self.w_qkv, pad], dim=0).contiguous()
         self.w_o = tensors[n["o"]].contiguous()
@@ -171,7 +180,7 @@ class GQAAttention(Part):
             self.k_gain = tensors[n["k_norm"]].contiguous() if self.own_kv else None
         if self.has_bias:
             self.qkv_bias = torch.cat([tensors[n[k + "_bias"]] for k in kinds], dim=0).contiguous()
-            self.o_bias = tensors[n["o_bias"]].contiguous()
+            self.o_bias = tensors[n["o_bias"]].contiguous() if self.has_o_bias else None
 
     def cache_need(self) -> CacheNeed | None:
         # (a chunked mask keeps every page: a layer that reads this lane may be masked otherwise)
@@ -202,19 +211,8 @@ class GQAAttention(Part):
         qkv = ctx.buffer("qkv", self.w_qkv.shape[0])
         if self.general:
             ops.linear(x, self.w_qkv, qkv)
-            if self.position is None:
-                raise ValueError("an attention mixer with qk_norm, v_dim, biases or borrowed keys takes a position part with the "
-                                 "general rotate_and_store")
-            if not self.own_kv and writes:
-                raise ValueError("an attention mixer without k and v projections reads a lane that another run writes")
-            qn = self.qk_norm
-            extra = {"bias": self.qkv_bias} if self.qkv_bias is not None else {}
-            self.position.rotate_and_store(qkv, ctx, lane, self.heads, self.kv_heads if self.own_kv else 0, self.head_dim, writes,
-                                           v_dim=self.v_dim, q_gain=self.q_gain, k_gain=self.k_gain,
-                                           eps=float(qn["eps"]) if qn else 0.0, **extra)
             attn = ctx.buffer("attn_out", self.o_in)
-            ops.attention(qkv, lane, ctx, attn, self.heads, self.kv_heads, self.head_dim, self.scale, self.window,
-                          self.keep_first, self.v_dim, self.wide_weights, self.chunk, self.softcap, sink=self.sink)
+            self._attend_general(qkv, ctx, lane, writes, attn)
             if self.o_bias is not None and leave_bias:
                 return ops.linear(attn, self.w_o, ctx.buffer("branch", self.hidden))
             if self.o_bias is not None:
@@ -232,6 +230,24 @@ class GQAAttention(Part):
                       wide_weights=self.wide_weights, chunk=self.chunk, softcap=self.softcap, sink=self.sink)
         return ops.linear(attn, self.w_o, ctx.buffer("branch", self.hidden), sink=sink)
 
+    def _attend_general(self, qkv: torch.Tensor, ctx: StepContext, lane: LaneView, writes: bool, attn: torch.Tensor) -> None:
+        """Everything between the two products for the general q/k/v preparation: biases, the whole-projection norms, the
+        rotation, the values' norm and the cache write in one kernel (in place), then the attention."""
+        if self.position is None:
+            raise ValueError("an attention mixer with qk_norm, v_norm, v_dim, biases or borrowed keys takes a position part with the "
+                             "general rotate_and_store")
+        if not self.own_kv and writes:
+            raise ValueError("an attention mixer without k and v projections reads a lane that another run writes")
+        qn = self.qk_norm or self.v_norm
+        extra = {"bias": self.qkv_bias} if self.qkv_bias is not None else {}
+        if self.v_norm is not None:
+            extra["v_norm"] = True
+        self.position.rotate_and_store(qkv, ctx, lane, self.heads, self.kv_heads if self.own_kv else 0, self.head_dim, writes,
+                                       v_dim=self.v_dim, q_gain=self.q_gain, k_gain=self.k_gain,
+                                       eps=float(qn["eps"]) if qn else 0.0, **extra)
+        ops.attention(qkv, lane, ctx, attn, self.heads, self.kv_heads, self.head_dim, self.scale, self.window,
+                      self.keep_first, self.v_dim, self.wide_weights, self.chunk, self.softcap, sink=self.sink)
+
     def _forward_per_head(self, x, ctx: StepContext, lane: LaneView, writes: bool):
         """Projection, the per-head steps and the attention (`forward_projected`), output projection."""
         proj = ops.linear(x, self.w_qkv, ctx.buffer("qkv_in" if self.taps > 1 else "qkv", self.w_qkv.shape[0]))
@@ -245,7 +261,7 @@ class GQAAttention(Part):
     # arrangement hands it: `forward_projected`)
     @property
     def packs_projections(self) -> bool:
-        return self.per_head
+        return self.per_head or (self.general and self.own_kv and not self.has_o_bias)
 
     @property
     def input_weight(self) -> torch.Tensor:
@@ -262,8 +278,10 @@ class GQAAttention(Part):
 
     def forward_projected(self, proj: torch.Tensor, ctx: StepContext, lane: LaneView, writes: bool, attn: torch.Tensor) -> None:
         """`proj` [N, >= columns of the packed projection] (rows may lie in a wider buffer): `ops.head_prepare_store` (convolution,
-        head norms, rotation, query temperature, cache write), then attention with the sink and the heads' gates in its epilogue into
-        `attn` [N, heads * v_dim] (likewise)."""
+        head norms, rotation, query temperature, cache write) or the general preparation, then attention with the sink and the heads'
+        gates in its epilogue into `attn` [N, heads * v_dim] (likewise)."""
+        if not self.per_head:
+            return self._attend_general(proj, ctx, lane, writes, attn)
         if self.taps > 1 and not writes:
             raise ValueError("an attention mixer with a convolution owns its state: its lane cannot be shared")
         # a convolution reads its neighbours' rows: not in place

@@ -35,7 +35,10 @@ input projection [mixer's columns | feed-forward's] of h, and one output project
 activations] by [W_o | W_down], whose float32 accumulator holds mixer(h) + feed_forward(h) before it is rounded once; the sublayers
 keep views of the packed matrices in place of their own (`adopt`), so weights are held once and replaced in place.  In a step of up
 to 64 tokens the packed output product also adds its result to the stream and applies the NEXT block's norm in its epilogue, when
-that norm is elementwise (`elementwise_sink`): a decode layer is then five kernels and the tail of a convolution.
+that norm is elementwise (`elementwise_sink`): a decode layer is then five kernels and the tail of a convolution.  An RMS norm is folded
+there as in "prenorm" when nothing but the packed input product reads it (`input_norm_sink`).
+A feed-forward that is only partly a pair of products (routed experts beside a shared one) offers `join_stream(h, ctx, resid)`, which
+adds that part to the float32 stream itself, and `forward_rest(h, ctx)` (or its projections) for what is left, None if nothing is.
 """
 
 from __future__ import annotations
@@ -190,6 +193,7 @@ class ParallelBlock:
         self.w_in: torch.Tensor | None = None   # [mixer's columns + feed-forward's, hidden] once packed
         self.w_out: torch.Tensor | None = None  # [hidden, heads' outputs + activations]
         self._packed: bool | None = None        # decided when the weights are bound
+        self._ranges: list[tuple[slice, slice]] = []  # of the mixer and of the feed-forward in the packed products
 
     def parts(self) -> dict:
         return {s: getattr(self, s) for s in self.slots if getattr(self, s) is not None}
@@ -206,24 +210,58 @@ class ParallelBlock:
             return pending[1]
         return pending
 
+    def _joins(self) -> bool:
+        return callable(getattr(self.feed_forward, "join_stream", None))
+
     def _pack(self) -> bool:
         """Packs the sublayers' projections once.  Widths in multiples of eight only: rows of the packed buffers then start on 16 bytes
-        in bfloat16, which the sublayers' kernels ask of their operands."""
+        in bfloat16, which the sublayers' kernels ask of their operands.  The input product gets rows of zeros up to a multiple of
+        128 when a norm may be folded into it (the fold's tile)."""
         m, f = self.mixer, self.feed_forward
-        if not (self.PACK and f is not None and getattr(m, "packs_projections", False) and getattr(f, "packs_projections", False)):
+        if not (self.PACK and getattr(m, "packs_projections", False)):
             return False
-        wi_m, wi_f, wo_m, wo_f = m.input_weight, f.input_weight, m.output_weight, f.output_weight
-        if any(w is None for w in (wi_m, wi_f, wo_m, wo_f)) or any(w.shape[0] % 8 or w.shape[1] % 8 for w in (wi_m, wi_f, wo_m, wo_f)):
+        parts = [m]
+        if f is not None:
+            if not getattr(f, "packs_projections", False):
+                return False
+            if f.input_weight is not None:  # (routed experts without a shared one have nothing to pack)
+                parts.append(f)
+        w_in, w_out = [p.input_weight for p in parts], [p.output_weight for p in parts]
+        if any(w is None for w in w_in + w_out) or any(w.shape[0] % 8 or w.shape[1] % 8 for w in w_in + w_out):
             return False
-        self.w_in = torch.cat([wi_m, wi_f], dim=0).contiguous()
-        self.w_out = torch.cat([wo_m, wo_f], dim=1).contiguous()
-        m.adopt(self.w_in[: wi_m.shape[0]], self.w_out[:, : wo_m.shape[1]])
-        f.adopt(self.w_in[wi_m.shape[0]:], self.w_out[:, wo_m.shape[1]:])
+        rows = sum(w.shape[0] for w in w_in)
+        if _folds(self.norm_mixer) and not self._joins() and rows % 128:
+            pad = torch.zeros((-rows % 128, w_in[0].shape[1]), dtype=w_in[0].dtype, device=w_in[0].device)
+        else:
+            pad = w_in[0][:0]
+        self.w_in = torch.cat(w_in + [pad], dim=0).contiguous()
+        self.w_out = torch.cat(w_out, dim=1).contiguous()
+        at_in = at_out = 0
+        self._ranges = []
+        for p, wi, wo in zip(parts, w_in, w_out):
+            ri, ro = slice(at_in, at_in + wi.shape[0]), slice(at_out, at_out + wo.shape[1])
+            p.adopt(self.w_in[ri], self.w_out[:, ro])
+            self._ranges.append((ri, ro))
+            at_in, at_out = ri.stop, ro.stop
         return True
 
     def after_bind(self) -> None:
         """Called by the model once every part has its weights."""
         self._packed = self._pack()
+
+    def input_norm_sink(self, resid: torch.Tensor, ctx: StepContext):
+        """What the product before this block needs to fold the block's norm in: an RMS norm that only the packed input product reads
+        (`ops.NormSink`); None otherwise."""
+        if self._packed and not self._joins() and _folds(self.norm_mixer) and ops.norm_fusion_ok(ctx.n_tokens, self.w_in.dtype, self.w_in):
+            return self.norm_mixer.sink(resid, ctx)
+        return None
+
+    def _next_sink(self, follow, resid: torch.Tensor, ctx: StepContext):
+        """The next block's norm, when this block's last product may take it over."""
+        nxt = getattr(follow, "norm_mixer", None) if isinstance(follow, ParallelBlock) else None
+        if nxt is not None and callable(getattr(nxt, "elementwise_sink", None)):
+            return nxt.elementwise_sink(resid, ctx)
+        return follow.input_norm_sink(resid, ctx) if hasattr(follow, "input_norm_sink") else None
 
     def forward(self, resid: torch.Tensor, pending, ctx: StepContext, lane: LaneView, writes: bool = True, follow=None):
         if self._packed is None:  # parts bound by hand: pack now, unless a graph is being captured (no allocation then)
@@ -231,21 +269,25 @@ class ParallelBlock:
         if isinstance(pending, tuple) and not self.takes_pair():
             pending = self._settle(resid, pending)
         h = self.norm_mixer.add_norm(resid, pending, ctx)
+        joins = self._joins()
+        if joins:
+            self.feed_forward.join_stream(h, ctx, resid)
         if self._packed:
-            cm, om = self.mixer.input_weight.shape[0], self.mixer.output_weight.shape[1]
             proj = ops.linear(h, self.w_in, ctx.buffer("par_in", self.w_in.shape[0]))
             mid = ctx.buffer("par_mid", self.w_out.shape[1])
-            self.mixer.forward_projected(proj[:, :cm], ctx, lane, writes, mid[:, :om])
-            self.feed_forward.forward_projected(proj[:, cm:], ctx, mid[:, om:])
+            (ri, ro), rest = self._ranges[0], self._ranges[1:]
+            self.mixer.forward_projected(proj[:, ri], ctx, lane, writes, mid[:, ro])
+            for ri, ro in rest:
+                self.feed_forward.forward_projected(proj[:, ri], ctx, mid[:, ro])
             # a step of a few tokens: the sum into the stream and the next block's norm in this product's epilogue
-            sink = None
-            nxt = getattr(follow, "norm_mixer", None) if isinstance(follow, ParallelBlock) else None
-            if nxt is not None and callable(getattr(nxt, "elementwise_sink", None)) and ops.norm_fusion_ok(ctx.n_tokens, self.w_out.dtype, self.w_out):
-                sink = nxt.elementwise_sink(resid, ctx)
+            sink = self._next_sink(follow, resid, ctx) if ops.norm_fusion_ok(ctx.n_tokens, self.w_out.dtype, self.w_out) else None
             return resid, ops.linear(mid, self.w_out, ctx.buffer("branch", resid.shape[1]), sink=sink)
         a = self.mixer.forward(h, ctx, lane, writes)
-        if self.feed_forward is None:
+        if self.feed_forward is None or (joins and self.feed_forward.input_weight is None):
             return resid, a
+        if joins:
+            ops.residual_add(resid, a)
+            return resid, self.feed_forward.forward_rest(h, ctx)
         # the pair stays pending only for a norm that is known to take it: the next block's, when that is of this kind
         pair = getattr(self.feed_forward, "names_output", False) and isinstance(follow, ParallelBlock) and follow.takes_pair()
         if pair:

@@ -7,6 +7,12 @@ up with weights from a router.
     the `top` eligible experts of largest s are chosen; weight_k = s_k / (sum of the chosen s + 1e-20) * scale
     y = sum_k weight_k * down_k(silu(gate_k h) * (up_k h))
 
+and, all optional:
+    correction   a float32 number per expert that is added to the scores that choose (groups and experts), not to the weights
+    renormalize  False: weight_k = s_k * scale
+    identity     the last so many outputs of the router stand for experts without tensors whose output is h itself
+    shared       {"intermediate": f}: one more gated feed-forward that every token runs, added with weight 1
+
 Four routes, the same numbers up to rounding.  A bfloat16 step (of up to `GROUPED_MAX` tokens when that is set, and every step that a CUDA
 graph captures) lays the (token, choice) pairs out by expert on the device (`ops.moe_plan`) and runs every expert over its
 rows in one tensor-core kernel that reads the counts on the device (`ops.moe_grouped`): each chosen expert's weights are
@@ -16,8 +22,13 @@ on the host; in bfloat16 every expert then owns the same number of rows (`ops.mo
 library product for gate/up and one for down; in float32 each expert that has tokens runs as the framework's gated product and down
 product over its run of rows.  `ops.moe_combine` adds the results per token in the order of the choice (float32 sums, one rounding).
 
-params: hidden, experts, top, intermediate (an expert's width), groups, keep, scale, score, names (optional: "router";
-the experts' tensors are e<k>.gate, e<k>.up, e<k>.down).
+params: hidden, experts (those with tensors), top, intermediate (an expert's width), groups, keep, scale, score, correction (bool),
+renormalize (default True), identity (default 0), shared, names (optional: "router", "correction"; the experts' tensors are e<k>.gate,
+e<k>.up, e<k>.down, the shared one's shared.gate, shared.up, shared.down).
+
+An arrangement that runs its sublayers side by side may take the part in two: `join_stream(h, ctx, resid)` adds the routed experts'
+sum to the float32 stream (no rounding in between), and the rest - the shared expert - offers its projections like any
+feed-forward (`packs_projections`; `input_weight` None when there is no shared expert), or runs alone (`forward_rest`).
 """
 
 from __future__ import annotations
@@ -25,9 +36,10 @@ from __future__ import annotations
 import torch
 
 from .. import ops
+from ..config.recipe import PartSpec
 from .base import Part, WeightSpec
 from .context import StepContext
-from .registry import register_part
+from .registry import build_part, register_part
 
 ROWS_MAX = 16      # steps of up to this many tokens stream the chosen experts' rows (float32, or widths that are no multiple of 8)
 # bfloat16 steps of up to this many tokens run every expert over its tokens in one tensor-core kernel that reads the counts on the
@@ -50,15 +62,29 @@ class RoutedExperts(Part):
         self.softmax = p.get("score", "sigmoid") == "softmax"
         if p.get("score", "sigmoid") not in ("sigmoid", "softmax"):
             raise ValueError(f"routed_experts: unknown score {p.get('score')!r}")
-        if self.top > self.experts or (self.groups > 1 and (self.experts % self.groups or not 1 <= self.keep <= self.groups
-                                                             or self.keep * (self.experts // self.groups) < self.top)):
-            raise ValueError(f"routed_experts: {self.top} of {self.experts} experts in {self.groups} groups of which {self.keep} stay")
-        self.n_router = dict(p.get("names") or {}).get("router", "router")
+        self.identity = int(p.get("identity") or 0)
+        self.choices = self.experts + self.identity  # the router's outputs
+        self.renormalize = bool(p.get("renormalize", True))
+        if self.top > self.choices or (self.groups > 1 and (self.choices % self.groups or not 1 <= self.keep <= self.groups
+                                                             or self.keep * (self.choices // self.groups) < self.top)):
+            raise ValueError(f"routed_experts: {self.top} of {self.choices} experts in {self.groups} groups of which {self.keep} stay")
+        names = dict(p.get("names") or {})
+        self.n_router, self.n_correction = names.get("router", "router"), names.get("correction", "correction")
+        self.has_correction = bool(p.get("correction"))
+        self.correction: torch.Tensor | None = None
+        shared = p.get("shared")
+        self.shared = None if shared is None else build_part("feed_forward", PartSpec("swiglu", {
+            "hidden": self.hidden, "intermediate": int(shared["intermediate"]),
+            "names": {k: f"shared.{k}" for k in ("gate", "up", "down")}}), dtype, device)
         self.w_router = self.w_gate = self.w_up = self.w_down = self.w_gate_up = None
         self.gate_block = 0
 
     def weight_specs(self) -> dict[str, WeightSpec]:
-        specs = {self.n_router: WeightSpec((self.experts, self.hidden), rule="float32", init="normal", std=0.1)}
+        specs = {self.n_router: WeightSpec((self.choices, self.hidden), rule="float32", init="normal", std=0.1)}
+        if self.has_correction:
+            specs[self.n_correction] = WeightSpec((self.choices,), rule="float32", init="normal", std=0.01)
+        if self.shared is not None:
+            specs.update(self.shared.weight_specs())
         for e in range(self.experts):
             specs[f"e{e}.gate"] = WeightSpec((self.inter, self.hidden))
             specs[f"e{e}.up"] = WeightSpec((self.inter, self.hidden))
@@ -68,6 +94,10 @@ class RoutedExperts(Part):
     def bind(self, tensors) -> None:
         E = self.experts
         self.w_router = tensors[self.n_router].contiguous()
+        if self.has_correction:
+            self.correction = tensors[self.n_correction].contiguous()
+        if self.shared is not None:
+            self.shared.bind({n: tensors[n] for n in self.shared.weight_specs()})
         self.w_gate = torch.stack([tensors[f"e{e}.gate"] for e in range(E)]).contiguous()   # [E, ff, width]
         self.w_up = torch.stack([tensors[f"e{e}.up"] for e in range(E)]).contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(E)]).contiguous()   # [E, width, ff]
@@ -83,43 +113,79 @@ class RoutedExperts(Part):
     def route(self, x, ctx: StepContext) -> tuple[torch.Tensor, torch.Tensor]:
         """(chosen experts int32 [N, top], their weights float32 [N, top])"""
         n = x.shape[0]
-        logits = ops.router_logits(x, self.w_router, ctx.buffer("router_logits", self.experts, torch.float32),
+        logits = ops.router_logits(x, self.w_router, ctx.buffer("router_logits", self.choices, torch.float32),
                                    scratch=lambda rows, cols: ctx.buffer("router_in", cols, torch.float32, rows=rows))
         ids = ctx.buffer("expert_ids", self.top, torch.int32)
         weights = ctx.buffer("expert_weights", self.top, torch.float32)
-        ops.moe_route(logits, self.groups, self.keep, self.top, self.scale, ids, weights, self.softmax)
+        ops.moe_route(logits, self.groups, self.keep, self.top, self.scale, ids, weights, self.softmax, self.correction, self.renormalize)
         return ids, weights
 
-    def _grouped(self, x, ids, weights, offsets, row_of, out, ctx: StepContext):
+    # ---- the three ways to run the part ------------------------------------------------------------------------------------
+    def forward(self, x, ctx: StepContext):
+        out = ctx.buffer("branch", self.hidden)
+        if self.shared is None:
+            return self._routed(x, ctx, out, None)
+        y = ops.cast_f32(self.shared.forward(x, ctx, out_name="branch_shared"), ctx.buffer("experts_sum", self.hidden, torch.float32))
+        self._routed(x, ctx, out, y)
+        return out.copy_(y)
+
+    def join_stream(self, x, ctx: StepContext, resid: torch.Tensor) -> None:
+        """The routed experts' sum, added to the float32 stream; everything but the shared expert."""
+        self._routed(x, ctx, ctx.buffer("experts_branch", self.hidden), resid)
+
+    def forward_rest(self, x, ctx: StepContext):
+        """What `join_stream` leaves: the shared expert's output, or None without one."""
+        return None if self.shared is None else self.shared.forward(x, ctx)
+
+    # ---- optional: the shared expert's products inside larger ones of an arrangement (see `GQAAttention.packs_projections`) ------
+    packs_projections = True
+
+    @property
+    def input_weight(self) -> torch.Tensor | None:
+        return None if self.shared is None else self.shared.input_weight
+
+    @property
+    def output_weight(self) -> torch.Tensor | None:
+        return None if self.shared is None else self.shared.output_weight
+
+    def adopt(self, w_in: torch.Tensor, w_out: torch.Tensor) -> None:
+        self.shared.adopt(w_in, w_out)
+
+    def forward_projected(self, u: torch.Tensor, ctx: StepContext, act: torch.Tensor) -> None:
+        self.shared.forward_projected(u, ctx, act)
+
+    # ---- the routed experts ---------------------------------------------------------------------------------------------------
+    def _grouped(self, x, ids, weights, offsets, row_of, out, ctx: StepContext, resid):
         n = x.shape[0]
         pair_of = ctx.buffer("expert_pairs", self.top, torch.int32)
         ops.moe_plan(ids, self.experts, offsets, row_of, pair_of)
         act = ctx.buffer("expert_act", self.inter, rows=n * self.top)
         ys = ctx.buffer("expert_out", self.hidden, rows=n * self.top)
         ops.moe_grouped(x, pair_of, offsets, self.w_gate, self.w_up, self.w_down, act, ys, self.top)
-        return ops.moe_combine(ys, row_of, weights, out, self.top)
+        return ops.moe_combine(ys, row_of, weights, out, self.top, x=x, resid=resid)
 
-    def forward(self, x, ctx: StepContext):
+    def _routed(self, x, ctx: StepContext, out: torch.Tensor, resid: torch.Tensor | None):
+        """The routed experts' sum in `out`, or added to the float32 `resid` when that is given; returns where it went."""
         n = x.shape[0]
         ids, weights = self.route(x, ctx)
-        out = ctx.buffer("branch", self.hidden)
         captured = bool(ctx.extras.get("graph")) or torch.cuda.is_current_stream_capturing()
         offsets = ctx.buffer("expert_offsets", 1, torch.int32, rows=self.experts + 1).view(-1)
         row_of = ctx.buffer("expert_rows", self.top, torch.int32)
         grouped_ok = ops.moe_grouped_ok(x, self.hidden, self.inter)
         if grouped_ok and (GROUPED_MAX is None or n <= GROUPED_MAX or captured):
-            return self._grouped(x, ids, weights, offsets, row_of, out, ctx)
+            return self._grouped(x, ids, weights, offsets, row_of, out, ctx, resid)
         if n <= ROWS_MAX or captured:
             act = ctx.buffer("expert_act", self.inter, rows=n * self.top)
-            return ops.moe_expert_rows(x, ids, weights, self.w_gate, self.w_up, self.w_down, act, out)
+            ops.moe_expert_rows(x, ids, weights, self.w_gate, self.w_up, self.w_down, act, out)
+            return out if resid is None else ops.residual_add(resid, out)
         ops.moe_plan(ids, self.experts, offsets, row_of)
         bounds = offsets.tolist()  # the one host round trip of the step's experts
         if grouped_ok:
             # bfloat16: every expert owns `cap` rows and all run as one batched product each for gate/up and down
-            cap = -(-max(b - a for a, b in zip(bounds, bounds[1:])) // 64) * 64
+            cap = max(64, -(-max(b - a for a, b in zip(bounds, bounds[1:])) // 64) * 64)
             rows = self.experts * cap
             if rows > PAD_WASTE_MAX * n * self.top:  # the tokens crowd a few experts: no layout of equal shares for them
-                return self._grouped(x, ids, weights, offsets, row_of, out, ctx)
+                return self._grouped(x, ids, weights, offsets, row_of, out, ctx, resid)
             ops.moe_pad_rows(ids, offsets, row_of, cap)
             xs = ops.moe_gather(x, row_of, ctx.buffer("expert_in", self.hidden, rows=rows), self.top)
             gu = ctx.buffer("expert_gate_up", 2 * self.inter, rows=rows)
@@ -127,7 +193,7 @@ class RoutedExperts(Part):
             act = ops.swiglu(gu, ctx.buffer("expert_act", self.inter, rows=rows), self.gate_block)
             ys = ctx.buffer("expert_out", self.hidden, rows=rows)
             torch.bmm(act.view(self.experts, cap, self.inter), self.w_down.transpose(1, 2), out=ys.view(self.experts, cap, self.hidden))
-            return ops.moe_combine(ys, row_of, weights, out, self.top)
+            return ops.moe_combine(ys, row_of, weights, out, self.top, x=x, resid=resid)
         xs = ops.moe_gather(x, row_of, ctx.buffer("expert_in", self.hidden, rows=n * self.top), self.top)
         ys = ctx.buffer("expert_out", self.hidden, rows=n * self.top)
         act = ctx.buffer("expert_act", self.inter, rows=n * self.top)
@@ -137,4 +203,4 @@ class RoutedExperts(Part):
             if hi > lo:
                 ops.gated_linear(xs[lo:hi], self.w_gate_up[e], act[lo:hi], scratch[lo:hi], self.gate_block)
                 ops.linear(act[lo:hi], self.w_down[e], ys[lo:hi])
-        return ops.moe_combine(ys, row_of, weights, out, self.top)
+        return ops.moe_combine(ys, row_of, weights, out, self.top, x=x, resid=resid)

@@ -21,7 +21,9 @@ from .registry import register_part
 @register_part("feed_forward", "swiglu")
 class SwiGLU(Part):
     """params: hidden, intermediate, names (optional: the tensors' names after the part's prefix, keys "gate", "up",
-    "down"; default the Hugging Face ones)."""
+    "down"; default the Hugging Face ones).  `forward` takes `out_name`, the step buffer that receives the result."""
+
+    names_output = True
 
     def __init__(self, spec, dtype, device) -> None:
         super().__init__(spec, dtype, device)
@@ -59,17 +61,39 @@ class SwiGLU(Part):
     def feeds_norm_sink(self, n_tokens: int) -> bool:
         return ops.norm_fusion_ok(n_tokens, self.dtype, self.w_down)
 
-    def forward(self, x, ctx: StepContext, sink: ops.NormSink | None = None):
+    def forward(self, x, ctx: StepContext, sink: ops.NormSink | None = None, out_name: str = "branch"):
         act = ops.gated_linear(x, self.w_gate_up, ctx.buffer("ffn_act", self.inter), ctx.buffer("gate_up", 2 * self.inter),
                                self.gate_block)
-        return ops.linear(act, self.w_down, ctx.buffer("branch", self.hidden), sink=sink)
+        return ops.linear(act, self.w_down, ctx.buffer(out_name, self.hidden), sink=sink)
+
+    # ---- optional: an arrangement that runs the two products inside larger ones of its own (see `GQAAttention.packs_projections`)
+    packs_projections = True
+
+    @property
+    def input_weight(self) -> torch.Tensor:
+        return self.w_gate_up
+
+    @property
+    def output_weight(self) -> torch.Tensor:
+        return self.w_down
+
+    def adopt(self, w_in: torch.Tensor, w_out: torch.Tensor) -> None:
+        if w_in.shape != self.w_gate_up.shape or w_out.shape != self.w_down.shape:
+            raise ValueError("adopt: views of the projections' own shapes are needed")
+        self.w_gate_up, self.w_down = w_in, w_out
+
+    def forward_projected(self, u: torch.Tensor, ctx: StepContext, act: torch.Tensor) -> None:
+        """`u` [N, 2 * intermediate] (rows may lie in a wider buffer): the gated activation into `act` (likewise)."""
+        ops.swiglu(u, act, self.gate_block)
 
 
 @register_part("feed_forward", "dense_act")
 class DenseAct(Part):
     """down(act(up(x))), no gate, no biases.  params: hidden, intermediate, activation ("gelu_erf": the exact gelu,
-    "gelu_tanh", "silu", "relu2": the square of relu), names (optional: keys "up", "down"; default "up", "down").  The activation is float32 on the
-    rounded product and is rounded once.  `forward` takes `out_name`, the step buffer that receives the result (an arrangement that
+    "gelu_tanh", "silu", "relu2": the square of relu, "xielu"), names (optional: keys "up", "down", "act"; default those words).  xielu has
+    two learned numbers p, q (tensor "act"): softplus(p) x^2 + x / 2 for x > 0 and (1/2 + softplus(q)) (exp(x) - 1 - x) + x / 2
+    otherwise; the two factors are taken once, when the weights are bound.  The activation is float32 on the rounded product and is
+    rounded once.  `forward` takes `out_name`, the step buffer that receives the result (an arrangement that
     holds two branches at once gives another name than the mixers' "branch")."""
 
     names_output = True
@@ -81,19 +105,28 @@ class DenseAct(Part):
         if self.activation not in ops.ACTIVATIONS:
             raise ValueError(f"dense_act: unknown activation {self.activation!r} (known: {', '.join(ops.ACTIVATIONS)})")
         names = dict(spec.params.get("names") or {})
-        self.n_up, self.n_down = names.get("up", "up"), names.get("down", "down")
+        self.n_up, self.n_down, self.n_act = names.get("up", "up"), names.get("down", "down"), names.get("act", "act")
+        self.coef: torch.Tensor | None = None  # xielu's two factors
         self.w_up: torch.Tensor | None = None
         self.w_down: torch.Tensor | None = None
 
     def weight_specs(self) -> dict[str, WeightSpec]:
-        return {self.n_up: WeightSpec((self.inter, self.hidden)), self.n_down: WeightSpec((self.hidden, self.inter))}
+        specs = {self.n_up: WeightSpec((self.inter, self.hidden)), self.n_down: WeightSpec((self.hidden, self.inter))}
+        if self.activation == "xielu":
+            specs[self.n_act] = WeightSpec((2,), rule="float32", init="normal", std=0.5)
+        return specs
 
     def bind(self, tensors) -> None:
         self.w_up, self.w_down = tensors[self.n_up].contiguous(), tensors[self.n_down].contiguous()
+        if self.activation == "xielu":
+            pq = tensors[self.n_act].double()
+            factors = pq.clamp(min=0.0) + torch.log1p(torch.exp(-pq.abs()))  # softplus
+            factors[1] += 0.5
+            self.coef = factors.float().contiguous()
 
     def forward(self, x, ctx: StepContext, out_name: str = "branch"):
         u = ops.linear(x, self.w_up, ctx.buffer("ffn_up", self.inter))
-        a = ops.activation(u, ctx.buffer("ffn_act", self.inter), self.activation)
+        a = ops.activation(u, ctx.buffer("ffn_act", self.inter), self.activation, self.coef)
         return ops.linear(a, self.w_down, ctx.buffer(out_name, self.hidden))
 
     # ---- optional: an arrangement that runs the two products inside larger ones of its own (see `GQAAttention.packs_projections`)
@@ -114,4 +147,4 @@ class DenseAct(Part):
 
     def forward_projected(self, u: torch.Tensor, ctx: StepContext, act: torch.Tensor) -> None:
         """`u` [N, intermediate] (rows may lie in a wider buffer): the activation into `act` (likewise)."""
-        ops.activation(u, act, self.activation)
+        ops.activation(u, act, self.activation, self.coef)

@@ -28,7 +28,8 @@ from .registry import register_part
 
 @register_part("norm", "rmsnorm")
 class RMSNorm(Part):
-    """params: hidden, eps, weight_name (the gain's name after the norm's prefix; default "weight")."""
+    """params: hidden, eps, weight_name (the gain's name after the norm's prefix; default "weight"), scalar (True: the gain is one
+    number for all features, a tensor of shape (); it is laid out once per feature, so every kernel and every fold takes it)."""
 
     centered = False
     bias: torch.Tensor | None = None
@@ -38,13 +39,15 @@ class RMSNorm(Part):
         self.hidden = int(spec["hidden"])
         self.eps = float(spec["eps"])
         self.weight_name = spec.params.get("weight_name", "weight")
+        self.scalar = bool(spec.params.get("scalar"))
         self.gain: torch.Tensor | None = None
 
     def weight_specs(self) -> dict[str, WeightSpec]:
-        return {self.weight_name: WeightSpec((self.hidden,), rule="float32", init="gain")}
+        return {self.weight_name: WeightSpec(() if self.scalar else (self.hidden,), rule="float32", init="gain")}
 
     def bind(self, tensors) -> None:
-        self.gain = tensors[self.weight_name].contiguous()
+        gain = tensors[self.weight_name]
+        self.gain = (gain.reshape(1).expand(self.hidden) if self.scalar else gain).contiguous()
 
     def sink(self, resid: torch.Tensor, ctx: StepContext) -> ops.NormSink:
         return ops.NormSink(resid, self.gain, self.eps, ctx.workspace)

@@ -137,8 +137,11 @@ class Rotary(Part):
         return self._inv_freq
 
     def rotate_and_store(self, qkv: torch.Tensor, ctx: StepContext, lane: LaneView, nq: int, nkv: int, head_dim: int,
-                         writes: bool, v_dim: int | None = None, q_gain=None, k_gain=None, eps: float = 0.0, bias=None) -> None:
+                         writes: bool, v_dim: int | None = None, q_gain=None, k_gain=None, eps: float = 0.0, bias=None,
+                         v_norm: bool = False) -> None:
         """`bias`: the projections' bias, one float32 per feature of the row, added before the norm.  `nkv` 0: the rows
-        hold queries alone (the mixer reads keys and values that another layer stored)."""
+        hold queries alone (the mixer reads keys and values that another layer stored).  `v_norm`: every head's value is divided
+        by its root mean square before it is stored."""
         ops.qk_norm_rope_store(qkv, ctx, lane, self.inv_freq if self.dims else None, self.magnitude, self.interleaved, nq, nkv,
-                               head_dim, head_dim if v_dim is None else v_dim, q_gain, k_gain, eps, write_kv=writes, bias=bias)
+                               head_dim, head_dim if v_dim is None else v_dim, q_gain, k_gain, eps, write_kv=writes, bias=bias,
+                               v_norm=v_norm)

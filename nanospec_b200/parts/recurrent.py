@@ -1,5 +1,5 @@
 """Mixers whose memory is a matrix per head instead of a growing cache: retention (linear attention with a fixed decay
-per head) and the gated delta rule.  Both keep S [heads, head_dim, v_dim] in float32 in the request's state slot and walk
+per head), the gated delta rule and the state space of Mamba-2.  All keep S [heads, head_dim, v_dim] in float32 in the request's state slot and walk
 a step's tokens in order (csrc/recurrent.cu), so portions of a prompt, single decoded tokens and whole prompts give the
 same numbers; under CUDA graphs they address the state through the device's `qo_indptr` and `state_slot`.
 
@@ -9,6 +9,10 @@ same numbers; under CUDA graphs they address the state through the device's `qo_
                 head_dim^-1/2; beta = sigmoid(b h), g = exp(-exp(A_log) softplus(a h + dt_bias));
                 S = g S;  u = beta (v - S^T k);  S = S + k u^T;  o = S^T q;  per head o / rms(o) times a gain shared by the
                 heads, times silu(gate), output projection.  The last taps - 1 inputs of the convolution are state as well.
+    mamba2      one projection [z | x | B | C | dt]; x, B and C pass a short causal convolution per channel (with a bias) and silu;
+                a = softplus(dt + dt_bias) is the step size of a head and exp(-exp(A_log) a) its decay g;
+                S_t = g S_(t-1) + B_t (a x_t)^T,  o_t = S_t^T C_t + D x_t, B and C shared by the heads of a group;
+                (o silu(z)) normed in equal parts, each by its own root mean square, times a gain, output projection.
 
 The projections are one packed product; the convolution, the rotation, the unit norms, the decay and the read-out's norm are
 float32.
@@ -165,3 +169,90 @@ class GatedDeltaRule(Part):
         gate = proj[:, self.off_g: self.off_g + self.v_size]
         y = ops.head_norm_gate(read, gate, self.gain, self.eps, ctx.buffer("rec_y", self.v_size), ctx, self.heads, self.v_dim)
         return ops.linear(y, self.w_o, ctx.buffer("branch", self.hidden))
+
+
+@register_part("mixer", "mamba2")
+class Mamba2(Part):
+    """params: hidden, heads, v_dim (features of a head), state (rows of S), groups (of heads that share B and C; head h reads group
+    h // (heads / groups)), conv (taps of the short convolution), norm_groups (parts of the read-out's norm), eps, names (optional: keys
+    "in", "conv", "conv_bias", "dt_bias", "A_log", "D", "norm", "o"; default those words, the bias "conv.b")."""
+
+    DEFAULT_NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "A_log": "A_log", "D": "D", "norm": "norm", "o": "o"}
+
+    def __init__(self, spec, dtype, device) -> None:
+        super().__init__(spec, dtype, device)
+        p = spec.params
+        self.hidden, self.heads, self.v_dim = int(p["hidden"]), int(p["heads"]), int(p["v_dim"])
+        self.state_dim, self.groups, self.taps = int(p["state"]), int(p["groups"]), int(p["conv"])
+        self.norm_groups, self.eps = int(p["norm_groups"]), float(p["eps"])
+        self.inner = self.heads * self.v_dim
+        if self.heads % self.groups or self.taps < 1 or self.inner % self.norm_groups:
+            raise ValueError(f"mamba2: {self.heads} heads in {self.groups} groups, {self.taps} taps, {self.inner} features in {self.norm_groups} parts")
+        names = dict(p.get("names") or {})
+        self.names = {k: names.get(k, d) for k, d in self.DEFAULT_NAMES.items()}
+        self.channels = self.inner + 2 * self.groups * self.state_dim        # what the convolution acts on
+        self.columns = self.inner + self.channels + self.heads
+        dp = ops.scan_padded_dim(self.state_dim)
+        self.off_x = 2 * self.groups * dp                                    # of x in the preparation's rows
+        self.rec_cols = -(-(self.off_x + self.inner + 2 * self.heads + self.groups) // 4) * 4
+        self.tail_off = -(-self.heads * self.state_dim * self.v_dim // 4) * 4
+        self.state_floats = -(-(self.tail_off + (self.taps - 1) * self.channels) // 4) * 4
+        self.w_in = self.w_o = self.conv_taps = self.conv_bias = self.a_log = self.dt_bias = self.skip = self.gain = None
+
+    def weight_specs(self) -> dict[str, WeightSpec]:
+        n = self.names
+        small = dict(rule="float32")
+        return {
+            n["in"]: WeightSpec((self.columns, self.hidden)), n["o"]: WeightSpec((self.hidden, self.inner)),
+            n["conv"]: WeightSpec((self.channels, self.taps), std=0.5, **small), n["conv_bias"]: WeightSpec((self.channels,), std=0.1, **small),
+            n["dt_bias"]: WeightSpec((self.heads,), std=0.5, **small), n["A_log"]: WeightSpec((self.heads,), std=0.5, **small),
+            n["D"]: WeightSpec((self.heads,), init="gain", **small), n["norm"]: WeightSpec((self.inner,), init="gain", **small),
+        }
+
+    def bind(self, tensors) -> None:
+        n = self.names
+        self.w_in, self.w_o = _pad_rows(tensors[n["in"]]), tensors[n["o"]].contiguous()
+        self.conv_taps = tensors[n["conv"]].t().contiguous()                 # one row per tap, as the kernel reads them
+        self.conv_bias, self.dt_bias = tensors[n["conv_bias"]].contiguous(), tensors[n["dt_bias"]].contiguous()
+        self.a_log, self.skip, self.gain = (tensors[n[k]].contiguous() for k in ("A_log", "D", "norm"))
+
+    def cache_need(self) -> CacheNeed | None:
+        return None
+
+    def state_need(self) -> StateNeed | None:
+        # S, then the convolution's last taps - 1 inputs [taps - 1, channels]
+        return StateNeed((self.state_floats,), torch.float32)
+
+    def forward(self, x, ctx: StepContext, lane: LaneView, writes: bool = True):
+        proj = ops.linear(x, self.w_in, ctx.buffer("rec_proj", self.w_in.shape[0]))
+        y = ctx.buffer("rec_y", self.inner)
+        self.forward_projected(proj, ctx, lane, writes, y)
+        return ops.linear(y, self.w_o, ctx.buffer("branch", self.hidden))
+
+    # ---- optional: an arrangement that runs the two products inside larger ones of its own (see `GQAAttention.packs_projections`)
+    packs_projections = True
+
+    @property
+    def input_weight(self) -> torch.Tensor:
+        return self.w_in
+
+    @property
+    def output_weight(self) -> torch.Tensor:
+        return self.w_o
+
+    def adopt(self, w_in: torch.Tensor, w_out: torch.Tensor) -> None:
+        if w_in.shape != self.w_in.shape or w_out.shape != self.w_o.shape:
+            raise ValueError("adopt: views of the projections' own shapes are needed")
+        self.w_in, self.w_o = w_in, w_out
+
+    def forward_projected(self, proj: torch.Tensor, ctx: StepContext, lane: LaneView, writes: bool, y: torch.Tensor) -> None:
+        """`proj` [N, >= columns] (rows may lie in a wider buffer): preparation, the state's walk, gate and norm into `y` [N, heads * v_dim]."""
+        if not writes:
+            raise ValueError("a mamba2 mixer owns its state: its lane cannot be shared")
+        rec = ctx.buffer("rec_in", self.rec_cols, torch.float32)
+        ops.ssm_prepare(proj, self.conv_taps, self.conv_bias, self.a_log, self.dt_bias, lane.state, self.tail_off, ctx, rec, self.groups,
+                        self.heads, self.state_dim, self.v_dim)
+        read = ops.linear_scan(rec, lane.state, ctx, ctx.buffer("rec_out", -(-self.inner // 4) * 4, torch.float32), self.heads, self.groups,
+                               self.state_dim, self.v_dim, gated=True, delta=False)
+        ops.ssm_gate_norm(read, rec[:, self.off_x: self.off_x + self.inner], proj, self.skip, self.gain, self.eps, self.norm_groups, y,
+                          lane.state, self.tail_off, self.channels, self.taps, ctx, self.heads, self.v_dim)
