@@ -33,13 +33,17 @@ outputs, the token's side input) beside Dezolorn layers of windowed attention an
 sets every Debuvik kernel's fraction of its bound over that of the sibling's kernel that does the like work.  `--design fubolix`:
 Fubolix models (one dynamic-tanh norm a layer whose output the mixer and a squared-relu feed-forward both read; attention with a
 sink in the denominator - windowed with kept first keys, gated heads and keys as values; with a query temperature; behind a short
-convolution) beside Dezolorn layers of windowed attention.
+convolution) beside Dezolorn layers of windowed attention.  `--design rasezen`: Rasezen models (one RMS norm a layer whose output the
+mixer and the feed-forward both read; windowed attention or the Mamba-2 state space, a dense xielu feed-forward or routed experts with
+identity experts and a shared one) beside Dezolorn layers of windowed attention and the gated delta rule, and Sorizen layers of routed
+experts; `like` as for Debuvik.
 """
 
 from __future__ import annotations
 
 import argparse
 import json
+import math
 import os
 import subprocess
 import sys
@@ -1020,6 +1024,173 @@ def run_design_fubolix(args) -> dict:
     }
 
 
+# ---- Rasezen beside Dezolorn layers of attention and the delta rule, and Sorizen layers of experts (--design rasezen) ---------
+
+RASEZEN_SIZES = {
+    # width; dense feed-forward; attention heads / kv heads / head size; state heads / features / rows / groups; experts (count, identity,
+    # chosen, width), the shared expert's width; layers (attention + dense, state + experts, attention + experts, state + experts);
+    # the siblings' delta rule: heads / q-k heads, of 128 x 128 - a state as large; their latent attention: heads
+    "w2048": dict(width=2048, ff=8192, heads=32, kv_heads=8, dim=64, s_heads=64, s_vdim=64, s_state=128, s_groups=8, experts=32, identity=4,
+                  top=4, eff=1024, shared=2048, layers=8, d_heads=32, d_kv=16, l_heads=16),
+    "w4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, s_heads=128, s_vdim=64, s_state=128, s_groups=8, experts=32, identity=4,
+                  top=4, eff=2048, shared=4096, layers=4, d_heads=64, d_kv=32, l_heads=32),
+}
+RASEZEN_WINDOW, RASEZEN_CONV = 1024, 4
+
+
+def rasezen_config(kind: str, sz: dict) -> dict:
+    """The model, and its siblings at equal width, feed-forward widths, heads, state size, experts and layer count."""
+    d, L, dense = sz["dim"], sz["layers"], {"kind": "dense", "ff": sz["ff"]}
+    base = {"vocab": DESIGN_VOCAB, "width": sz["width"], "norm": {"eps": 1e-6}}
+    if kind == "rasezen":
+        moe = {"kind": "moe", "expert": {"ff": sz["eff"]}, "shared": {"ff": sz["shared"]},
+               "router": {"experts": sz["experts"], "identity": sz["identity"], "top": sz["top"], "scale": 2.0}}
+        attention = {"type": "attention", "mixer": {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5,
+                                                    "mask": {"size": RASEZEN_WINDOW}, "rot": {"dims": d, "base": 1000000.0}}}
+        state = {"type": "mamba2", "mixer": {"heads": sz["s_heads"], "vdim": sz["s_vdim"], "state": sz["s_state"], "groups": sz["s_groups"],
+                                             "conv": RASEZEN_CONV, "norm_groups": sz["s_groups"]}, "mlp": moe}
+        pattern = [{**attention, "mlp": dense}, state, {**attention, "mlp": moe}, state]
+        return {"architecture": "Rasezen", **base, "layers": [pattern[i % 4] for i in range(L)]}
+    if kind == "dezolorn":
+        attention = {"type": "attention", "mlp": dense, "mixer": {
+            "heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": RASEZEN_WINDOW, "keep_first": 0},
+            "rot": {"dims": d, "base": 1000000.0}}}
+        delta = {"type": "delta", "mlp": dense, "mixer": {"heads": sz["d_heads"], "kv_heads": sz["d_kv"], "dim": 128, "vdim": 128, "conv": RASEZEN_CONV}}
+        return {"architecture": "Dezolorn", **base, "layers": [(attention, delta)[i % 2] for i in range(L)],
+                "loop": {"start": 0, "stop": 0, "times": 1}, "logit_scale": 1.0, "logit_softcap": 0.0}
+    mixer = {"heads": sz["l_heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "mask": {"size": RASEZEN_WINDOW},
+             "rot": {"dims": 64, "base": 1000000.0}}
+    moe = {"kind": "moe", "expert": {"ff": sz["eff"]}, "router": {"experts": sz["experts"], "top": sz["top"], "scale": 2.0}}
+    return {"architecture": "Sorizen", **base, "embedding": {"scale": 1.0},
+            "layers": [{"type": "latent_attention", "mixer": mixer, "mlp": dense if i % 4 == 0 else moe} for i in range(L)]}
+
+
+def rasezen_bounds(kind: str, sz: dict, tokens: int, batch: int, context: int, pk: dict) -> dict[str, float]:
+    """Seconds that every kernel of one step needs at least, over all its calls (see kernel_bounds)."""
+    N = tokens or batch
+    W, L, H, nkv, d = sz["width"], sz["layers"], sz["heads"], sz["kv_heads"], sz["dim"]
+    bw, tc, cc = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12, FP32_TFLOPS_NOMINAL * 1e12
+    seen = lambda p: min(p + 1, RASEZEN_WINDOW)
+    pairs = sum(seen(p) for p in range(tokens)) if tokens else batch * seen(context)
+    out: dict[str, float] = {}
+
+    def attention(n):
+        out["ns_qk_norm_rope_store"] = n * 2.0 * N * ((H + nkv) * d * 2 + nkv * d + 2 * nkv * d) / bw
+        if tokens:
+            out["ns_attention_prefill_kept"] = n * 4.0 * H * d * pairs / tc
+        else:
+            out["ns_attention_decode_kept"] = n * 4.0 * pairs * nkv * d / bw
+
+    def scan(n, heads, groups, rows, cols, flops, per_head):  # the state walked on CUDA cores, or read and written once per request
+        operands = (2 * groups * rows + heads * (cols + per_head)) * 4.0 + heads * cols * 4.0
+        out["ns_linear_scan"] = n * (flops * tokens * heads * rows * cols / cc if tokens else batch * (8.0 * heads * rows * cols + operands) / bw)
+
+    def experts(n, identity, rounded_sum):
+        E, top, eff = sz["experts"], sz["top"], sz["eff"]
+        out["ns_router_logits"] = n * (2.0 * N * W + 4.0 * (E + identity) * W) / bw
+        out["ns_moe_combine"] = n * N * W * (2.0 * top + (2.0 if rounded_sum else 8.0)) / bw
+        if tokens:  # the chosen experts' products (an identity choice has none: counted as evenly spread)
+            out["ns_moe_grouped"] = n * 6.0 * N * top * E / (E + identity) * eff * W / tc
+        else:       # the chosen experts' weights, once
+            out["ns_moe_grouped"] = n * min(E, batch * top) * 6.0 * eff * W / bw
+
+    if kind == "dezolorn":
+        out["ns_add_layernorm"] = 2 * L * 12.0 * N * W / bw
+        attention(L // 2)
+        dh, dk = sz["d_heads"], sz["d_kv"]
+        chan = 2 * dk * 128 + dh * 128
+        out["ns_delta_prepare"] = L // 2 * N * (chan * 2 + (chan + 2 * dh) * 4.0) / bw
+        scan(L // 2, dh, dk, 128, 128, 7.0, 2)
+        out["ns_head_norm_gate"] = L // 2 * N * dh * 128 * 8.0 / bw
+        out["ns_swiglu"] = L * 6.0 * N * sz["ff"] / bw
+        return out
+    n_dense = sum(1 for i in range(L) if i % 4 == 0)
+    if kind == "sorizen":
+        out["ns_stream_mix_norm"] = (2 * L + 1) * N * 12.0 * W / bw
+        out["ns_activation"] = n_dense * 4.0 * N * sz["ff"] / bw
+        experts(L - n_dense, 0, True)
+        return out
+    n_state = sum(1 for i in range(L) if i % 4 in (1, 3))
+    sh, sg, sn, sv = sz["s_heads"], sz["s_groups"], sz["s_state"], sz["s_vdim"]
+    out["ns_add_rmsnorm"] = L * 12.0 * N * W / bw
+    attention(L - n_state)
+    chan = sh * sv + 2 * sg * sn
+    out["ns_ssm_prepare"] = n_state * N * (chan * 2 + (chan + 2 * sh) * 4.0) / bw
+    scan(n_state, sh, sg, sn, sv, 5.0, 2)
+    out["ns_ssm_gate_norm"] = n_state * N * sh * sv * 12.0 / bw  # read-out and input in float32, gate and result in bfloat16
+    out["ns_activation_rows"] = n_dense * 4.0 * N * sz["ff"] / bw
+    out["ns_swiglu_rows"] = (L - n_dense) * 6.0 * N * sz["shared"] / bw
+    experts(L - n_dense, sz["identity"], False)
+    return out
+
+
+RASEZEN_LIKE = {"ns_add_rmsnorm": ("dezolorn", "ns_add_layernorm"), "ns_qk_norm_rope_store": ("dezolorn", "ns_qk_norm_rope_store"),
+                "ns_attention_prefill_kept": ("dezolorn", "ns_attention_prefill_kept"),
+                "ns_attention_decode_kept": ("dezolorn", "ns_attention_decode_kept"), "ns_ssm_prepare": ("dezolorn", "ns_delta_prepare"),
+                "ns_linear_scan": ("dezolorn", "ns_linear_scan"), "ns_ssm_gate_norm": ("dezolorn", "ns_head_norm_gate"),
+                "ns_activation_rows": ("sorizen", "ns_activation"), "ns_swiglu_rows": ("dezolorn", "ns_swiglu"),
+                "ns_router_logits": ("sorizen", "ns_router_logits"), "ns_moe_combine": ("sorizen", "ns_moe_combine"),
+                "ns_moe_grouped": ("sorizen", "ns_moe_grouped")}
+
+
+def run_design_rasezen(args) -> dict:
+    import torch
+
+    from nanospec_b200 import random_model
+
+    pk, pk_src = peaks()
+    out_sizes, headline = {}, None
+    for name, sz in RASEZEN_SIZES.items():
+        row = {}
+        for kind in ("rasezen", "dezolorn", "sorizen"):
+            model = random_model(rasezen_config(kind, sz), seed=1, device="cuda", dtype=torch.bfloat16)
+            pages_per_req = -(-(CONTEXT + args.repeats * args.steps + args.warmup + 64) // PAGE)
+            eng = design_engine(model, 64, max(64 * pages_per_req, -(-PREFILL_TOKENS // PAGE) + 8) + 8)
+            rec = {"parameters": sum(math.prod(s.shape) for s in model.weight_specs().values())}
+            for b in (8, 64):
+                pt = time_decode(eng, b, args.steps, args.warmup, args.repeats)
+                rec[f"decode_b{b}_tok_s"] = round(b * 1000.0 / pt["ms"], 1)
+                rec[f"decode_b{b}_ms"] = round(pt["ms"], 4)
+                rec[f"decode_b{b}_clocks"] = {"sm_mhz": pt["clocks"].get("sm_mhz"), "reasons": pt["clocks"].get("reasons")}
+                if b == 8 and kind == "rasezen" and name == "w4096":
+                    headline = pt
+            pre_ms, pre_clocks = time_prefill(eng, warmup=3, iters=5)
+            rec["prefill_tok_s"] = round(PREFILL_TOKENS * 1000.0 / pre_ms, 1)
+            rec["prefill_ms"] = round(pre_ms, 3)
+            rec["prefill_clocks"] = {"sm_mhz": pre_clocks.get("sm_mhz"), "reasons": pre_clocks.get("reasons")}
+            del eng
+            torch.cuda.empty_cache()
+            kernels = {}
+            for what, tokens, batch in (("prefill", PREFILL_TOKENS, 0), ("decode_b64", 0, 64)):
+                timed = time_kernels(model, tokens, batch, CONTEXT)
+                bounds = rasezen_bounds(kind, sz, tokens, batch, CONTEXT, pk)
+                kernels[what] = {k: {"calls": n, "ms": round(ms, 4), "bound_ms": round(bounds[k] * 1e3, 4) if k in bounds else None,
+                                     "frac": round(bounds[k] * 1e3 / ms, 4) if k in bounds and ms > 0 else None}
+                                 for k, (n, ms) in sorted(timed.items(), key=lambda kv: -kv[1][1])}
+            rec["kernels"] = kernels
+            row[kind] = rec
+            del model
+            torch.cuda.empty_cache()
+        # every kernel's fraction of its bound over that of the sibling's kernel that does the like work (below 0.5: twice as far)
+        row["like"] = {what: {k: round(v["frac"] / row[sib]["kernels"][what][other]["frac"], 2)
+                              for k, v in row["rasezen"]["kernels"][what].items() if k in RASEZEN_LIKE and v["frac"]
+                              for sib, other in (RASEZEN_LIKE[k],) if row[sib]["kernels"][what].get(other, {}).get("frac")}
+                       for what in ("prefill", "decode_b64")}
+        out_sizes[name] = row
+    value = out_sizes["w4096"]["rasezen"]["decode_b8_tok_s"]
+    return {
+        "metric": "decode tok/s (Rasezen, width 4,096, 4 layers, batch 8, 1,024-token context)", "value": value, "unit": "tokens/s",
+        "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "ms_per_step": out_sizes["w4096"]["rasezen"]["decode_b8_ms"],
+        "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+        "data": "synthetic: seeded uniform random token ids, random weights",
+        "config": {"design": "rasezen beside dezolorn (attention and delta layers) and sorizen (expert layers)", "sizes": RASEZEN_SIZES,
+                   "vocab": DESIGN_VOCAB, "window": RASEZEN_WINDOW, "conv": RASEZEN_CONV, "seq_len": CONTEXT, "prefill_tokens": PREFILL_TOKENS,
+                   "page": PAGE, "cuda_graphs": True, "peaks": pk_src, "fp32_tflops_nominal": round(FP32_TFLOPS_NOMINAL, 1),
+                   "l2": "the weights of every step are larger than L2"},
+        "gpu_launches": headline["launches"], "clocks": headline["clocks"], "sizes": out_sizes,
+    }
+
+
 def run_reference(args) -> dict:
     from baseline import reference_arm
 
@@ -1036,7 +1207,7 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=SHAPE["num_hidden_layers"])
     ap.add_argument("--no-workloads", action="store_true", help="leave out the 3B continuous-batching and 1B mixed workloads")
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    ap.add_argument("--design", choices=["dezolorn", "sorizen", "debuvik", "fubolix"], help="measure this design beside its closest sibling of equal size instead")
+    ap.add_argument("--design", choices=["dezolorn", "sorizen", "debuvik", "fubolix", "rasezen"], help="measure this design beside its closest sibling of equal size instead")
     args = ap.parse_args()
     args.warmup = max(3, args.warmup)
     args.repeats = max(1, args.repeats)
@@ -1044,7 +1215,7 @@ def main() -> int:
         if int(os.environ.get("RANK", "0")) == 0:
             print(f"bench.py measures a single-GPU engine; --gpus {args.gpus} is not supported")
         return 2
-    out = run_reference(args) if args.impl == "reference" else run_design_fubolix(args) if args.design == "fubolix" else run_design_sorizen(args) if args.design == "sorizen" else run_design_debuvik(args) if args.design == "debuvik" else run_design(args) if args.design else run_ours(args)
+    out = run_reference(args) if args.impl == "reference" else run_design_fubolix(args) if args.design == "fubolix" else run_design_rasezen(args) if args.design == "rasezen" else run_design_sorizen(args) if args.design == "sorizen" else run_design_debuvik(args) if args.design == "debuvik" else run_design(args) if args.design else run_ours(args)
     print(json.dumps(out), flush=True)
     return 0
 
