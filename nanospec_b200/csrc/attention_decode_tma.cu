@@ -434,7 +434,7 @@ int launch_decode_tma(const CUtensorMap& mk, const CUtensorMap& mv, const void* 
     cfg.stream = stream;
     cudaLaunchAttribute attr[2];
     int n_attr = 0;
-    if (ns_pdl_enabled) {
+    if (ns_take_pdl()) {
         attr[n_attr].id = cudaLaunchAttributeProgrammaticStreamSerialization;
         attr[n_attr].val.programmaticStreamSerializationAllowed = 1;
         ++n_attr;

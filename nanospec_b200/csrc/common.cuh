@@ -120,7 +120,14 @@ __device__ __forceinline__ float ns_block_max(float v, float* scratch) {
 // Every block waits before it returns, also one that has nothing to do (a padding row): a grid none of
 // whose blocks waited would complete while its predecessor still runs, and the wait of ITS successor,
 // which covers the grid directly before it only, would no longer mean "everything earlier is done".
-extern int ns_pdl_enabled;
+// A launch right after streams have forked or joined is made without it (ns_full_launch_next): such a kernel has prerequisites
+// beside its predecessor in the stream, and starts when all of them are complete.
+extern int ns_pdl_enabled, ns_pdl_skip_one;
+inline bool ns_take_pdl() {
+    const bool use = ns_pdl_enabled && !ns_pdl_skip_one;
+    ns_pdl_skip_one = 0;
+    return use;
+}
 
 __device__ __forceinline__ void ns_pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void ns_pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
@@ -137,7 +144,7 @@ inline cudaError_t ns_launch_impl(void (*kernel)(KArgs...), dim3 grid, dim3 bloc
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
-    cfg.numAttrs = ns_pdl_enabled ? 1 : 0;
+    cfg.numAttrs = ns_take_pdl() ? 1 : 0;
     return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
 }
 #define NS_LAUNCH(kernel, grid, block, smem, stream, ...) \

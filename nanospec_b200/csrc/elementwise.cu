@@ -8,7 +8,13 @@
 thread_local char ns_error_text[512] = "";
 NS_API const char* ns_last_error() { return ns_error_text; }
 
-int ns_pdl_enabled = 1;
+int ns_pdl_enabled = 1, ns_pdl_skip_one = 0;
+
+// The next kernel launch (on whatever stream) starts only when everything before it is complete.
+NS_API int ns_full_launch_next() {
+    ns_pdl_skip_one = 1;
+    return NS_OK;
+}
 // 1 (default): kernels are launched so that they may overlap the tail of their predecessor
 // (programmatic dependent launch); 0: plain stream order.
 NS_API int ns_set_pdl(int enabled) {

@@ -560,7 +560,7 @@ int launch_tc(const CUtensorMap& mw, const CUtensorMap& mx, void* out, int ldo, 
     cfg.stream = stream;
     cudaLaunchAttribute attr[2];
     int n_attr = 0;
-    if (ns_pdl_enabled) {
+    if (ns_take_pdl()) {
         attr[n_attr].id = cudaLaunchAttributeProgrammaticStreamSerialization;
         attr[n_attr].val.programmaticStreamSerializationAllowed = 1;
         ++n_attr;

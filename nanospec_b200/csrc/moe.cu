@@ -2,7 +2,7 @@
 // the experts' products for steps of a few tokens.
 //
 //   ns_cast_f32        rows of the compute type as float (the router's input: its logits are a float product)
-//   ns_router_logits   the router's float product for a few tokens (longer steps: ns_cast_f32 and the float GEMM)
+//   ns_router_logits   the router's float product (the largest steps and routers: ns_cast_f32 and the float GEMM)
 //   ns_moe_route       scores = sigmoid(logits) (or softmax); consecutive experts form `groups` groups of equal size, ranked by
 //                      the top-2 sum of their scores; all but the `keep` highest-ranked groups are barred; then the `top`
 //                      highest-scoring experts that are not barred; weights = score / (sum of the chosen + 1e-20) * scale,
@@ -11,6 +11,7 @@
 //   ns_moe_plan        counts per expert, their running offsets, and for every (token, choice) its row in the
 //                      order that has each expert's tokens side by side; a choice beyond the experts that have weights (an
 //                      expert that returns its input) has no row: -1
+//   ns_moe_route_plan  both in one launch, for steps of a few tokens
 //   ns_moe_pad_rows    the same rows in a layout where every expert owns a fixed number of rows (for one batched product)
 //   ns_moe_gather      x rows into that order
 //   ns_moe_combine     out[n] = sum_k weight[n, k] * y[row(n, k)] in float (x[n] in place of y for a choice without a row),
@@ -34,51 +35,78 @@ __global__ void cast_f32_kernel(const T* __restrict__ x, long long ldx, float* _
 
 constexpr int kMaxExperts = 1024;
 
-// logits[n, e] = x[n] . w[e] in float, for steps of a few tokens: a block per token, its row in shared memory,
-// a warp per expert in turn (the sum over the row in a fixed order)
-template <typename T>
+// logits[n, e] = x[n] . w[e] in float: a block takes TOK tokens (their rows in shared memory) and eight experts, a warp per expert,
+// so a row of w is read once for TOK tokens.  The sum over a row runs in the same order whatever TOK is.
+template <typename T, int TOK>
 __global__ void __launch_bounds__(256)
-router_logits_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, float* __restrict__ logits, int E, int K) {
+router_logits_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, float* __restrict__ logits, int n_tokens, int E,
+                     int K) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
-    extern __shared__ float xrow[];
-    const int n = blockIdx.x, lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
-    for (int k = threadIdx.x; k < K; k += blockDim.x) xrow[k] = ns_ld(x, (size_t)n * ldx + k);
-    __syncthreads();
-    const bool vec = K % 4 == 0 && ((uintptr_t)w % 16 == 0);
-    for (int e = wib; e < E; e += 8) {
-        const float* wr = w + (size_t)e * K;
-        float a = 0.f;
-        if (vec) {
-            for (int k = lane * 4; k < K; k += 128) {
-                const float4 v = *reinterpret_cast<const float4*>(wr + k);
-                const float4 u = *reinterpret_cast<const float4*>(xrow + k);
-                a = fmaf(v.x, u.x, a); a = fmaf(v.y, u.y, a); a = fmaf(v.z, u.z, a); a = fmaf(v.w, u.w, a);
-            }
-        } else {
-            for (int k = lane; k < K; k += 32) a = fmaf(wr[k], xrow[k], a);
+    extern __shared__ __align__(16) float xrow[];  // [TOK][K4]
+    const int K4 = (K + 3) / 4 * 4;
+    const int n0 = blockIdx.x * TOK, lane = threadIdx.x & 31, e = blockIdx.y * 8 + (threadIdx.x >> 5);
+    const int cnt = min(TOK, n_tokens - n0);
+    const bool vec = K % 8 == 0 && ldx % 8 == 0 && (((uintptr_t)w | (uintptr_t)x) % 16 == 0);
+    if (vec) {
+        const int per_row = K / 8;
+        for (int i = threadIdx.x; i < TOK * per_row; i += blockDim.x) {
+            const int t = i / per_row, k = (i - t * per_row) * 8;
+            float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+            if (t < cnt) ld8(x + (size_t)(n0 + t) * ldx + k, v);
+            st8(xrow + (size_t)t * K4 + k, v);
         }
-        a = ns_warp_sum(a);
-        if (lane == 0) logits[(size_t)n * E + e] = a;
+    } else {
+        for (int i = threadIdx.x; i < TOK * K; i += blockDim.x) {
+            const int t = i / K, k = i - t * K;
+            xrow[(size_t)t * K4 + k] = t < cnt ? ns_ld(x, (size_t)(n0 + t) * ldx + k) : 0.f;
+        }
+    }
+    __syncthreads();
+    if (e >= E) return;
+    const float* wr = w + (size_t)e * K;
+    float a[TOK];
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) a[t] = 0.f;
+    if (vec) {
+#pragma unroll 4
+        for (int k = lane * 4; k < K; k += 128) {
+            const float4 v = *reinterpret_cast<const float4*>(wr + k);
+#pragma unroll
+            for (int t = 0; t < TOK; ++t) {
+                const float4 u = *reinterpret_cast<const float4*>(xrow + (size_t)t * K4 + k);
+                a[t] = fmaf(v.x, u.x, a[t]); a[t] = fmaf(v.y, u.y, a[t]); a[t] = fmaf(v.z, u.z, a[t]); a[t] = fmaf(v.w, u.w, a[t]);
+            }
+        }
+    } else {
+        for (int k = lane; k < K; k += 32) {
+            const float v = wr[k];
+#pragma unroll
+            for (int t = 0; t < TOK; ++t) a[t] = fmaf(v, xrow[(size_t)t * K4 + k], a[t]);
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) {
+        const float v = ns_warp_sum(a[t]);
+        if (lane == 0 && t < cnt) logits[(size_t)(n0 + t) * E + e] = v;
     }
 }
 
-// one warp per token
-__global__ void __launch_bounds__(128)
-moe_route_kernel(const float* __restrict__ logits, int n_tokens, int E, int groups, int keep, int top, float scale,
-                 int softmax, const float* __restrict__ correction, int renormalize, int* __restrict__ ids,
-                 float* __restrict__ weights) {
-    ns_pdl_launch_dependents();
-    ns_pdl_wait();
-    extern __shared__ float rs[];
-    const int lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
-    const int n = blockIdx.x * 4 + wib;
-    if (n >= n_tokens) return;
-    float* sc = rs + (size_t)wib * 3 * E;  // scores, the scores that choose, then group scores (at most E of them)
-    float* cs = sc + E;
+struct RouteRule {
+    int E, groups, keep, top;
+    float scale;
+    int softmax;
+    const float* correction;
+    int renormalize;
+};
+
+// one token by one warp: z [E] its logits, sc [3 E] scratch in shared memory, ids and weights [top] its results
+__device__ __forceinline__ void route_token(const float* __restrict__ z, const RouteRule& r, float* sc, int* __restrict__ ids,
+                                            float* __restrict__ weights, int lane) {
+    const int E = r.E, groups = r.groups, top = r.top;
+    float* cs = sc + E;  // scores, the scores that choose, then group scores (at most E of them)
     float* gs = cs + E;
-    const float* z = logits + (size_t)n * E;
-    if (softmax) {
+    if (r.softmax) {
         float mx = -INFINITY;
         for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
         mx = ns_warp_max(mx);
@@ -93,7 +121,7 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int E, int grou
     } else {
         for (int e = lane; e < E; e += 32) sc[e] = 1.f / (1.f + expf(-z[e]));
     }
-    for (int e = lane; e < E; e += 32) cs[e] = sc[e] + (correction ? correction[e] : 0.f);
+    for (int e = lane; e < E; e += 32) cs[e] = sc[e] + (r.correction ? r.correction[e] : 0.f);
     __syncwarp();
     const float taken = -INFINITY;  // a taken or barred entry
     if (groups > 1) {
@@ -108,7 +136,7 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int E, int grou
         }
         __syncwarp();
         // the best `keep` groups stay; the others' experts are barred
-        for (int round = 0; round < groups - keep; ++round) {  // bar the worst, one a round (the higher index at a tie)
+        for (int round = 0; round < groups - r.keep; ++round) {  // bar the worst, one a round (the higher index at a tie)
             float worst = INFINITY;
             int wi = -1;
             for (int g = lane; g < groups; g += 32) {
@@ -146,42 +174,59 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int E, int grou
         total += w;
         if (lane == k % 32 && k < 32) { mine = w; mine_id = bi; }
         if (k >= 32 && lane == 0) {  // more than 32 choices: written unnormalised, fixed up below
-            ids[(size_t)n * top + k] = bi;
-            weights[(size_t)n * top + k] = w;
+            ids[k] = bi;
+            weights[k] = w;
         }
         if (lane == 0) cs[bi] = taken;
         __syncwarp();
     }
-    const float f = renormalize ? scale / (total + 1e-20f) : scale;
+    const float f = r.renormalize ? r.scale / (total + 1e-20f) : r.scale;
     if (lane < top && lane < 32) {
-        ids[(size_t)n * top + lane] = mine_id;
-        weights[(size_t)n * top + lane] = mine * f;
+        ids[lane] = mine_id;
+        weights[lane] = mine * f;
     }
     __syncwarp();
-    for (int k = 32 + lane; k < top; k += 32) weights[(size_t)n * top + k] *= f;
+    for (int k = 32 + lane; k < top; k += 32) weights[k] *= f;
+}
+
+// one warp per token
+__global__ void __launch_bounds__(128)
+moe_route_kernel(const float* __restrict__ logits, int n_tokens, RouteRule r, int* __restrict__ ids, float* __restrict__ weights) {
+    ns_pdl_launch_dependents();
+    ns_pdl_wait();
+    extern __shared__ float rs[];
+    const int wib = threadIdx.x >> 5;
+    const int n = blockIdx.x * 4 + wib;
+    if (n >= n_tokens) return;
+    route_token(logits + (size_t)n * r.E, r, rs + (size_t)wib * 3 * r.E, ids + (size_t)n * r.top, weights + (size_t)n * r.top, threadIdx.x & 31);
 }
 
 // one block: counts, offsets, rows
-__global__ void __launch_bounds__(1024)
-moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int E, int* __restrict__ offsets, int* __restrict__ row_of,
-                int* __restrict__ pair_of) {
-    ns_pdl_launch_dependents();
-    ns_pdl_wait();
-    __shared__ int count[kMaxExperts], cursor[kMaxExperts];
+__device__ __forceinline__ void plan_pairs(const int* ids, int n_pairs, int E, int* __restrict__ offsets, int* __restrict__ row_of,
+                                           int* __restrict__ pair_of, int* count, int* cursor) {
     const int tid = threadIdx.x;
     for (int e = tid; e < E; e += blockDim.x) count[e] = 0;
     __syncthreads();
     for (int i = tid; i < n_pairs; i += blockDim.x)
         if (ids[i] < E) atomicAdd(&count[ids[i]], 1);
     __syncthreads();
-    if (tid == 0) {
+    if (tid < 32) {  // running sums, 32 experts at a time
         int at = 0;
-        for (int e = 0; e < E; ++e) {
-            offsets[e] = at;
-            cursor[e] = at;
-            at += count[e];
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + tid, c = e < E ? count[e] : 0;
+            int sum = c;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int v = __shfl_up_sync(0xffffffffu, sum, o);
+                if (tid >= o) sum += v;
+            }
+            if (e < E) {
+                offsets[e] = at + sum - c;
+                cursor[e] = at + sum - c;
+            }
+            at += __shfl_sync(0xffffffffu, sum, 31);
         }
-        offsets[E] = at;
+        if (tid == 0) offsets[E] = at;
     }
     __syncthreads();
     // which row of its expert's run a pair gets does not matter to any result: rows are computed alone
@@ -191,6 +236,30 @@ moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int E, int* __restrict
         row_of[i] = row;
         if (pair_of && row >= 0) pair_of[row] = i;
     }
+}
+
+__global__ void __launch_bounds__(1024)
+moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int E, int* __restrict__ offsets, int* __restrict__ row_of,
+                int* __restrict__ pair_of) {
+    ns_pdl_launch_dependents();
+    ns_pdl_wait();
+    __shared__ int count[kMaxExperts], cursor[kMaxExperts];
+    plan_pairs(ids, n_pairs, E, offsets, row_of, pair_of, count, cursor);
+}
+
+// both for a step of a few tokens: one block, its warps take the tokens in turn, then the plan over what they chose
+__global__ void __launch_bounds__(1024)
+moe_route_plan_kernel(const float* __restrict__ logits, int n_tokens, RouteRule r, int* ids, float* __restrict__ weights, int E,
+                      int* __restrict__ offsets, int* __restrict__ row_of, int* __restrict__ pair_of) {
+    ns_pdl_launch_dependents();
+    ns_pdl_wait();
+    __shared__ int count[kMaxExperts], cursor[kMaxExperts];
+    extern __shared__ float rs[];
+    const int warp = threadIdx.x >> 5;
+    for (int n = warp; n < n_tokens; n += blockDim.x >> 5)
+        route_token(logits + (size_t)n * r.E, r, rs + (size_t)warp * 3 * r.E, ids + (size_t)n * r.top, weights + (size_t)n * r.top, threadIdx.x & 31);
+    __syncthreads();  // (a block's own writes to global memory are visible to it after the barrier)
+    plan_pairs(ids, n_tokens * r.top, E, offsets, row_of, pair_of, count, cursor);
 }
 
 // rows of the plan moved to a layout in which every expert owns `capacity` rows: row = expert * capacity + rank in the expert
@@ -403,31 +472,62 @@ NS_API int ns_cast_f32(const void* x, long long ldx, float* out, int n_rows, int
 NS_API int ns_router_logits(const void* x, long long ldx, const float* w, float* logits, int n_tokens, int E, int K, int dtype,
                             cudaStream_t stream) {
     if (n_tokens <= 0) return NS_OK;
-    const size_t smem = (size_t)K * sizeof(float);
-    if (smem > 200 * 1024) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_router_logits: a row of %d floats does not fit shared memory", K);
-    if (dtype == NS_F32) {
-        if (smem > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(router_logits_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-        NS_LAUNCH((router_logits_kernel<float>), n_tokens, 256, smem, stream, (const float*)x, ldx, w, logits, E, K);
-    } else if (dtype == NS_BF16) {
-        if (smem > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(router_logits_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-        NS_LAUNCH((router_logits_kernel<__nv_bfloat16>), n_tokens, 256, smem, stream, (const __nv_bfloat16*)x, ldx, w, logits, E, K);
-    } else {
-        NS_FAIL(NS_ERR_ARGUMENT, "ns_router_logits: unknown dtype %d", dtype);
+    const size_t row = (size_t)(K + 3) / 4 * 4 * sizeof(float);
+    if (row > 200 * 1024) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_router_logits: a row of %d floats does not fit shared memory", K);
+    if (dtype != NS_F32 && dtype != NS_BF16) NS_FAIL(NS_ERR_ARGUMENT, "ns_router_logits: unknown dtype %d", dtype);
+    // tokens to a block: one while that gives few blocks, more as the step grows (two blocks of 100 KB an SM)
+    int tok = n_tokens <= 32 ? 1 : n_tokens <= 128 ? 2 : n_tokens <= 512 ? 4 : 8;
+    while (tok > 1 && tok * row > 100 * 1024) tok /= 2;
+    const size_t smem = tok * row;
+    const dim3 grid((n_tokens + tok - 1) / tok, (E + 7) / 8);
+#define NS_ROUTER(T, TK)                                                                                                              \
+    {                                                                                                                                 \
+        if (smem > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(router_logits_kernel<T, TK>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
+        NS_LAUNCH((router_logits_kernel<T, TK>), grid, 256, smem, stream, (const T*)x, ldx, w, logits, n_tokens, E, K);               \
     }
+#define NS_ROUTER_T(T) { if (tok == 1) NS_ROUTER(T, 1) else if (tok == 2) NS_ROUTER(T, 2) else if (tok == 4) NS_ROUTER(T, 4) else NS_ROUTER(T, 8) }
+    if (dtype == NS_F32) NS_ROUTER_T(float)
+    else NS_ROUTER_T(__nv_bfloat16)
+#undef NS_ROUTER_T
+#undef NS_ROUTER
     NS_CHECK_LAUNCH("ns_router_logits");
     return NS_OK;
 }
 
+namespace {
+int check_rule(const RouteRule& r) {
+    if (r.E < 1 || r.E > kMaxExperts || r.top < 1 || r.top > r.E)
+        NS_FAIL(NS_ERR_UNSUPPORTED, "ns_moe_route: %d experts, %d chosen (at most %d experts)", r.E, r.top, kMaxExperts);
+    if (r.groups > 1 && (r.E % r.groups || r.keep < 1 || r.keep > r.groups || r.keep * (r.E / r.groups) < r.top))
+        NS_FAIL(NS_ERR_ARGUMENT, "ns_moe_route: %d groups over %d experts, %d kept, %d chosen", r.groups, r.E, r.keep, r.top);
+    return NS_OK;
+}
+}  // namespace
+
 NS_API int ns_moe_route(const float* logits, int n_tokens, int E, int groups, int keep, int top, float scale, int softmax,
                         const float* correction, int renormalize, int* ids, float* weights, cudaStream_t stream) {
     if (n_tokens <= 0) return NS_OK;
-    if (E < 1 || E > kMaxExperts || top < 1 || top > E) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_moe_route: %d experts, %d chosen (at most %d experts)", E, top, kMaxExperts);
-    if (groups > 1 && (E % groups || keep < 1 || keep > groups || keep * (E / groups) < top))
-        NS_FAIL(NS_ERR_ARGUMENT, "ns_moe_route: %d groups over %d experts, %d kept, %d chosen", groups, E, keep, top);
+    const RouteRule r{E, groups, keep, top, scale, softmax, correction, renormalize};
+    if (const int rc = check_rule(r)) return rc;
     const size_t smem = (size_t)4 * 3 * E * sizeof(float);
-    NS_LAUNCH(moe_route_kernel, (n_tokens + 3) / 4, 128, smem, stream, logits, n_tokens, E, groups, keep, top, scale, softmax,
-              correction, renormalize, ids, weights);
+    NS_LAUNCH(moe_route_kernel, (n_tokens + 3) / 4, 128, smem, stream, logits, n_tokens, r, ids, weights);
     NS_CHECK_LAUNCH("ns_moe_route");
+    return NS_OK;
+}
+
+// ns_moe_route and ns_moe_plan in one launch of one block: E router outputs, n_experts of them with rows in the plan (at most 512 outputs)
+NS_API int ns_moe_route_plan(const float* logits, int n_tokens, int E, int groups, int keep, int top, float scale, int softmax,
+                             const float* correction, int renormalize, int* ids, float* weights, int n_experts, int* offsets, int* row_of,
+                             int* pair_of, cudaStream_t stream) {
+    if (n_tokens <= 0) return NS_OK;
+    const RouteRule r{E, groups, keep, top, scale, softmax, correction, renormalize};
+    if (const int rc = check_rule(r)) return rc;
+    const int warps = n_tokens < 32 ? (n_tokens < 4 ? 4 : n_tokens) : 32;
+    const size_t smem = (size_t)warps * 3 * E * sizeof(float);
+    if (E > 512 || n_experts < 1 || n_experts > E) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_moe_route_plan: %d of %d experts (at most 512)", n_experts, E);
+    if (smem > 40 * 1024) NS_CUDA(cudaFuncSetAttribute(moe_route_plan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    NS_LAUNCH(moe_route_plan_kernel, 1, warps * 32, smem, stream, logits, n_tokens, r, ids, weights, n_experts, offsets, row_of, pair_of);
+    NS_CHECK_LAUNCH("ns_moe_route_plan");
     return NS_OK;
 }
 

@@ -756,6 +756,42 @@ OVERLAP_MIXED_ATTENTION = True
 _side: dict = {}
 
 
+class SideLane:
+    """A second stream for work that runs beside the current one between two points of a step: `fork()` where its inputs are complete,
+    `with lane.stream():` around its launches, `join()` before anything uses what it made.  Works under graph capture (the events
+    become edges of the graph)."""
+
+    def __init__(self, device: torch.device) -> None:
+        self._stream = torch.cuda.Stream(device=device)
+        self._fork, self._join = torch.cuda.Event(), torch.cuda.Event()
+
+    def fork(self) -> None:
+        self._fork.record(torch.cuda.current_stream())
+        self._stream.wait_event(self._fork)
+
+    def stream(self):
+        lib.load().ns_full_launch_next()
+        return torch.cuda.stream(self._stream)
+
+    def join(self) -> None:
+        self._join.record(self._stream)
+        torch.cuda.current_stream().wait_event(self._join)
+        lib.load().ns_full_launch_next()
+
+
+RUN_BESIDE = True  # False: one stream (measurements and tests)
+
+
+def side_lane(device: torch.device, name: str) -> SideLane | None:
+    """The device's side stream of that name, or None while kernels are timed one by one."""
+    if not RUN_BESIDE or lib.timing_kernels():
+        return None
+    lane = _side.get((device, name))
+    if lane is None:
+        lane = _side[(device, name)] = SideLane(device)
+    return lane
+
+
 def _side_stream(device: torch.device) -> torch.cuda.Stream:
     st = _side.get((device, "stream"))
     if st is None:
@@ -1113,14 +1149,14 @@ def cast_f32(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     return out
 
 
-# the router's logits come from ns_router_logits (every token's block reads the whole router, from L2) while tokens x
-# experts x width stays under this; beyond it from the float32 GEMM, which reads the router once per 64 tokens
-ROUTER_DIRECT_MAX = 1 << 28
+# the router's logits come from ns_router_logits (the router read from L2 once per few tokens) while tokens x experts x width stays
+# under this; beyond it from the float32 GEMM, which reads the router once per 64 tokens
+ROUTER_DIRECT_MAX = 1 << 31
 
 
 def router_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch=None) -> torch.Tensor:
-    """out [N, E] float32 = x @ w^T with float32 products and sums, x in the compute type, w [E, K] float32.  A few tokens:
-    one kernel, a warp per (token, expert); many tokens and a large router: x as float32 (into `scratch(...)`'s buffer) and the float32 GEMM."""
+    """out [N, E] float32 = x @ w^T with float32 products and sums, x in the compute type, w [E, K] float32:
+    one kernel, a warp per expert and a few tokens; very many tokens and a large router: x as float32 (into `scratch(...)`'s buffer) and the float32 GEMM."""
     _cuda(x, w, out)
     n, K = x.shape
     E = w.shape[0]
@@ -1148,6 +1184,28 @@ def moe_route(logits: torch.Tensor, groups: int, keep: int, top: int, scale: flo
         raise KernelError("moe_route: float32 logits [N, E], int32 ids and float32 weights [N, top], contiguous")
     lib.call("ns_moe_route", logits.data_ptr(), n, E, int(groups), int(keep), int(top), float(scale), int(bool(softmax)),
              _ptr(correction), int(bool(renormalize)), ids.data_ptr(), weights.data_ptr(), _stream())
+
+
+def moe_route_plan(logits: torch.Tensor, groups: int, keep: int, top: int, scale: float, ids: torch.Tensor, weights: torch.Tensor, softmax: bool,
+                   correction: torch.Tensor | None, renormalize: bool, n_experts: int, offsets: torch.Tensor, row_of: torch.Tensor,
+                   pair_of: torch.Tensor) -> None:
+    """`moe_route` and `moe_plan` in one launch of one block (`route_plan_ok`)."""
+    _cuda(logits, ids, weights, correction, offsets, row_of, pair_of)
+    n, E = logits.shape
+    for t, name in ((ids, "ids"), (offsets, "offsets"), (row_of, "row_of"), (pair_of, "pair_of")):
+        _i32(t, name)
+    if logits.dtype != torch.float32 or not logits.is_contiguous() or weights.dtype != torch.float32 or not weights.is_contiguous() \
+            or ids.shape != (n, top) or weights.shape != (n, top) or row_of.numel() != n * top or pair_of.numel() != n * top \
+            or offsets.numel() != n_experts + 1 \
+            or (correction is not None and (correction.dtype != torch.float32 or correction.numel() != E or not correction.is_contiguous())):
+        raise KernelError("moe_route_plan: operands as moe_route and moe_plan take them")
+    lib.call("ns_moe_route_plan", logits.data_ptr(), n, E, int(groups), int(keep), int(top), float(scale), int(bool(softmax)), _ptr(correction),
+             int(bool(renormalize)), ids.data_ptr(), weights.data_ptr(), int(n_experts), offsets.data_ptr(), row_of.data_ptr(),
+             pair_of.data_ptr(), _stream())
+
+
+def route_plan_ok(n_tokens: int, n_outputs: int) -> bool:
+    return n_tokens <= 128 and n_outputs <= 512
 
 
 def moe_plan(ids: torch.Tensor, n_experts: int, offsets: torch.Tensor, row_of: torch.Tensor, pair_of: torch.Tensor | None = None) -> None:

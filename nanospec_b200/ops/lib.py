@@ -49,6 +49,7 @@ _SIGNATURES: dict[str, list] = {
     "ns_gemm_bf16_tc_rope": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _F, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I,
                              _P, _P],
     "ns_set_pdl": [_I],
+    "ns_full_launch_next": [],
     "ns_attention_decode_stages": [_I],
     "ns_gemm_bf16_tc": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "ns_gemm_bf16_tc_gated": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
@@ -72,6 +73,7 @@ _SIGNATURES: dict[str, list] = {
     "ns_cast_f32": [_P, _L, _P, _I, _I, _I, _P],
     "ns_router_logits": [_P, _L, _P, _P, _I, _I, _I, _I, _P],
     "ns_moe_route": [_P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P, _P],
+    "ns_moe_route_plan": [_P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P, _I, _P, _P, _P, _P],
     "ns_moe_plan": [_P, _I, _I, _P, _P, _P, _P],
     "ns_moe_grouped": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "ns_moe_pad_rows": [_P, _P, _P, _I, _I, _P],
@@ -132,6 +134,10 @@ def start_kernel_timing() -> None:
     the events keep neighbouring kernels from overlapping, and nothing may be captured into a graph meanwhile)."""
     global _timed
     _timed = []
+
+
+def timing_kernels() -> bool:
+    return _timed is not None
 
 
 def stop_kernel_timing() -> dict[str, tuple[int, float]]:

@@ -270,8 +270,19 @@ class ParallelBlock:
             pending = self._settle(resid, pending)
         h = self.norm_mixer.add_norm(resid, pending, ctx)
         joins = self._joins()
-        if joins:
+        # what joins the stream by itself reads h and touches nothing that the mixer works on: it runs on a stream of its own beside it
+        side = ops.side_lane(resid.device, "feed_forward") if joins else None
+        if side is not None:
+            side.fork()
+        elif joins:
             self.feed_forward.join_stream(h, ctx, resid)
+
+        def rejoin():
+            if side is not None:
+                with side.stream():
+                    self.feed_forward.join_stream(h, ctx, resid)
+                side.join()
+
         if self._packed:
             proj = ops.linear(h, self.w_in, ctx.buffer("par_in", self.w_in.shape[0]))
             mid = ctx.buffer("par_mid", self.w_out.shape[1])
@@ -281,8 +292,14 @@ class ParallelBlock:
                 self.feed_forward.forward_projected(proj[:, ri], ctx, mid[:, ro])
             # a step of a few tokens: the sum into the stream and the next block's norm in this product's epilogue
             sink = self._next_sink(follow, resid, ctx) if ops.norm_fusion_ok(ctx.n_tokens, self.w_out.dtype, self.w_out) else None
-            return resid, ops.linear(mid, self.w_out, ctx.buffer("branch", resid.shape[1]), sink=sink)
+            if sink is not None:  # the product writes the stream itself
+                rejoin()
+            out = ops.linear(mid, self.w_out, ctx.buffer("branch", resid.shape[1]), sink=sink)
+            if sink is None:
+                rejoin()
+            return resid, out
         a = self.mixer.forward(h, ctx, lane, writes)
+        rejoin()
         if self.feed_forward is None or (joins and self.feed_forward.input_weight is None):
             return resid, a
         if joins:

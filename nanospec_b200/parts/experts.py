@@ -110,14 +110,15 @@ class RoutedExperts(Part):
         else:
             self.w_gate_up = torch.cat([self.w_gate, self.w_up], dim=1).contiguous()
 
+    def _logits(self, x, ctx: StepContext) -> torch.Tensor:
+        return ops.router_logits(x, self.w_router, ctx.buffer("router_logits", self.choices, torch.float32),
+                                 scratch=lambda rows, cols: ctx.buffer("router_in", cols, torch.float32, rows=rows))
+
     def route(self, x, ctx: StepContext) -> tuple[torch.Tensor, torch.Tensor]:
         """(chosen experts int32 [N, top], their weights float32 [N, top])"""
-        n = x.shape[0]
-        logits = ops.router_logits(x, self.w_router, ctx.buffer("router_logits", self.choices, torch.float32),
-                                   scratch=lambda rows, cols: ctx.buffer("router_in", cols, torch.float32, rows=rows))
         ids = ctx.buffer("expert_ids", self.top, torch.int32)
         weights = ctx.buffer("expert_weights", self.top, torch.float32)
-        ops.moe_route(logits, self.groups, self.keep, self.top, self.scale, ids, weights, self.softmax, self.correction, self.renormalize)
+        ops.moe_route(self._logits(x, ctx), self.groups, self.keep, self.top, self.scale, ids, weights, self.softmax, self.correction, self.renormalize)
         return ids, weights
 
     # ---- the three ways to run the part ------------------------------------------------------------------------------------
@@ -158,7 +159,13 @@ class RoutedExperts(Part):
     def _grouped(self, x, ids, weights, offsets, row_of, out, ctx: StepContext, resid):
         n = x.shape[0]
         pair_of = ctx.buffer("expert_pairs", self.top, torch.int32)
-        ops.moe_plan(ids, self.experts, offsets, row_of, pair_of)
+        if ids is None:  # a few tokens: the choice and the plan in one launch
+            ids = ctx.buffer("expert_ids", self.top, torch.int32)
+            weights = ctx.buffer("expert_weights", self.top, torch.float32)
+            ops.moe_route_plan(self._logits(x, ctx), self.groups, self.keep, self.top, self.scale, ids, weights, self.softmax, self.correction,
+                               self.renormalize, self.experts, offsets, row_of, pair_of)
+        else:
+            ops.moe_plan(ids, self.experts, offsets, row_of, pair_of)
         act = ctx.buffer("expert_act", self.inter, rows=n * self.top)
         ys = ctx.buffer("expert_out", self.hidden, rows=n * self.top)
         ops.moe_grouped(x, pair_of, offsets, self.w_gate, self.w_up, self.w_down, act, ys, self.top)
@@ -167,12 +174,15 @@ class RoutedExperts(Part):
     def _routed(self, x, ctx: StepContext, out: torch.Tensor, resid: torch.Tensor | None):
         """The routed experts' sum in `out`, or added to the float32 `resid` when that is given; returns where it went."""
         n = x.shape[0]
-        ids, weights = self.route(x, ctx)
         captured = bool(ctx.extras.get("graph")) or torch.cuda.is_current_stream_capturing()
         offsets = ctx.buffer("expert_offsets", 1, torch.int32, rows=self.experts + 1).view(-1)
         row_of = ctx.buffer("expert_rows", self.top, torch.int32)
         grouped_ok = ops.moe_grouped_ok(x, self.hidden, self.inter)
-        if grouped_ok and (GROUPED_MAX is None or n <= GROUPED_MAX or captured):
+        grouped = grouped_ok and (GROUPED_MAX is None or n <= GROUPED_MAX or captured)
+        if grouped and ops.route_plan_ok(n, self.choices):
+            return self._grouped(x, None, None, offsets, row_of, out, ctx, resid)
+        ids, weights = self.route(x, ctx)
+        if grouped:
             return self._grouped(x, ids, weights, offsets, row_of, out, ctx, resid)
         if n <= ROWS_MAX or captured:
             act = ctx.buffer("expert_act", self.inter, rows=n * self.top)

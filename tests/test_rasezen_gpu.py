@@ -217,7 +217,7 @@ def test_routing_with_a_correction_and_identity_experts(E, identity, top, N):
     weights = torch.empty(N, top, dtype=F32, device="cuda")
     ops.moe_route(logits.cuda(), 1, 1, top, 2.5, ids, weights, softmax=True, correction=correction.cuda(), renormalize=False)
     s = torch.softmax(logits.double(), -1)
-    want_ids = torch.argsort(s + correction.double(), dim=-1, descending=True, stable=True)[:, :top]
+    want_ids = torch.argsort(s + correction.double(), dim=-1, descending=True, stable=True)[:, :top].contiguous()
     assert torch.equal(ids.cpu().long(), want_ids)
     assert (weights.cpu().double() - 2.5 * s.gather(1, want_ids)).abs().max() <= 1e-6
     offsets = torch.empty(E + 1, dtype=torch.int32, device="cuda")
