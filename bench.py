@@ -1090,9 +1090,10 @@ def rasezen_bounds(kind: str, sz: dict, tokens: int, batch: int, context: int, p
         out["ns_router_logits"] = n * (2.0 * N * W + 4.0 * (E + identity) * W) / bw
         out["ns_moe_combine"] = n * N * W * (2.0 * top + (2.0 if rounded_sum else 8.0)) / bw
         if tokens:  # the chosen experts' products (an identity choice has none: counted as evenly spread)
-            out["ns_moe_grouped"] = n * 6.0 * N * top * E / (E + identity) * eff * W / tc
+            out["ns_moe_grouped_tc"] = n * 6.0 * N * top * E / (E + identity) * eff * W / tc
+            out["ns_moe_gather"] = n * 4.0 * N * top * E / (E + identity) * W / bw
         else:       # the chosen experts' weights, once
-            out["ns_moe_grouped"] = n * min(E, batch * top) * 6.0 * eff * W / bw
+            out["ns_moe_grouped_tc"] = n * min(E, batch * top) * 6.0 * eff * W / bw
 
     if kind == "dezolorn":
         out["ns_add_layernorm"] = 2 * L * 12.0 * N * W / bw
@@ -1130,7 +1131,7 @@ RASEZEN_LIKE = {"ns_add_rmsnorm": ("dezolorn", "ns_add_layernorm"), "ns_qk_norm_
                 "ns_linear_scan": ("dezolorn", "ns_linear_scan"), "ns_ssm_gate_norm": ("dezolorn", "ns_head_norm_gate"),
                 "ns_activation_rows": ("sorizen", "ns_activation"), "ns_swiglu_rows": ("dezolorn", "ns_swiglu"),
                 "ns_router_logits": ("sorizen", "ns_router_logits"), "ns_moe_combine": ("sorizen", "ns_moe_combine"),
-                "ns_moe_grouped": ("sorizen", "ns_moe_grouped")}
+                "ns_moe_grouped_tc": ("sorizen", "ns_moe_grouped_tc"), "ns_moe_gather": ("sorizen", "ns_moe_gather")}
 
 
 def run_design_rasezen(args) -> dict:

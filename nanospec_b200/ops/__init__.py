@@ -179,6 +179,8 @@ def check_kernel_errors(device: torch.device | None = None) -> None:
                     11: "prefill attention: the loader waited for a free stage", 12: "prefill attention: the MMA issuer waited",
                     13: "prefill attention: a softmax warp waited", 21: "decode attention: the loader waited for a free stage",
                     22: "decode attention: a warp waited for its keys",
+                    41: "routed experts: the TMA producer waited for a free stage", 42: "routed experts: the MMA issuer waited for a tile",
+                    43: "routed experts: the epilogue waited for the accumulator", 44: "routed experts: copies in flight did not land",
                     31: "wait probe: nobody arrives at its barrier"}.get(code, "?")
             raise KernelError(f"a kernel gave up waiting on an mbarrier (the limit is two seconds) - {what} (code {code}); "
                               "its output is not valid")
@@ -1236,6 +1238,26 @@ def moe_grouped(x: torch.Tensor, pair_of: torch.Tensor, offsets: torch.Tensor, w
         raise KernelError("moe_grouped: contiguous bfloat16 operands of the sizes the experts have")
     lib.call("ns_moe_grouped", x.data_ptr(), pair_of.data_ptr(), offsets.data_ptr(), w_gate.data_ptr(), w_up.data_ptr(),
              w_down.data_ptr(), act.data_ptr(), ys.data_ptr(), E, int(top), width, ff, (n * int(top)) // E, _stream())
+    return ys
+
+
+MOE_TILE: int | None = None  # rows of a tile in `moe_grouped_tc` (None: by the rows an expert holds on average)
+
+
+def moe_grouped_tc(xs: torch.Tensor, offsets: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, act: torch.Tensor, ys: torch.Tensor) -> torch.Tensor:
+    """Every expert over its rows of the plan as tcgen05 products whose tiles are found from the offsets on the device
+    (csrc/moe_tcgen05.cu): xs [pairs, width] in the plan's order (`moe_gather`), w_gate_up [E, 2 ff, width] with gate and up rows alternating in
+    runs of GATE_BLOCK, act [pairs, ff] = silu(gate) * up, ys [pairs, width] = act . down."""
+    _cuda(xs, offsets, w_gate_up, w_down, act, ys)
+    _i32(offsets, "offsets")
+    n, width = xs.shape
+    E, ff = w_gate_up.shape[0], w_gate_up.shape[1] // 2
+    if not all(t.is_contiguous() and t.dtype == torch.bfloat16 for t in (xs, w_gate_up, w_down, act, ys)) or w_gate_up.shape[2] != width \
+            or w_down.shape != (E, width, ff) or act.shape != (n, ff) or ys.shape != (n, width) or offsets.numel() != E + 1:
+        raise KernelError("moe_grouped_tc: contiguous bfloat16 operands of the sizes the experts have")
+    tile = MOE_TILE or (256 if n >= 300 * E else 128 if n > 24 * E else 32)
+    lib.call("ns_moe_grouped_tc", xs.data_ptr(), offsets.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), act.data_ptr(), ys.data_ptr(),
+             E, n, width, ff, tile, _tc(xs.device).error.data_ptr(), _stream())
     return ys
 
 

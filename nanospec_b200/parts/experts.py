@@ -13,14 +13,16 @@ and, all optional:
     identity     the last so many outputs of the router stand for experts without tensors whose output is h itself
     shared       {"intermediate": f}: one more gated feed-forward that every token runs, added with weight 1
 
-Four routes, the same numbers up to rounding.  A bfloat16 step (of up to `GROUPED_MAX` tokens when that is set, and every step that a CUDA
-graph captures) lays the (token, choice) pairs out by expert on the device (`ops.moe_plan`) and runs every expert over its
-rows in one tensor-core kernel that reads the counts on the device (`ops.moe_grouped`): each chosen expert's weights are
-read once, nothing comes back to the host.  float32 steps of a few tokens (`ROWS_MAX` or fewer, or captured) run
-`ops.moe_expert_rows`: the chosen experts' rows are streamed per (token, choice).  A longer step brings every expert's tokens side by side (`ops.moe_plan`, `ops.moe_gather`) and reads the counts
-on the host; in bfloat16 every expert then owns the same number of rows (`ops.moe_pad_rows`) and all experts run as one batched
-library product for gate/up and one for down; in float32 each expert that has tokens runs as the framework's gated product and down
-product over its run of rows.  `ops.moe_combine` adds the results per token in the order of the choice (float32 sums, one rounding).
+Several routes, the same numbers up to rounding.  In bfloat16 the (token, choice) pairs are laid out by expert on the device
+(`ops.moe_plan`; up to 128 tokens the choice and the plan are one launch, `ops.moe_route_plan`), and where the experts' width is a multiple
+of 64 every step, short or long, brings the pairs' rows side by side (`ops.moe_gather`) and runs all experts as tcgen05 products
+whose tiles are found from the plan's counts on the device (`ops.moe_grouped_tc`): each chosen expert's weights are read once per 32 to
+256 rows and nothing comes back to the host.  Other widths in multiples of 8: steps of up to `GROUPED_MAX` tokens, and those that a CUDA graph
+captures, run the m16n8k16 kernel `ops.moe_grouped` in the same manner; a longer step reads the counts on the host, every expert then owns the
+same number of rows (`ops.moe_pad_rows`) and all experts run as one batched library product for gate/up and one for down.  float32 steps of a
+few tokens (`ROWS_MAX` or fewer, or captured) run `ops.moe_expert_rows`: the chosen experts' rows are streamed per (token, choice); longer ones
+read the counts on the host and run the framework's products per expert.  `ops.moe_combine` adds the results per token in the order of the
+choice (float32 sums, one rounding).
 
 params: hidden, experts (those with tensors), top, intermediate (an expert's width), groups, keep, scale, score, correction (bool),
 renormalize (default True), identity (default 0), shared, names (optional: "router", "correction"; the experts' tensors are e<k>.gate,
@@ -41,6 +43,7 @@ from .base import Part, WeightSpec
 from .context import StepContext
 from .registry import build_part, register_part
 
+USE_TCGEN05 = True # False: parts built from now on take the m16n8k16 kernel and the library's batched products (measurements)
 ROWS_MAX = 16      # steps of up to this many tokens stream the chosen experts' rows (float32, or widths that are no multiple of 8)
 # bfloat16 steps of up to this many tokens run every expert over its tokens in one tensor-core kernel that reads the counts on the
 # device (None: every step).  Longer steps read the counts on the host and run all experts as ONE batched library product over a
@@ -76,6 +79,7 @@ class RoutedExperts(Part):
         self.shared = None if shared is None else build_part("feed_forward", PartSpec("swiglu", {
             "hidden": self.hidden, "intermediate": int(shared["intermediate"]),
             "names": {k: f"shared.{k}" for k in ("gate", "up", "down")}}), dtype, device)
+        self.tcgen05 = USE_TCGEN05 and dtype == torch.bfloat16 and self.hidden % 8 == 0 and self.inter % ops.GATE_BLOCK == 0
         self.w_router = self.w_gate = self.w_up = self.w_down = self.w_gate_up = None
         self.gate_block = 0
 
@@ -109,6 +113,8 @@ class RoutedExperts(Part):
             self.w_gate_up = packed.reshape(E, 2 * self.inter, self.hidden).contiguous()
         else:
             self.w_gate_up = torch.cat([self.w_gate, self.w_up], dim=1).contiguous()
+        if self.tcgen05:  # every step reads the packed form alone
+            self.w_gate = self.w_up = None
 
     def _logits(self, x, ctx: StepContext) -> torch.Tensor:
         return ops.router_logits(x, self.w_router, ctx.buffer("router_logits", self.choices, torch.float32),
@@ -156,14 +162,22 @@ class RoutedExperts(Part):
         self.shared.forward_projected(u, ctx, act)
 
     # ---- the routed experts ---------------------------------------------------------------------------------------------------
+    def _choose_and_plan(self, x, ctx: StepContext, offsets, row_of, pair_of=None) -> torch.Tensor:
+        """The router, the choice and the pairs' layout by expert; returns the weights float32 [N, top]."""
+        if ops.route_plan_ok(x.shape[0], self.choices):
+            ids, weights = ctx.buffer("expert_ids", self.top, torch.int32), ctx.buffer("expert_weights", self.top, torch.float32)
+            ops.moe_route_plan(self._logits(x, ctx), self.groups, self.keep, self.top, self.scale, ids, weights, self.softmax, self.correction,
+                               self.renormalize, self.experts, offsets, row_of, ctx.buffer("expert_pairs", self.top, torch.int32))
+            return weights
+        ids, weights = self.route(x, ctx)
+        ops.moe_plan(ids, self.experts, offsets, row_of, pair_of)
+        return weights
+
     def _grouped(self, x, ids, weights, offsets, row_of, out, ctx: StepContext, resid):
         n = x.shape[0]
         pair_of = ctx.buffer("expert_pairs", self.top, torch.int32)
-        if ids is None:  # a few tokens: the choice and the plan in one launch
-            ids = ctx.buffer("expert_ids", self.top, torch.int32)
-            weights = ctx.buffer("expert_weights", self.top, torch.float32)
-            ops.moe_route_plan(self._logits(x, ctx), self.groups, self.keep, self.top, self.scale, ids, weights, self.softmax, self.correction,
-                               self.renormalize, self.experts, offsets, row_of, pair_of)
+        if ids is None:
+            weights = self._choose_and_plan(x, ctx, offsets, row_of, pair_of)
         else:
             ops.moe_plan(ids, self.experts, offsets, row_of, pair_of)
         act = ctx.buffer("expert_act", self.inter, rows=n * self.top)
@@ -177,13 +191,16 @@ class RoutedExperts(Part):
         captured = bool(ctx.extras.get("graph")) or torch.cuda.is_current_stream_capturing()
         offsets = ctx.buffer("expert_offsets", 1, torch.int32, rows=self.experts + 1).view(-1)
         row_of = ctx.buffer("expert_rows", self.top, torch.int32)
+        if self.tcgen05:
+            weights = self._choose_and_plan(x, ctx, offsets, row_of)
+            xs = ops.moe_gather(x, row_of, ctx.buffer("expert_in", self.hidden, rows=n * self.top), self.top)
+            ys = ctx.buffer("expert_out", self.hidden, rows=n * self.top)
+            ops.moe_grouped_tc(xs, offsets, self.w_gate_up, self.w_down, ctx.buffer("expert_act", self.inter, rows=n * self.top), ys)
+            return ops.moe_combine(ys, row_of, weights, out, self.top, x=x, resid=resid)
         grouped_ok = ops.moe_grouped_ok(x, self.hidden, self.inter)
-        grouped = grouped_ok and (GROUPED_MAX is None or n <= GROUPED_MAX or captured)
-        if grouped and ops.route_plan_ok(n, self.choices):
+        if grouped_ok and (GROUPED_MAX is None or n <= GROUPED_MAX or captured):
             return self._grouped(x, None, None, offsets, row_of, out, ctx, resid)
         ids, weights = self.route(x, ctx)
-        if grouped:
-            return self._grouped(x, ids, weights, offsets, row_of, out, ctx, resid)
         if n <= ROWS_MAX or captured:
             act = ctx.buffer("expert_act", self.inter, rows=n * self.top)
             ops.moe_expert_rows(x, ids, weights, self.w_gate, self.w_up, self.w_down, act, out)

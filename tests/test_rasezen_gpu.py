@@ -722,20 +722,59 @@ def test_tensor_core_sizes(dim, vdim, heads, kv_heads, size, state, tmp_path):
             close(run_cut(runner, 0, ids, cuts), want, dtype, f"head size {dim}, portions {cuts[:4]}", noise, True)
 
 
+@pytest.mark.parametrize("tile", [32, 128, 256])
+@pytest.mark.parametrize("E,identity,top,N,width,ff", [(6, 2, 3, 300, 72, 64), (3, 1, 2, 7, 64, 128), (40, 0, 2, 90, 136, 192), (1, 1, 1, 40, 8, 64)])
+def test_experts_as_tcgen05_products(E, identity, top, N, width, ff, tile):
+    """The products whose tiles are found from the plan on the device, against float64 on their own operands: experts with no token,
+    with one, with more than a tile holds; rows behind the last pair hold garbage that nothing may pick up."""
+    from nanospec_b200 import ops
+
+    g = torch.Generator().manual_seed(E + N)
+    x = torch.randn(N, width, generator=g).to(BF16)
+    wg, wu = ((torch.randn(E, ff, width, generator=g) / math.sqrt(width)).to(BF16) for _ in range(2))
+    wd = (torch.randn(E, width, ff, generator=g) / math.sqrt(ff)).to(BF16)
+    ids = torch.stack([torch.randperm(E + identity, generator=g)[:top] for _ in range(N)]).int()
+    if E > 2:
+        ids[ids == 0] = E - 1            # expert 0 gets nobody, the last one more than its share (some tokens twice)
+    packed = torch.stack([wg.view(E, ff // 64, 64, width), wu.view(E, ff // 64, 64, width)], dim=2).reshape(E, 2 * ff, width).contiguous().cuda()
+    offsets = torch.empty(E + 1, dtype=torch.int32, device="cuda")
+    row_of = torch.empty(N, top, dtype=torch.int32, device="cuda")
+    ops.moe_plan(ids.cuda(), E, offsets, row_of)
+    buf = lambda cols: torch.full((N * top, cols), float("nan"), dtype=BF16, device="cuda")
+    xs, act, ys = ops.moe_gather(x.cuda(), row_of, buf(width), top), buf(ff), buf(width)
+    old, ops.MOE_TILE = ops.MOE_TILE, tile
+    try:
+        ops.moe_grouped_tc(xs, offsets, packed, wd.cuda(), act, ys)
+    finally:
+        ops.MOE_TILE = old
+    torch.cuda.synchronize()
+    ops.check_kernel_errors()
+    n = int(offsets[-1])
+    assert n == int((ids < E).sum()) and torch.isnan(ys[n:]).all()
+    for t in range(N):
+        for k in range(top):
+            e, row = int(ids[t, k]), int(row_of[t, k])
+            if e >= E:
+                assert row == -1
+                continue
+            a = plain.silu(x[t].double() @ wg[e].double().T) * (x[t].double() @ wu[e].double().T)
+            want = a.to(BF16).double() @ wd[e].double().T
+            assert (ys[row].cpu().double() - want).abs().max() <= 0.02 * max(1.0, float(want.abs().max())), (t, k)
+
+
+@pytest.mark.parametrize("ff", [64, 16], ids=["tcgen05 products", "other widths"])
 @pytest.mark.parametrize("crowded", [False, True], ids=["spread", "crowded"])
-def test_experts_in_long_steps(crowded, tmp_path):
-    """A step of more tokens than the grouped kernel takes: one batched product over equal shares while the experts are chosen evenly,
-    the grouped kernel when a few of them take every token; identity experts among the chosen in both."""
+def test_experts_in_long_steps(crowded, ff, tmp_path):
+    """A step of 600 tokens, its experts chosen evenly or nearly all of them the same two, identity experts among the chosen; expert widths
+    in multiples of 64, and others: one batched product over equal shares while the choice is even."""
     from nanospec_b200.ops import lib
 
-    cfg = config([attn(moe(experts=6, identity=2, top=3, ff=16, shared=16), size=40)])
+    experts = 30 if crowded else 6
+    cfg = config([attn(moe(experts=experts, identity=2, top=3, ff=ff, shared=16), size=40)])
     w = random_weights(cfg, 66)
-    w["l0.mlp.correction"] = torch.zeros(8)
+    w["l0.mlp.correction"] = torch.zeros(experts + 2)
     if crowded:
-        w["l0.mlp.correction"][torch.tensor([1, 7])] = 4.0
-        w["l0.mlp.router"] = w["l0.mlp.router"] * 0.1
-        w["l0.mlp.router"][2] = 0.0
-        w["l0.mlp.correction"][2] = 2.0
+        w["l0.mlp.correction"][torch.tensor([1, 2, experts + 1])] = 2.0
     w = {k: v.to(BF16).float() for k, v in w.items()}
     ids = tokens(600, cfg["vocab"], 67)
     want = plain.forward(cfg, w, ids)
@@ -744,9 +783,10 @@ def test_experts_in_long_steps(crowded, tmp_path):
         lib.start_kernel_timing()
         got = run_cut(runner, 0, ids, [600])
         seen = lib.stop_kernel_timing()
-        if dtype == BF16 and not crowded:
-            assert "ns_moe_pad_rows" in seen, sorted(seen)
+        if dtype == BF16:
+            assert ("ns_moe_grouped_tc" if ff == 64 else "ns_moe_grouped" if crowded else "ns_moe_pad_rows") in seen, sorted(seen)
         close(got, want, dtype, "experts in a long step", torch.full((600,), 0.03), True)
+        close(run_cut(runner, 1, ids, [600]), want, dtype, "the same on two streams", torch.full((600,), 0.03), True)
 
 
 # ---- through the engine: scheduler, graphs, sampling, command line ------------------------------------------------------------
