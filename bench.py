@@ -1084,6 +1084,7 @@ def rasezen_bounds(kind: str, sz: dict, tokens: int, batch: int, context: int, p
     def scan(n, heads, groups, rows, cols, flops, per_head):  # the state walked on CUDA cores, or read and written once per request
         operands = (2 * groups * rows + heads * (cols + per_head)) * 4.0 + heads * cols * 4.0
         out["ns_linear_scan"] = n * (flops * tokens * heads * rows * cols / cc if tokens else batch * (8.0 * heads * rows * cols + operands) / bw)
+        out["ns_ssm_chunked"] = out["ns_linear_scan"]  # (the same work; the chunked form does more flops than the walk needs)
 
     def experts(n, identity, rounded_sum):
         E, top, eff = sz["experts"], sz["top"], sz["eff"]
@@ -1128,7 +1129,7 @@ def rasezen_bounds(kind: str, sz: dict, tokens: int, batch: int, context: int, p
 RASEZEN_LIKE = {"ns_add_rmsnorm": ("dezolorn", "ns_add_layernorm"), "ns_qk_norm_rope_store": ("dezolorn", "ns_qk_norm_rope_store"),
                 "ns_attention_prefill_kept": ("dezolorn", "ns_attention_prefill_kept"),
                 "ns_attention_decode_kept": ("dezolorn", "ns_attention_decode_kept"), "ns_ssm_prepare": ("dezolorn", "ns_delta_prepare"),
-                "ns_linear_scan": ("dezolorn", "ns_linear_scan"), "ns_ssm_gate_norm": ("dezolorn", "ns_head_norm_gate"),
+                "ns_linear_scan": ("dezolorn", "ns_linear_scan"), "ns_ssm_chunked": ("dezolorn", "ns_linear_scan"), "ns_ssm_gate_norm": ("dezolorn", "ns_head_norm_gate"),
                 "ns_activation_rows": ("sorizen", "ns_activation"), "ns_swiglu_rows": ("dezolorn", "ns_swiglu"),
                 "ns_router_logits": ("sorizen", "ns_router_logits"), "ns_moe_combine": ("sorizen", "ns_moe_combine"),
                 "ns_moe_grouped_tc": ("sorizen", "ns_moe_grouped_tc"), "ns_moe_gather": ("sorizen", "ns_moe_gather")}

@@ -225,7 +225,7 @@ linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, con
                    const float* __restrict__ gate, const float* __restrict__ beta, const float* __restrict__ kq,
                    const float* __restrict__ decay, int ld, float* __restrict__ state, long long state_floats,
                    const int* __restrict__ qo_indptr, const int* __restrict__ state_slot, float* __restrict__ out, int ld_out,
-                   int H, int G, int D, int V, int delta) {
+                   int H, int G, int D, int V, int delta, int max_len) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     using Sh = ScanShape<R, LPC, C, ONE>;
@@ -238,7 +238,7 @@ linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, con
     const int col = warp * CW + (lane % CW);       // this lane's first column within the block; the others follow CB apart
     const int e0 = blockIdx.z * Sh::kCols;
     const int start = qo_indptr[b], end = qo_indptr[b + 1];
-    if (end <= start) return;
+    if (end <= start || (max_len > 0 && end - start > max_len)) return;
     const int hk = h / (H / G);
     float* S_mem = state + (long long)state_slot[b] * state_floats + ((long long)h * D + part * R) * V + e0 + col;
     bool active[C];
@@ -632,7 +632,7 @@ namespace {
 template <int R, int LPC, int C, bool ONE>
 int launch_scan_as(const float* q, const float* k, const float* v, const float* gate, const float* beta, const float* kq,
                 const float* decay, int ld, float* state, long long state_floats, const int* qo_indptr, const int* state_slot, float* out, int ld_out,
-                int n_requests, int H, int G, int D, int V, int delta, cudaStream_t stream) {
+                int n_requests, int H, int G, int D, int V, int delta, int max_len, cudaStream_t stream) {
     using Sh = ScanShape<R, LPC, C, ONE>;
     static bool configured = false;
     if (!configured && Sh::kBytes > 48 * 1024) {
@@ -642,7 +642,7 @@ int launch_scan_as(const float* q, const float* k, const float* v, const float* 
     const int col_blocks = (V + Sh::kCols - 1) / Sh::kCols;
     if (H > 65535 || col_blocks > 65535) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_linear_scan: %d heads of %d columns exceed the grid", H, V);
     NS_LAUNCH((linear_scan_kernel<R, LPC, C, ONE>), dim3(n_requests, H, col_blocks), 128, Sh::kBytes, stream, q, k, v, gate, beta, kq, decay, ld,
-              state, state_floats, qo_indptr, state_slot, out, ld_out, H, G, D, V, delta);
+              state, state_floats, qo_indptr, state_slot, out, ld_out, H, G, D, V, delta, max_len);
     NS_CHECK_LAUNCH("ns_linear_scan");
     return NS_OK;
 }
@@ -650,12 +650,12 @@ int launch_scan_as(const float* q, const float* k, const float* v, const float* 
 template <int R, int LPC, int C>
 int launch_scan(const float* q, const float* k, const float* v, const float* gate, const float* beta, const float* kq,
                 const float* decay, int ld, float* state, long long state_floats, const int* qo_indptr, const int* state_slot,
-                float* out, int ld_out, int n_requests, int H, int G, int D, int V, int delta, cudaStream_t stream, int longest) {
+                float* out, int ld_out, int n_requests, int H, int G, int D, int V, int delta, int max_len, cudaStream_t stream, int longest) {
     if (longest <= 1)
         return launch_scan_as<R, LPC, C, true>(q, k, v, gate, beta, kq, decay, ld, state, state_floats, qo_indptr, state_slot, out,
-                                               ld_out, n_requests, H, G, D, V, delta, stream);
+                                               ld_out, n_requests, H, G, D, V, delta, max_len, stream);
     return launch_scan_as<R, LPC, C, false>(q, k, v, gate, beta, kq, decay, ld, state, state_floats, qo_indptr, state_slot, out,
-                                            ld_out, n_requests, H, G, D, V, delta, stream);
+                                            ld_out, n_requests, H, G, D, V, delta, max_len, stream);
 }
 }  // namespace
 
@@ -666,11 +666,13 @@ NS_API int ns_linear_scan_lanes(int lanes) {
     return NS_OK;
 }
 
+// `max_len` > 0: requests of more tokens are left alone (another kernel walks them).
 // `longest`: the most tokens any request brings to this step (1 for decoding).  Long walks over few columns take eight lanes
 // per column instead of four: twice the blocks and half the work per token and lane.
 NS_API int ns_linear_scan(const float* q, const float* k, const float* v, const float* gate, const float* beta, const float* kq,
                           const float* decay, int ld, float* state, long long state_floats, const int* qo_indptr, const int* state_slot, float* out,
-                          int ld_out, int n_requests, int H, int G, int D, int V, int delta, int longest, int n_sms, cudaStream_t stream) {
+                          int ld_out, int n_requests, int H, int G, int D, int V, int delta, int longest, int max_len, int n_sms,
+                          cudaStream_t stream) {
     if (n_requests <= 0) return NS_OK;
     const int R4 = ns_linear_scan_rows(D);
     if (!R4) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_linear_scan: a head of %d features (at most 256)", D);
@@ -686,7 +688,7 @@ NS_API int ns_linear_scan(const float* q, const float* k, const float* v, const 
     const long long blocks4 = (long long)n_requests * H * ((V + 31) / 32);
     const int sms = n_sms > 0 ? n_sms : 148;
     const int lanes = g_scan_lanes == 4 || g_scan_lanes == 8 ? g_scan_lanes : (longest >= 64 && R4 >= 8 && blocks4 < 4ll * sms ? 8 : 4);
-#define NS_SCAN_ARGS q, k, v, gate, beta, kq, decay, ld, state, state_floats, qo_indptr, state_slot, out, ld_out, n_requests, H, G, D, V, delta, stream, longest
+#define NS_SCAN_ARGS q, k, v, gate, beta, kq, decay, ld, state, state_floats, qo_indptr, state_slot, out, ld_out, n_requests, H, G, D, V, delta, max_len, stream, longest
     switch (R4) {
         case 4: return launch_scan<4, 4, 1>(NS_SCAN_ARGS);
         case 8: return lanes == 8 ? launch_scan<4, 8, 1>(NS_SCAN_ARGS) : launch_scan<8, 4, 1>(NS_SCAN_ARGS);

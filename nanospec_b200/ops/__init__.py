@@ -915,11 +915,14 @@ def rotary_prepare(proj: torch.Tensor, ctx, inv_freq: torch.Tensor | None, magni
 
 
 def linear_scan(rec: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, heads: int, kv_heads: int, head_dim: int, v_dim: int,
-                decay: torch.Tensor | None = None, gated: bool = False, delta: bool = True) -> torch.Tensor:
+                decay: torch.Tensor | None = None, gated: bool = False, delta: bool = True, longest: int | None = None,
+                max_len: int = 0) -> torch.Tensor:
     """The recurrence over each request's tokens of this step (csrc/recurrent.cu).  `rec` rows, as the preparation kernels write
     them: [q: kv_heads*Dp | k: kv_heads*Dp | v: heads*v_dim], then, when `gated`, [g: heads | beta: heads] (the delta rule, or with
     `delta` False the state space, whose write is beta * v), then [k . q: kv_heads]; without `gated`, `decay` [heads] float32.
-    `state` [slots, floats] holds S [heads, head_dim, v_dim] at the start of each slot's row; `out` [N, heads*v_dim] float32."""
+    `state` [slots, floats] holds S [heads, head_dim, v_dim] at the start of each slot's row; `out` [N, heads*v_dim] float32.
+    `longest`: the most tokens that a request which is walked brings (default: of the step); `max_len` > 0: requests of more tokens are
+    left alone."""
     _cuda(rec, state, out, decay)
     dp = scan_padded_dim(head_dim)
     off_v = 2 * kv_heads * dp
@@ -936,7 +939,42 @@ def linear_scan(rec: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, 
     lib.call("ns_linear_scan", base, base + 4 * kv_heads * dp, base + 4 * off_v, g_ptr, b_ptr, base + 4 * off_kq,
              None if gated else decay.data_ptr(),
              rec.stride(0), state.data_ptr(), state.stride(0), ctx.qo_indptr.data_ptr(), ctx.state_slot.data_ptr(), out.data_ptr(),
-             out.stride(0), ctx.n_requests, heads, kv_heads, head_dim, v_dim, int(bool(gated and delta)), int(ctx.max_q_len or 1), sm_count(), _stream())
+             out.stride(0), ctx.n_requests, heads, kv_heads, head_dim, v_dim, int(bool(gated and delta)), int(longest or ctx.max_q_len or 1),
+             int(max_len), sm_count(), _stream())
+    return out
+
+
+SSM_CHUNK = 64           # tokens of a chunk in csrc/ssm_chunked.cu
+# requests of at least so many tokens in a step go a chunk at a time, shorter ones (and decoding) a token at a time
+SSM_CHUNKED_MIN = 96
+SSM_SCRATCH_MAX = 1 << 31  # bytes of chunk states; a step that would need more walks token by token
+
+
+def ssm_scan(rec: torch.Tensor, a_log: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, heads: int, groups: int, state_dim: int,
+             v_dim: int) -> torch.Tensor:
+    """The state space over each request's tokens of this step: the preparation's rows `rec` to the read-out `out` [N, heads*v_dim] float32,
+    S in `state` carried on.  Long portions of prompts in chunks of 64 tokens (csrc/ssm_chunked.cu), everything else token by token."""
+    lens = [] if ctx.extras.get("graph") else ctx.q_lens
+    chunks = sum(-(-n // SSM_CHUNK) for n in lens if n >= SSM_CHUNKED_MIN)
+    per_chunk = heads * state_dim * v_dim
+    if not chunks or chunks * per_chunk * 4 > SSM_SCRATCH_MAX:
+        return linear_scan(rec, state, ctx, out, heads, groups, state_dim, v_dim, gated=True, delta=False)
+    short = max((n for n in lens if n < SSM_CHUNKED_MIN), default=0)
+    if short:
+        linear_scan(rec, state, ctx, out, heads, groups, state_dim, v_dim, gated=True, delta=False, longest=short, max_len=SSM_CHUNKED_MIN - 1)
+    _cuda(rec, a_log, state, out)
+    dp = scan_padded_dim(state_dim)
+    off_x = 2 * groups * dp
+    if rec.dtype != torch.float32 or out.dtype != torch.float32 or state.dtype != torch.float32 or rec.stride(1) != 1 or out.stride(1) != 1 \
+            or rec.shape[1] < off_x + heads * (v_dim + 2) or not state.is_contiguous() or state.shape[1] < per_chunk or a_log.dtype != torch.float32 \
+            or a_log.numel() != heads or not a_log.is_contiguous():
+        raise KernelError("ssm_scan: float32 operands of the sizes the heads need")
+    states = ctx.buffer("ssm_states", -(-per_chunk // 4) * 4, torch.float32, rows=chunks)
+    decays = ctx.buffer("ssm_decays", heads, torch.float32, rows=chunks)
+    base = rec.data_ptr()
+    lib.call("ns_ssm_chunked", base, base + 4 * groups * dp, base + 4 * off_x, base + 4 * (off_x + heads * v_dim + heads), rec.stride(0),
+             a_log.data_ptr(), state.data_ptr(), state.stride(0), ctx.qo_indptr.data_ptr(), ctx.state_slot.data_ptr(), out.data_ptr(), out.stride(0),
+             ctx.n_requests, SSM_CHUNKED_MIN, chunks, states.data_ptr(), decays.data_ptr(), heads, groups, state_dim, dp, v_dim, _stream())
     return out
 
 

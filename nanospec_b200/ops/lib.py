@@ -36,7 +36,8 @@ _SIGNATURES: dict[str, list] = {
     "ns_qk_norm_rope_store": [_P, _I, _P, _P, _P, _I, _P, _F, _I, _I, _P, _P, _F, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
     "ns_delta_prepare": [_P, _I, _P, _I, _P, _P, _P, _L, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P],
     "ns_rotary_prepare": [_P, _I, _P, _P, _P, _F, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P],
-    "ns_linear_scan": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+    "ns_linear_scan": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+    "ns_ssm_chunked": [_P, _P, _P, _P, _I, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _P],
     "ns_ssm_prepare": [_P, _I, _P, _P, _I, _P, _P, _P, _L, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "ns_ssm_gate_norm": [_P, _I, _P, _I, _P, _I, _P, _P, _F, _I, _P, _I, _P, _P, _P, _P, _L, _L, _I, _I, _I, _I, _I, _I, _P],
     "ns_head_norm_gate": [_P, _I, _P, _I, _P, _F, _P, _I, _P, _I, _I, _I, _I, _P],

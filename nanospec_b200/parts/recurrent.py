@@ -13,6 +13,8 @@ same numbers; under CUDA graphs they address the state through the device's `qo_
                 a = softplus(dt + dt_bias) is the step size of a head and exp(-exp(A_log) a) its decay g;
                 S_t = g S_(t-1) + B_t (a x_t)^T,  o_t = S_t^T C_t + D x_t, B and C shared by the heads of a group;
                 (o silu(z)) normed in equal parts, each by its own root mean square, times a gain, output projection.
+                Long portions of prompts run in chunks of 64 tokens (csrc/ssm_chunked.cu: products over the chunk's tokens, the state
+                carried between chunks), the same sums in another order.
 
 The projections are one packed product; the convolution, the rotation, the unit norms, the decay and the read-out's norm are
 float32.
@@ -252,7 +254,7 @@ class Mamba2(Part):
         rec = ctx.buffer("rec_in", self.rec_cols, torch.float32)
         ops.ssm_prepare(proj, self.conv_taps, self.conv_bias, self.a_log, self.dt_bias, lane.state, self.tail_off, ctx, rec, self.groups,
                         self.heads, self.state_dim, self.v_dim)
-        read = ops.linear_scan(rec, lane.state, ctx, ctx.buffer("rec_out", -(-self.inner // 4) * 4, torch.float32), self.heads, self.groups,
-                               self.state_dim, self.v_dim, gated=True, delta=False)
+        read = ops.ssm_scan(rec, self.a_log, lane.state, ctx, ctx.buffer("rec_out", -(-self.inner // 4) * 4, torch.float32), self.heads,
+                            self.groups, self.state_dim, self.v_dim)
         ops.ssm_gate_norm(read, rec[:, self.off_x: self.off_x + self.inner], proj, self.skip, self.gain, self.eps, self.norm_groups, y,
                           lane.state, self.tail_off, self.channels, self.taps, ctx, self.heads, self.v_dim)

@@ -301,10 +301,13 @@ def test_preparation_with_biases_norms_and_unit_values(H, G, d, dv, dims, dtype)
 
 @BOTH
 @pytest.mark.parametrize("H,V,N,G,taps,parts", [(4, 6, 5, 2, 3, 3), (2, 16, 16, 1, 4, 1), (6, 8, 24, 3, 2, 4), (3, 5, 40, 3, 1, 5), (8, 64, 64, 2, 4, 2),
-                                               (1, 40, 130, 1, 6, 20), (12, 8, 8, 4, 5, 12)])
-def test_state_space_kernels_alone(H, V, N, G, taps, parts, dtype):
-    """Preparation, scan, gate and norm over two requests in portions (state and convolution tail carried in their slots) against
-    the plain walk over the whole sequences; rows wider than the projection; decays from fast to slow, one step size near zero."""
+                                               (1, 40, 130, 1, 6, 20), (12, 8, 8, 4, 5, 12), (2, 150, 70, 1, 4, 3)])
+@pytest.mark.parametrize("chunked", [False, True], ids=["token by token", "in chunks"])
+def test_state_space_kernels_alone(chunked, H, V, N, G, taps, parts, dtype, monkeypatch):
+    """Preparation, the state's walk, gate and norm over two requests in portions (state and convolution tail carried in their slots)
+    against the plain walk over the whole sequences; rows wider than the projection; decays from fast to slow, one step size near
+    zero and one head that forgets nearly everything.  In chunks: portions of one chunk, of several and of a part of one, beside
+    a request of one token."""
     from nanospec_b200 import ops
     from nanospec_b200.parts.recurrent import Mamba2
     from nanospec_b200.config.recipe import PartSpec
@@ -315,8 +318,10 @@ def test_state_space_kernels_alone(H, V, N, G, taps, parts, dtype):
     t = {n: torch.randn(s.shape, generator=g) for n, s in part.weight_specs().items()}
     t["A_log"], t["dt_bias"], t["conv"] = 0.8 * t["A_log"] - 1.0, t["dt_bias"] - 1.0, 0.5 * t["conv"]
     t["dt_bias"][0] = -9.0
+    t["A_log"][-1] = 2.5
+    monkeypatch.setattr(ops, "SSM_CHUNKED_MIN", 2 if chunked else 1 << 30)
     part.bind({n: v.to(dtype if n in ("in", "o") else F32).cuda() for n, v in t.items()})
-    lengths, cuts = [90, 23], [[40, 1, 2, 47], [3, 7, 1, 12]]
+    lengths, cuts = [240, 80], [[130, 1, 2, 107], [3, 64, 1, 12]]
     seqs = [torch.randn(n, part.columns + 8, generator=g).to(dtype) for n in lengths]
     want = []
     rnd = (lambda x: x) if dtype == F32 else (lambda x: x.to(BF16).double())  # the convolution's result is rounded like a projection's
@@ -332,7 +337,7 @@ def test_state_space_kernels_alone(H, V, N, G, taps, parts, dtype):
     bufs = {}
 
     def buffer(name, cols, dt=None, rows=None):
-        bufs[name] = torch.full((n_rows, cols), float("nan"), dtype=dt or dtype, device="cuda")
+        bufs[name] = torch.full((rows or n_rows, cols), float("nan"), dtype=dt or dtype, device="cuda")
         return bufs[name]
 
     at, got = [0, 0], [[], []]
@@ -343,7 +348,7 @@ def test_state_space_kernels_alone(H, V, N, G, taps, parts, dtype):
         ctx = SimpleNamespace(
             token_req=torch.tensor([b for b in range(2) for _ in range(ns[b])], dtype=torch.int32, device="cuda"),
             qo_indptr=torch.tensor([0, ns[0], n_rows], dtype=torch.int32, device="cuda"),
-            state_slot=torch.tensor([2, 0], dtype=torch.int32, device="cuda"), n_requests=2, max_q_len=max(ns), buffer=buffer)
+            state_slot=torch.tensor([2, 0], dtype=torch.int32, device="cuda"), n_requests=2, max_q_len=max(ns), q_lens=ns, extras={}, buffer=buffer)
         out = torch.zeros(n_rows, inner + 8, dtype=dtype, device="cuda")
         part.forward_projected(rows, ctx, lane, True, out[:, :inner])
         o = out.cpu().double()
@@ -353,7 +358,7 @@ def test_state_space_kernels_alone(H, V, N, G, taps, parts, dtype):
         at = [at[b] + ns[b] for b in range(2)]
     assert not lane.state[1].any()  # the slot that nobody holds
     for b in range(2):
-        off = (torch.cat(got[b]) - want[b]).abs()
+        off = (torch.cat(got[b]) - want[b]).abs()  # (nothing may stay unwritten: a NaN fails the comparison)
         size = float(want[b].abs().max())
         if dtype == F32:
             assert off.max() <= 5e-5 * size, (b, float(off.max()), size)
@@ -579,6 +584,22 @@ def far_token_case():
     lost = list(ids)
     lost[31] = 47
     return cfg, w, ids, lost
+
+
+@BOTH
+@pytest.mark.parametrize("least", [2, 1 << 30], ids=["in chunks", "token by token"])
+def test_the_walk_does_not_depend_on_the_cut(least, dtype, tmp_path, monkeypatch):
+    """Portions that begin and end inside chunks, on their edges and one beside them, with the state walked in chunks and token by token."""
+    from nanospec_b200 import ops
+
+    monkeypatch.setattr(ops, "SSM_CHUNKED_MIN", least)
+    cfg = config([mamba(dense(16), heads=4, vdim=12, state=24, groups=2, conv=4), attn(None, dim=16, vdim=8, size=30), mamba(None, heads=6, vdim=5, state=7, groups=3)])
+    runner, w = make(tmp_path, cfg, seed=58, dtype=dtype, page=16, blocks=40)
+    ids = tokens(260, cfg["vocab"], 59)
+    want = plain.forward(cfg, w, ids)
+    noise = rounding(cfg, w, ids, want, samples=1) if dtype == BF16 else None
+    for cuts in ([260], [64, 64, 65, 63], [2, 127, 1, 2, 66], [100, 3, 100]):
+        close(run_cut(runner, 0, ids, cuts), want, dtype, f"portions {cuts}", noise)
 
 
 @BOTH
