@@ -725,15 +725,18 @@ NS_API int ns_ssm_prepare(const void* proj, int ld_proj, const float* taps, cons
     if (n_taps < 1 || G < 1 || H % G || Dp < D || Dp % 4) NS_FAIL(NS_ERR_ARGUMENT, "ns_ssm_prepare: taps=%d heads=%d/%d D=%d Dp=%d", n_taps, H, G, D, Dp);
     if (dtype != NS_F32 && dtype != NS_BF16) NS_FAIL(NS_ERR_ARGUMENT, "ns_ssm_prepare: unknown dtype %d", dtype);
     const size_t smem = (size_t)2 * G * D * sizeof(float);
-    if (smem > 48 * 1024) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_ssm_prepare: %d groups of %d features do not fit shared memory", G, D);
+    if (smem > 200 * 1024) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_ssm_prepare: %d groups of %d features do not fit shared memory", G, D);
     const size_t esz = dtype == NS_F32 ? 4 : 2;
     const bool vec = (H * V) % 8 == 0 && D % 8 == 0 && (ld_proj * esz) % 16 == 0 && ld_rec % 4 == 0 && state_floats % 4 == 0 && tail_off % 4 == 0 &&
                      (((uintptr_t)proj | (uintptr_t)taps | (uintptr_t)conv_bias | (uintptr_t)state | (uintptr_t)rec) % 16 == 0);
 #define NS_SSM_PREPARE(T, VC)                                                                                                         \
-    NS_LAUNCH((ssm_prepare_kernel<T, VC>), n_tokens, 256, smem, stream, (const T*)proj, ld_proj, taps, conv_bias, n_taps, a_log, dt_bias, \
-              state, state_floats, tail_off, token_req, qo_indptr, state_slot, rec, ld_rec, G, H, D, Dp, V)
-    if (dtype == NS_F32) { if (vec) NS_SSM_PREPARE(float, 8); else NS_SSM_PREPARE(float, 1); }
-    else { if (vec) NS_SSM_PREPARE(__nv_bfloat16, 8); else NS_SSM_PREPARE(__nv_bfloat16, 1); }
+    {                                                                                                                                  \
+        if (smem > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(ssm_prepare_kernel<T, VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
+        NS_LAUNCH((ssm_prepare_kernel<T, VC>), n_tokens, 256, smem, stream, (const T*)proj, ld_proj, taps, conv_bias, n_taps, a_log, dt_bias, \
+                  state, state_floats, tail_off, token_req, qo_indptr, state_slot, rec, ld_rec, G, H, D, Dp, V);                        \
+    }
+    if (dtype == NS_F32) { if (vec) NS_SSM_PREPARE(float, 8) else NS_SSM_PREPARE(float, 1) }
+    else { if (vec) NS_SSM_PREPARE(__nv_bfloat16, 8) else NS_SSM_PREPARE(__nv_bfloat16, 1) }
 #undef NS_SSM_PREPARE
     NS_CHECK_LAUNCH("ns_ssm_prepare");
     return NS_OK;

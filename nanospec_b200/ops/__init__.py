@@ -944,6 +944,14 @@ def linear_scan(rec: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, 
     return out
 
 
+SCAN_MAX_DIM = 256       # rows of S that the token walk holds in registers
+
+
+def ssm_padded_dim(state_dim: int) -> int:
+    """The width that a group's B and C are padded to in the preparation's rows: the token walk's, or a multiple of 4 beyond its limit."""
+    return scan_padded_dim(state_dim) if state_dim <= SCAN_MAX_DIM else -(-state_dim // 4) * 4
+
+
 SSM_CHUNK = 64           # tokens of a chunk in csrc/ssm_chunked.cu
 # requests of at least so many tokens in a step go a chunk at a time, shorter ones (and decoding) a token at a time
 SSM_CHUNKED_MIN = 96
@@ -953,17 +961,20 @@ SSM_SCRATCH_MAX = 1 << 31  # bytes of chunk states; a step that would need more 
 def ssm_scan(rec: torch.Tensor, a_log: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, heads: int, groups: int, state_dim: int,
              v_dim: int) -> torch.Tensor:
     """The state space over each request's tokens of this step: the preparation's rows `rec` to the read-out `out` [N, heads*v_dim] float32,
-    S in `state` carried on.  Long portions of prompts in chunks of 64 tokens (csrc/ssm_chunked.cu), everything else token by token."""
-    lens = [] if ctx.extras.get("graph") else ctx.q_lens
-    chunks = sum(-(-n // SSM_CHUNK) for n in lens if n >= SSM_CHUNKED_MIN)
+    S in `state` carried on.  Long portions of prompts in chunks of 64 tokens (csrc/ssm_chunked.cu), everything else token by token; states
+    of more rows than the token walk takes always in chunks (single tokens as chunks of one)."""
+    lens = [1] * ctx.n_requests if ctx.extras.get("graph") else ctx.q_lens
+    least = SSM_CHUNKED_MIN if state_dim <= SCAN_MAX_DIM else 1
+    chunks = sum(-(-n // SSM_CHUNK) for n in lens if n >= least)
     per_chunk = heads * state_dim * v_dim
-    if not chunks or chunks * per_chunk * 4 > SSM_SCRATCH_MAX:
-        return linear_scan(rec, state, ctx, out, heads, groups, state_dim, v_dim, gated=True, delta=False)
-    short = max((n for n in lens if n < SSM_CHUNKED_MIN), default=0)
-    if short:
-        linear_scan(rec, state, ctx, out, heads, groups, state_dim, v_dim, gated=True, delta=False, longest=short, max_len=SSM_CHUNKED_MIN - 1)
+    if least > 1:
+        if not chunks or chunks * per_chunk * 4 > SSM_SCRATCH_MAX:
+            return linear_scan(rec, state, ctx, out, heads, groups, state_dim, v_dim, gated=True, delta=False)
+        short = max((n for n in lens if n < least), default=0)
+        if short:
+            linear_scan(rec, state, ctx, out, heads, groups, state_dim, v_dim, gated=True, delta=False, longest=short, max_len=least - 1)
     _cuda(rec, a_log, state, out)
-    dp = scan_padded_dim(state_dim)
+    dp = ssm_padded_dim(state_dim)
     off_x = 2 * groups * dp
     if rec.dtype != torch.float32 or out.dtype != torch.float32 or state.dtype != torch.float32 or rec.stride(1) != 1 or out.stride(1) != 1 \
             or rec.shape[1] < off_x + heads * (v_dim + 2) or not state.is_contiguous() or state.shape[1] < per_chunk or a_log.dtype != torch.float32 \
@@ -974,7 +985,7 @@ def ssm_scan(rec: torch.Tensor, a_log: torch.Tensor, state: torch.Tensor, ctx, o
     base = rec.data_ptr()
     lib.call("ns_ssm_chunked", base, base + 4 * groups * dp, base + 4 * off_x, base + 4 * (off_x + heads * v_dim + heads), rec.stride(0),
              a_log.data_ptr(), state.data_ptr(), state.stride(0), ctx.qo_indptr.data_ptr(), ctx.state_slot.data_ptr(), out.data_ptr(), out.stride(0),
-             ctx.n_requests, SSM_CHUNKED_MIN, chunks, states.data_ptr(), decays.data_ptr(), heads, groups, state_dim, dp, v_dim, _stream())
+             ctx.n_requests, least, chunks, states.data_ptr(), decays.data_ptr(), heads, groups, state_dim, dp, v_dim, _stream())
     return out
 
 
@@ -990,7 +1001,7 @@ def ssm_prepare(proj: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor,
     for t, size, name in ((taps, None, "taps"), (conv_bias, channels, "conv_bias"), (a_log, heads, "a_log"), (dt_bias, heads, "dt_bias")):
         if t.dtype != torch.float32 or not t.is_contiguous() or (size is not None and t.numel() != size):
             raise KernelError(f"ssm_prepare: {name} must be contiguous float32" + (f" of {size} entries" if size else ""))
-    dp = scan_padded_dim(state_dim)
+    dp = ssm_padded_dim(state_dim)
     if taps.dim() != 2 or taps.shape[1] != channels or proj.stride(1) != 1 or proj.shape[1] < heads * v_dim + channels + heads \
             or rec.dtype != torch.float32 or rec.stride(1) != 1 or rec.shape[1] < 2 * groups * dp + heads * v_dim + 2 * heads + groups \
             or state.dtype != torch.float32 or not state.is_contiguous() or state.shape[1] < tail_off + (taps.shape[0] - 1) * channels:

@@ -194,7 +194,7 @@ class Mamba2(Part):
         self.names = {k: names.get(k, d) for k, d in self.DEFAULT_NAMES.items()}
         self.channels = self.inner + 2 * self.groups * self.state_dim        # what the convolution acts on
         self.columns = self.inner + self.channels + self.heads
-        dp = ops.scan_padded_dim(self.state_dim)
+        dp = ops.ssm_padded_dim(self.state_dim)
         self.off_x = 2 * self.groups * dp                                    # of x in the preparation's rows
         self.rec_cols = -(-(self.off_x + self.inner + 2 * self.heads + self.groups) // 4) * 4
         self.tail_off = -(-self.heads * self.state_dim * self.v_dim // 4) * 4

@@ -301,7 +301,7 @@ def test_preparation_with_biases_norms_and_unit_values(H, G, d, dv, dims, dtype)
 
 @BOTH
 @pytest.mark.parametrize("H,V,N,G,taps,parts", [(4, 6, 5, 2, 3, 3), (2, 16, 16, 1, 4, 1), (6, 8, 24, 3, 2, 4), (3, 5, 40, 3, 1, 5), (8, 64, 64, 2, 4, 2),
-                                               (1, 40, 130, 1, 6, 20), (12, 8, 8, 4, 5, 12), (2, 150, 70, 1, 4, 3)])
+                                               (1, 40, 130, 1, 6, 20), (12, 8, 8, 4, 5, 12), (2, 150, 70, 1, 4, 3), (4, 6, 300, 2, 3, 1)])
 @pytest.mark.parametrize("chunked", [False, True], ids=["token by token", "in chunks"])
 def test_state_space_kernels_alone(chunked, H, V, N, G, taps, parts, dtype, monkeypatch):
     """Preparation, the state's walk, gate and norm over two requests in portions (state and convolution tail carried in their slots)
@@ -823,6 +823,20 @@ def test_greedy_generation_through_the_engine(dtype, graphs, tmp_path):
     eng = Engine(model, EngineConfig(num_blocks=64, block_size=4, max_running=3, prefill_chunk=11, cuda_graphs=graphs,
                                      graph_buckets=(1, 2, 4)))
     greedy(eng, cfg, w, [tokens(n, cfg["vocab"], 80 + n) for n in (3, 30, 1, 17, 12)], 12, dtype)
+
+
+def test_a_state_larger_than_the_token_walk_takes(tmp_path):
+    """More rows of the state than the token walk holds: single tokens too run as chunks, under graphs as well."""
+    from nanospec_b200 import Engine, EngineConfig
+
+    cfg = config([mamba(dense(16), heads=2, vdim=8, state=260, groups=1), mamba(None, heads=2, vdim=8, state=16, groups=1)])
+    runner, w = make(tmp_path, cfg, seed=61)
+    ids = tokens(80, cfg["vocab"], 62)
+    want = plain.forward(cfg, w, ids)
+    for cuts in ([80], [], [30, 2, 40]):
+        close(run_cut(runner, 0, ids, cuts), want, F32, f"portions {cuts}")
+    eng = Engine(runner.model, EngineConfig(num_blocks=64, block_size=4, max_running=3, prefill_chunk=11, graph_buckets=(1, 2, 4)))
+    greedy(eng, cfg, w, [tokens(n, cfg["vocab"], 70 + n) for n in (3, 30, 1)], 8, F32)
 
 
 def test_command_line(tmp_path):
