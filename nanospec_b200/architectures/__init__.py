@@ -1,3 +1,3 @@
-from . import debuvik, dezolorn, fubolix, llama, rasezen, sorizen  # registers Debuvik, Dezolorn, Fubolix, LlamaForCausalLM, Rasezen and Sorizen
+from . import debuvik, dezolorn, fubolix, llama, rasezen, sorizen, tafesun  # registers Debuvik, Dezolorn, Fubolix, LlamaForCausalLM, Rasezen, Sorizen and Tafesun
 
-__all__ = ["debuvik", "dezolorn", "fubolix", "llama", "rasezen", "sorizen"]
+__all__ = ["debuvik", "dezolorn", "fubolix", "llama", "rasezen", "sorizen", "tafesun"]

@@ -35,7 +35,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
                         float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters,
                         const int* __restrict__ rows, int nq, int nkv, int page_size, float scale, int window,
                         int n_splits, int head_tiles, int keep_first, int wide_weights, int mask_chunk, float softcap,
-                        int dk, int dv, const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int gate_stride) {
+                        int dk, int dv_row, int dv_slice, int slices, const float* __restrict__ sink, const OutGate og) {
     ns_pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one before it reads
     ns_pdl_wait();               // everything below sees the previous kernel's results
     using Tile = NsTile<D>;
@@ -47,7 +47,11 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
 
     const int split = blockIdx.x, z = blockIdx.z;
     const int n = rows ? rows[z] : z;  // the token this block works for
-    const int hk = blockIdx.y / head_tiles, ht = blockIdx.y - hk * head_tiles;
+    // (kv head, tile of 16 query heads, slice of the values' features)
+    const int slice = blockIdx.y % slices, hy = blockIdx.y / slices;
+    const int v0 = slice * dv_slice, dv = min(dv_slice, dv_row - v0);
+    v_cache += v0;
+    const int hk = hy / head_tiles, ht = hy - hk * head_tiles;
     const int req = token_req[n];
     if (req < 0) return;
     if (qo_indptr[req + 1] - qo_indptr[req] != 1) return;
@@ -86,7 +90,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
     for (int st = 0; st < kStages - 1; ++st) {
         if (st < n_tiles) {
             __nv_bfloat16* kn = kv + (size_t)st * 2 * kTileKeys * S;
-            load_kv_tile<D>(kn, kn + kTileKeys * S, k_cache, v_cache, bt, k0 + st * kTileKeys, kstart, k1, hk, nkv, page_size, page_shift, win_start, gap, dk, dv);
+            load_kv_tile<D>(kn, kn + kTileKeys * S, k_cache, v_cache, bt, k0 + st * kTileKeys, kstart, k1, hk, nkv, page_size, page_shift, win_start, gap, dk, dv, dv_row);
         }
         ns_cp_async_commit();
     }
@@ -109,7 +113,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
         if (t + kStages - 1 < n_tiles) {
             __nv_bfloat16* kn = kv + (size_t)((t + kStages - 1) % kStages) * 2 * kTileKeys * S;
             load_kv_tile<D>(kn, kn + kTileKeys * S, k_cache, v_cache, bt, k0 + (t + kStages - 1) * kTileKeys, kstart, k1, hk,
-                            nkv, page_size, page_shift, win_start, gap, dk, dv);
+                            nkv, page_size, page_shift, win_start, gap, dk, dv, dv_row);
         }
         ns_cp_async_commit();
         ns_cp_async_wait<kStages - 1>();  // tile t has landed; the two after it stay in flight
@@ -236,10 +240,9 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
             // a sink: exp(sink[h]) joins the denominator (maxima and sums are in base 2); a gate: the head's output times its sigmoid
             if (sink) lt += ns_exp2(sink[h] * kLog2e - mt);
             float res = acc / lt;
-            if (gate) res *= 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)n * gate_stride + h])));
-            out[(size_t)n * o_stride + (size_t)h * dv + col] = __float2bfloat16_rn(res);
+            out[(size_t)n * o_stride + (size_t)h * dv_row + v0 + col] = __float2bfloat16_rn(res * gate_factor(og, n, h, h * dv_row + v0 + col));
         } else {
-            const size_t slot = ((size_t)z * nq + h) * n_splits + split;
+            const size_t slot = (((size_t)z * nq + h) * slices + slice) * n_splits + split;
             part_o[slot * D + col] = acc;
             if (col == 0) {
                 part_ml[slot * 2] = mt;
@@ -265,7 +268,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
         const int row = e / D, col = e - row * D;
         if (col >= dv) continue;
         const int h = h0 + row;
-        const size_t base = ((size_t)z * nq + h) * n_splits;
+        const size_t base = (((size_t)z * nq + h) * slices + slice) * n_splits;
         // every split's maximum, sum and partial value are requested together, then combined in split order
         float ms[kMaxSplits], ls[kMaxSplits], os[kMaxSplits];
 #pragma unroll
@@ -287,8 +290,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
         }
         if (sink) lt += ns_exp2(sink[h] * kLog2e - mt);
         float res = acc / lt;
-        if (gate) res *= 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)n * gate_stride + h])));
-        out[(size_t)n * o_stride + (size_t)h * dv + col] = __float2bfloat16_rn(res);
+        out[(size_t)n * o_stride + (size_t)h * dv_row + v0 + col] = __float2bfloat16_rn(res * gate_factor(og, n, h, h * dv_row + v0 + col));
     }
 }
 
@@ -297,7 +299,7 @@ int launch_decode_stages(const void* q, int q_stride, const void* k_cache, const
                   int table_stride, const int* token_req, const int* positions, const int* qo_indptr, void* out,
                   int o_stride, float* part_o, float* part_ml, int* counters, const int* rows, int n_tokens, int nq,
                   int nkv, int page_size, float scale, int window, int n_splits, cudaStream_t stream, int keep_first, int wide_weights,
-                  int mask_chunk, float softcap, int dk, int dv, const float* sink, const void* gate, int gate_stride) {
+                  int mask_chunk, float softcap, int dk, int dv, const ValueSlices& vs, const float* sink, const OutGate& og) {
     constexpr int S = NsTile<D>::kStride;
     const size_t tiles = (size_t)(16 + 2 * kStages * kTileKeys) * S * sizeof(__nv_bfloat16);
     const size_t scratch = (size_t)(4 * 16 * D + 128) * sizeof(float);  // the warps' partial results reuse the k/v stages
@@ -308,12 +310,11 @@ int launch_decode_stages(const void* q, int q_stride, const void* k_cache, const
         configured = true;
     }
     const int G = nq / nkv, head_tiles = (G + 15) / 16;
-    dim3 grid(n_splits, nkv * head_tiles, n_tokens);
+    dim3 grid(n_splits, nkv * head_tiles * vs.count, n_tokens);
     NS_LAUNCH((attention_decode_kernel<D, kStages>), grid, kThreads, smem, stream, 
         (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_table,
         table_stride, token_req, positions, qo_indptr, (__nv_bfloat16*)out, o_stride, part_o, part_ml, counters, rows, nq,
-        nkv, page_size, scale, window, n_splits, head_tiles, keep_first, wide_weights, mask_chunk, softcap, dk, dv, sink,
-        (const __nv_bfloat16*)gate, gate_stride);
+        nkv, page_size, scale, window, n_splits, head_tiles, keep_first, wide_weights, mask_chunk, softcap, dk, dv, vs.width, vs.count, sink, og);
     NS_CHECK_LAUNCH("ns_attention_decode");
     return NS_OK;
 }
@@ -325,14 +326,14 @@ int launch_decode(const void* q, int q_stride, const void* k_cache, const void* 
                   int table_stride, const int* token_req, const int* positions, const int* qo_indptr, void* out,
                   int o_stride, float* part_o, float* part_ml, int* counters, const int* rows, int n_tokens, int nq,
                   int nkv, int page_size, float scale, int window, int n_splits, cudaStream_t stream, int keep_first, int wide_weights,
-                  int mask_chunk, float softcap, int dk, int dv, const float* sink, const void* gate, int gate_stride) {
+                  int mask_chunk, float softcap, int dk, int dv, const ValueSlices& vs, const float* sink, const OutGate& og) {
     if (g_decode_stages == 2)
         return launch_decode_stages<D, 2>(q, q_stride, k_cache, v_cache, block_table, table_stride, token_req, positions,
                                           qo_indptr, out, o_stride, part_o, part_ml, counters, rows, n_tokens, nq, nkv,
-                                          page_size, scale, window, n_splits, stream, keep_first, wide_weights, mask_chunk, softcap, dk, dv, sink, gate, gate_stride);
+                                          page_size, scale, window, n_splits, stream, keep_first, wide_weights, mask_chunk, softcap, dk, dv, vs, sink, og);
     return launch_decode_stages<D, 3>(q, q_stride, k_cache, v_cache, block_table, table_stride, token_req, positions,
                                       qo_indptr, out, o_stride, part_o, part_ml, counters, rows, n_tokens, nq, nkv,
-                                      page_size, scale, window, n_splits, stream, keep_first, wide_weights, mask_chunk, softcap, dk, dv, sink, gate, gate_stride);
+                                      page_size, scale, window, n_splits, stream, keep_first, wide_weights, mask_chunk, softcap, dk, dv, vs, sink, og);
 }
 
 }  // namespace
@@ -364,22 +365,28 @@ NS_API int ns_attention_decode_scratch(int n_tokens, int nq, int nkv, int d, int
 // `dv` > 0: values of that many features where the keys have `d` (both multiples of 8 then; the output rows are nq * dv wide
 // and `part_o` holds as many columns per row as the instance that runs: the larger of d and dv rounded up to 16).
 // `sink` (optional, float [nq]): every query's denominator also holds exp(sink[h]), a term without key or value, counted once
-// however the keys are split.  `gate` (optional, bfloat16, gate[token * gate_stride + h]): head h's output times the sigmoid of its gate.
+// however the keys are split.  `gate` (optional, bfloat16, gate[token * gate_stride + h]): head h's output times the sigmoid of its gate;
+// with gate_per_feature every feature has its own, gate[token * gate_stride + h * dv + e].  `out_scale` multiplies every output.
+// Values of more than 128 features run in slices of `width` features, each with partial results (`instance` columns) and a counter of
+// its own (value_slices, attention_common.cuh).
 NS_API int ns_attention_decode_kept(const void* q, int q_stride, const void* k_cache, const void* v_cache,
                                     const int* block_table, int table_stride, const int* token_req, const int* positions,
                                     const int* qo_indptr, void* out, int o_stride, float* part_o, float* part_ml,
                                     int* counters, const int* rows, int n_tokens, int nq, int nkv, int d, int page_size,
                                     float scale, int window, int keep_first, int wide_weights, int mask_chunk, float softcap, int n_splits,
-                                    int dv, const float* sink, const void* gate, int gate_stride, cudaStream_t stream) {
+                                    int dv, const float* sink, const void* gate, int gate_stride, int gate_per_feature, float out_scale,
+                                    cudaStream_t stream) {
     if (n_tokens <= 0) return NS_OK;
     if (keep_first < 0 || window < 0) NS_FAIL(NS_ERR_ARGUMENT, "ns_attention_decode: window=%d keep_first=%d", window, keep_first);
     if (window == 0) keep_first = 0;
     if (mask_chunk < 0 || (mask_chunk > 0 && keep_first > 0))
         NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_decode: mask_chunk=%d with keep_first=%d", mask_chunk, keep_first);
     if (dv <= 0) dv = d;
-    const int dk = d, dmax = ((d > dv ? d : dv) + 15) / 16 * 16;  // dmax: the instance that runs
-    if (dv == d ? (d % 16 || d < 16 || d > 128) : (d % 8 || dv % 8 || d < 8 || dv < 8 || dmax > 128))
-        NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_decode: head_dim=%d, values of %d (equal: multiples of 16 up to 128; else of 8)", d, dv);
+    const int dk = d;
+    const ValueSlices vs = value_slices(d, dv);
+    const OutGate og{(const __nv_bfloat16*)gate, gate_stride, gate_per_feature, out_scale};
+    if (dv == d ? (d % 16 || d < 16 || d > 128) : (d % 8 || dv % 8 || d < 8 || dv < 8 || d > 128))
+        NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_decode: head_dim=%d, values of %d (equal: multiples of 16 up to 128; else of 8, keys up to 128)", d, dv);
     if (nkv < 1 || nq % nkv) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_decode: %d query heads over %d kv heads", nq, nkv);
     if (n_splits < 1 || n_splits > kMaxSplits) NS_FAIL(NS_ERR_ARGUMENT, "ns_attention_decode: n_splits=%d (1..%d)", n_splits, kMaxSplits);
     if (q_stride % 8 || ((uintptr_t)q % 16)) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_decode: q rows must be 16-byte aligned");
@@ -388,8 +395,8 @@ NS_API int ns_attention_decode_kept(const void* q, int q_stride, const void* k_c
     case DD:                                                                                                           \
         return launch_decode<DD>(q, q_stride, k_cache, v_cache, block_table, table_stride, token_req, positions,       \
                                  qo_indptr, out, o_stride, part_o, part_ml, counters, rows, n_tokens, nq, nkv,         \
-                                 page_size, scale, window, n_splits, stream, keep_first, wide_weights, mask_chunk, softcap, dk, dv, sink, gate, gate_stride);
-    switch (dmax) {
+                                 page_size, scale, window, n_splits, stream, keep_first, wide_weights, mask_chunk, softcap, dk, dv, vs, sink, og);
+    switch (vs.instance) {
         NS_DECODE_CASE(16) NS_DECODE_CASE(32) NS_DECODE_CASE(48) NS_DECODE_CASE(64)
         NS_DECODE_CASE(80) NS_DECODE_CASE(96) NS_DECODE_CASE(112) NS_DECODE_CASE(128)
     }
@@ -404,7 +411,7 @@ NS_API int ns_attention_decode(const void* q, int q_stride, const void* k_cache,
                                float scale, int window, int n_splits, cudaStream_t stream) {
     return ns_attention_decode_kept(q, q_stride, k_cache, v_cache, block_table, table_stride, token_req, positions, qo_indptr, out,
                                     o_stride, part_o, part_ml, counters, rows, n_tokens, nq, nkv, d, page_size, scale, window, 0, 0,
-                                    0, 0.f, n_splits, 0, nullptr, nullptr, 0, stream);
+                                    0, 0.f, n_splits, 0, nullptr, nullptr, 0, 0, 1.f, stream);
 }
 
 // ---------------------------------------------------------------------------------------

@@ -1,4 +1,4 @@
-// Attention over the paged cache, one warp per (token, query head), any head size up to 256.
+// Attention over the paged cache, one warp per (token, query head), any head size up to 512.
 //
 // This is the exact kernel: every score, the softmax and the weighted sum are fp32 with
 // accurate expf, and the keys of one query are always visited in the same order (ascending
@@ -28,7 +28,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
                          const int* __restrict__ token_req, const int* __restrict__ positions, T* __restrict__ out,
                          int o_stride, int n_tokens, int nq, int nkv, int d, int dv, int page_size, float scale, int window,
                          int keep_first, int chunk, float softcap, const float* __restrict__ sink,
-                         const T* __restrict__ gate, int gate_stride) {
+                         const T* __restrict__ gate, int gate_stride, int gate_per_feature, float out_scale) {
     ns_pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one before it reads
     ns_pdl_wait();               // everything below sees the previous kernel's results
     extern __shared__ float qsm[];
@@ -102,12 +102,13 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
 #pragma unroll
         for (int i = 0; i < DPL; ++i) acc[i] *= corr;
     }
-    float inv = 1.f / l;
-    if (gate) inv *= 1.f / (1.f + expf(-ns_ld(gate, (size_t)n * gate_stride + h)));  // the head's output gate
+    float inv = out_scale / l;
+    if (gate && !gate_per_feature) inv *= 1.f / (1.f + expf(-ns_ld(gate, (size_t)n * gate_stride + h)));  // the head's output gate
+    const T* fg = gate && gate_per_feature ? gate + (size_t)n * gate_stride + (size_t)h * dv : nullptr;  // ... or one per feature
 #pragma unroll
     for (int i = 0; i < DPL; ++i) {
         const int e = lane + 32 * i;
-        if (e < dv) ns_st(o, e, acc[i] * inv);
+        if (e < dv) ns_st(o, e, fg ? acc[i] * inv / (1.f + expf(-ns_ld(fg, e))) : acc[i] * inv);
     }
 }
 
@@ -115,21 +116,23 @@ template <typename T>
 int launch(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* block_table,
            int table_stride, const int* token_req, const int* positions, void* out, int o_stride, int n_tokens, int nq,
            int nkv, int d, int dv, int page_size, float scale, int window, int keep_first, int chunk, float softcap,
-           const float* sink, const void* gate, int gate_stride, cudaStream_t stream) {
+           const float* sink, const void* gate, int gate_stride, int gate_per_feature, float out_scale, cudaStream_t stream) {
     const long long warps = (long long)n_tokens * nq;
     const unsigned blocks = (unsigned)((warps + kWarpsPerBlock - 1) / kWarpsPerBlock);
     const size_t smem = (size_t)kWarpsPerBlock * d * sizeof(float);
-    const int dpl = (dv + 31) / 32;
+    int dpl = (dv + 31) / 32;
+    if (dpl > 8) dpl += dpl % 2;
 #define NS_ATTN_CASE(D)                                                                                              \
     case D:                                                                                                          \
         NS_LAUNCH((attention_generic_kernel<T, D>), blocks, kWarpsPerBlock * 32, smem, stream,                                \
             (const T*)q, q_stride, (const T*)k_cache, (const T*)v_cache, block_table, table_stride, token_req,       \
             positions, (T*)out, o_stride, n_tokens, nq, nkv, d, dv, page_size, scale, window, keep_first, chunk, softcap, \
-            sink, (const T*)gate, gate_stride);                                                                       \
+            sink, (const T*)gate, gate_stride, gate_per_feature, out_scale);                                                                    \
         break;
     switch (dpl) {
         NS_ATTN_CASE(1) NS_ATTN_CASE(2) NS_ATTN_CASE(3) NS_ATTN_CASE(4)
         NS_ATTN_CASE(5) NS_ATTN_CASE(6) NS_ATTN_CASE(7) NS_ATTN_CASE(8)
+        NS_ATTN_CASE(10) NS_ATTN_CASE(12) NS_ATTN_CASE(14) NS_ATTN_CASE(16)
     }
 #undef NS_ATTN_CASE
     NS_CHECK_LAUNCH("ns_attention_generic");
@@ -140,24 +143,25 @@ int launch(const void* q, int q_stride, const void* k_cache, const void* v_cache
 
 // `sink` (optional, float [nq]): every query's denominator also holds exp(sink[h]), a term without key or value (zeros: "one
 // added to the denominator").  `gate` (optional, the activations' type, one number per token and head at
-// gate[n * gate_stride + h]): head h's output is multiplied by its sigmoid.
+// gate[n * gate_stride + h]): head h's output is multiplied by its sigmoid; with gate_per_feature every feature has its own, at
+// gate[n * gate_stride + h * dv + e].  `out_scale` multiplies every output.
 NS_API int ns_attention_generic_sink(const void* q, int q_stride, const void* k_cache, const void* v_cache,
                                 const int* block_table, int table_stride, const int* token_req, const int* positions,
                                 void* out, int o_stride, int n_tokens, int nq, int nkv, int d, int dv, int page_size,
                                 float scale, int window, int keep_first, int chunk, float softcap, const float* sink,
-                                const void* gate, int gate_stride, int dtype, cudaStream_t stream) {
+                                const void* gate, int gate_stride, int gate_per_feature, float out_scale, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return NS_OK;
-    if (d < 1 || d > 256 || dv < 1 || dv > 256)
-        NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_generic: head sizes %d (keys) and %d (values) must lie in 1..256", d, dv);
+    if (d < 1 || d > 512 || dv < 1 || dv > 512)
+        NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_generic: head sizes %d (keys) and %d (values) must lie in 1..512", d, dv);
     if (keep_first < 0 || window < 0 || chunk < 0) NS_FAIL(NS_ERR_ARGUMENT, "ns_attention_generic: window=%d keep_first=%d chunk=%d", window, keep_first, chunk);
     if (chunk > 0 && keep_first > 0) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_generic: kept first keys and chunks do not go together");
     if (nkv < 1 || nq % nkv) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_generic: %d query heads over %d kv heads", nq, nkv);
     if (dtype == NS_F32)
         return launch<float>(q, q_stride, k_cache, v_cache, block_table, table_stride, token_req, positions, out,
-                             o_stride, n_tokens, nq, nkv, d, dv, page_size, scale, window, keep_first, chunk, softcap, sink, gate, gate_stride, stream);
+                             o_stride, n_tokens, nq, nkv, d, dv, page_size, scale, window, keep_first, chunk, softcap, sink, gate, gate_stride, gate_per_feature, out_scale, stream);
     if (dtype == NS_BF16)
         return launch<__nv_bfloat16>(q, q_stride, k_cache, v_cache, block_table, table_stride, token_req, positions,
-                                     out, o_stride, n_tokens, nq, nkv, d, dv, page_size, scale, window, keep_first, chunk, softcap, sink, gate, gate_stride, stream);
+                                     out, o_stride, n_tokens, nq, nkv, d, dv, page_size, scale, window, keep_first, chunk, softcap, sink, gate, gate_stride, gate_per_feature, out_scale, stream);
     NS_FAIL(NS_ERR_ARGUMENT, "ns_attention_generic: unknown dtype %d", dtype);
 }
 
@@ -167,5 +171,5 @@ NS_API int ns_attention_generic(const void* q, int q_stride, const void* k_cache
                                 float scale, int window, int keep_first, int chunk, float softcap, int dtype, cudaStream_t stream) {
     return ns_attention_generic_sink(q, q_stride, k_cache, v_cache, block_table, table_stride, token_req, positions, out, o_stride,
                                      n_tokens, nq, nkv, d, dv, page_size, scale, window, keep_first, chunk, softcap, nullptr, nullptr,
-                                     0, dtype, stream);
+                                     0, 0, 1.f, dtype, stream);
 }

@@ -31,7 +31,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
                          int table_stride, const int* __restrict__ positions, const int* __restrict__ qo_indptr,
                          const int* __restrict__ tiles, __nv_bfloat16* __restrict__ out, int o_stride, int nq, int nkv,
                          int page_size, float scale, int window, int keep_first, int wide_weights, int mask_chunk, float softcap,
-                         int dk, int dv, const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int gate_stride) {
+                         int dk, int dv_row, int dv_slice, const float* __restrict__ sink, const OutGate og) {
     ns_pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one before it reads
     ns_pdl_wait();               // everything below sees the previous kernel's results
     using Tile = NsTile<D>;
@@ -42,6 +42,9 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
 
     const int req = tiles[2 * blockIdx.x], q_off = tiles[2 * blockIdx.x + 1];
     const int h = blockIdx.y;
+    // the slice of the values' features that this block takes
+    const int v0 = blockIdx.z * dv_slice, dv = min(dv_slice, dv_row - v0);
+    v_cache += v0;
     const int hk = h / (nq / nkv);
     const int tok0 = qo_indptr[req] + q_off;
     const int rows = min(kTileQ, qo_indptr[req + 1] - tok0);  // valid query rows of this tile
@@ -67,7 +70,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
             ns_cp_async16(Tile::at(qs, row, ch * 8), qbase + (valid ? (size_t)row * q_stride + ch * 8 : 0), valid);
         }
     }
-    load_kv_tile<D, kPrefillThreads>(kv, kv + kTileKeys * S, k_cache, v_cache, bt, k_begin, kfirst, kend, hk, nkv, page_size, page_shift, win_first, gap, dk, dv);
+    load_kv_tile<D, kPrefillThreads>(kv, kv + kTileKeys * S, k_cache, v_cache, bt, k_begin, kfirst, kend, hk, nkv, page_size, page_shift, win_first, gap, dk, dv, dv_row);
     ns_cp_async_commit();
 
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
@@ -98,7 +101,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
         if (t + 1 < n_tiles) {
             __nv_bfloat16* kn = kv + (size_t)((t + 1) & 1) * 2 * kTileKeys * S;
             load_kv_tile<D, kPrefillThreads>(kn, kn + kTileKeys * S, k_cache, v_cache, bt, k_begin + (t + 1) * kTileKeys, kfirst, kend, hk,
-                            nkv, page_size, page_shift, win_first, gap, dk, dv);
+                            nkv, page_size, page_shift, win_first, gap, dk, dv, dv_row);
         }
         ns_cp_async_commit();
         ns_cp_async_wait<1>();
@@ -222,12 +225,20 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
         // a sink: exp(sink[h]) joins the denominator (m and the sums are in base 2); a gate: the head's output times its sigmoid
         if (sink) l[i] += ns_exp2(sink[h] * kLog2e - m[i]);
         float inv = 1.f / l[i];
-        if (gate) inv *= 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)(tok0 + row) * gate_stride + h])));
-        __nv_bfloat16* orow = out + (size_t)(tok0 + row) * o_stride + (size_t)h * dv;
+        if (!og.per_feature) inv *= gate_factor(og, tok0 + row, h, 0);
+        __nv_bfloat16* orow = out + (size_t)(tok0 + row) * o_stride + (size_t)h * dv_row + v0;
+        const __nv_bfloat16* grow = og.gate + (size_t)(tok0 + row) * og.stride + (size_t)h * dv_row + v0;
 #pragma unroll
         for (int nb = 0; nb < D / 8; ++nb) {
             const int col = nb * 8 + 2 * (lane & 3);
-            if (col < dv) *reinterpret_cast<__nv_bfloat162*>(orow + col) = __floats2bfloat162_rn(o[nb][2 * i] * inv, o[nb][2 * i + 1] * inv);
+            if (col >= dv) continue;
+            float y0 = o[nb][2 * i] * inv, y1 = o[nb][2 * i + 1] * inv;
+            if (og.per_feature) {
+                const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(grow + col));
+                y0 *= __fdividef(og.out_scale, 1.f + __expf(-z.x));
+                y1 *= __fdividef(og.out_scale, 1.f + __expf(-z.y));
+            }
+            *reinterpret_cast<__nv_bfloat162*>(orow + col) = __floats2bfloat162_rn(y0, y1);
         }
     }
 }
@@ -237,7 +248,7 @@ int launch_prefill(const void* q, int q_stride, const void* k_cache, const void*
                    int table_stride, const int* positions, const int* qo_indptr, const int* tiles, int n_tiles,
                    void* out, int o_stride, int nq, int nkv, int page_size, float scale, int window,
                    cudaStream_t stream, int keep_first, int wide_weights, int mask_chunk, float softcap, int dk, int dv,
-                   const float* sink, const void* gate, int gate_stride) {
+                   const ValueSlices& vs, const float* sink, const OutGate& og) {
     constexpr int S = NsTile<D>::kStride;
     const size_t smem = (size_t)(kTileQ + 4 * kTileKeys) * S * sizeof(__nv_bfloat16);
     static bool configured = false;
@@ -245,11 +256,11 @@ int launch_prefill(const void* q, int q_stride, const void* k_cache, const void*
         NS_CUDA(cudaFuncSetAttribute(attention_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         configured = true;
     }
-    dim3 grid(n_tiles, nq);
+    dim3 grid(n_tiles, nq, vs.count);
     NS_LAUNCH((attention_prefill_kernel<D>), grid, kPrefillThreads, smem, stream, 
         (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_table,
         table_stride, positions, qo_indptr, tiles, (__nv_bfloat16*)out, o_stride, nq, nkv, page_size, scale, window, keep_first, wide_weights,
-        mask_chunk, softcap, dk, dv, sink, (const __nv_bfloat16*)gate, gate_stride);
+        mask_chunk, softcap, dk, dv, vs.width, sink, og);
     NS_CHECK_LAUNCH("ns_attention_prefill");
     return NS_OK;
 }
@@ -263,31 +274,36 @@ int launch_prefill(const void* q, int q_stride, const void* k_cache, const void*
 // `mask_chunk`, `softcap`: see the top of the file (0: off); kept first keys and chunks do not go together.
 // `dv` > 0: values of that many features where the keys have `d` (both multiples of 8 then, the output rows nq * dv wide).
 // `sink` (optional, float [nq]): every query's denominator also holds exp(sink[h]), a term without key or value.
-// `gate` (optional, bfloat16, gate[token * gate_stride + h]): head h's output is multiplied by the sigmoid of its gate.
+// `gate` (optional, bfloat16, gate[token * gate_stride + h]): head h's output is multiplied by the sigmoid of its gate; with
+// gate_per_feature every feature has its own, gate[token * gate_stride + h * dv + e].  `out_scale` multiplies every output.
+// Values of more than 128 features run in slices (keys of at most 128).
 NS_API int ns_attention_prefill_kept(const void* q, int q_stride, const void* k_cache, const void* v_cache,
                                      const int* block_table, int table_stride, const int* positions, const int* qo_indptr,
                                      const int* tiles, int n_tiles, void* out, int o_stride, int nq, int nkv, int d,
                                      int page_size, float scale, int window, int keep_first, int wide_weights, int mask_chunk, float softcap,
-                                     int dv, const float* sink, const void* gate, int gate_stride, cudaStream_t stream) {
+                                     int dv, const float* sink, const void* gate, int gate_stride, int gate_per_feature, float out_scale,
+                                     cudaStream_t stream) {
     if (n_tiles <= 0) return NS_OK;
     if (keep_first < 0 || window < 0) NS_FAIL(NS_ERR_ARGUMENT, "ns_attention_prefill: window=%d keep_first=%d", window, keep_first);
     if (window == 0) keep_first = 0;
     if (mask_chunk < 0 || (mask_chunk > 0 && keep_first > 0))
         NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_prefill: mask_chunk=%d with keep_first=%d", mask_chunk, keep_first);
     if (dv <= 0) dv = d;
-    const int dmax = ((d > dv ? d : dv) + 15) / 16 * 16;  // the instance that runs
-    if (dv == d ? (d % 16 || d < 16 || d > 128) : (d % 8 || dv % 8 || d < 8 || dv < 8 || dmax > 128))
-        NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_prefill: head_dim=%d, values of %d (equal: multiples of 16 up to 128; else of 8)", d, dv);
+    const ValueSlices vs = value_slices(d, dv);
+    if (dv == d ? (d % 16 || d < 16 || d > 128) : (d % 8 || dv % 8 || d < 8 || dv < 8 || d > 128))
+        NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_prefill: head_dim=%d, values of %d (equal: multiples of 16 up to 128; else of 8, keys up to 128)", d, dv);
     if (nkv < 1 || nq % nkv) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_prefill: %d query heads over %d kv heads", nq, nkv);
     if (q_stride % 8 || ((uintptr_t)q % 16) || o_stride % 2)
         NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_prefill: q rows must be 16-byte aligned and out rows 4-byte aligned");
+    if (gate_per_feature && (gate_stride % 2 || (uintptr_t)gate % 4)) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_prefill: gate rows must be 4-byte aligned");
+    const OutGate og{(const __nv_bfloat16*)gate, gate_stride, gate ? gate_per_feature : 0, out_scale};
     if (nq > 65535) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_attention_prefill: %d heads exceed the grid's y extent", nq);
 #define NS_PREFILL_CASE(DD)                                                                                          \
     case DD:                                                                                                         \
         return launch_prefill<DD>(q, q_stride, k_cache, v_cache, block_table, table_stride, positions, qo_indptr,   \
                                   tiles, n_tiles, out, o_stride, nq, nkv, page_size, scale, window, stream, keep_first, wide_weights, \
-                                  mask_chunk, softcap, d, dv, sink, gate, gate_stride);
-    switch (dmax) {
+                                  mask_chunk, softcap, d, dv, vs, sink, og);
+    switch (vs.instance) {
         NS_PREFILL_CASE(16) NS_PREFILL_CASE(32) NS_PREFILL_CASE(48) NS_PREFILL_CASE(64)
         NS_PREFILL_CASE(80) NS_PREFILL_CASE(96) NS_PREFILL_CASE(112) NS_PREFILL_CASE(128)
     }
@@ -300,5 +316,5 @@ NS_API int ns_attention_prefill(const void* q, int q_stride, const void* k_cache
                                 const int* tiles, int n_tiles, void* out, int o_stride, int nq, int nkv, int d,
                                 int page_size, float scale, int window, cudaStream_t stream) {
     return ns_attention_prefill_kept(q, q_stride, k_cache, v_cache, block_table, table_stride, positions, qo_indptr, tiles, n_tiles,
-                                     out, o_stride, nq, nkv, d, page_size, scale, window, 0, 0, 0, 0.f, 0, nullptr, nullptr, 0, stream);
+                                     out, o_stride, nq, nkv, d, page_size, scale, window, 0, 0, 0, 0.f, 0, nullptr, nullptr, 0, 0, 1.f, stream);
 }

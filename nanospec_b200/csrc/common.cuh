@@ -69,6 +69,20 @@ __device__ __forceinline__ void st8(__nv_bfloat16* p, const float (&v)[8]) {
     *reinterpret_cast<uint4*>(p) = u;
 }
 
+// A gated unit's activation: with g held below `limit` and u within +-limit (limit 0: as they are),
+// g sigmoid(alpha g) (u + shift).  {1, 0, 0} is silu(g) * u.  FAST takes the hardware exponential and division (about 2 ulp in
+// float, far below the rounding of a bfloat16 result).
+struct NsGate { float alpha, shift, limit; };
+template <bool FAST>
+__device__ __forceinline__ float ns_gate_mul(const NsGate& a, float g, float u) {
+    if (a.limit > 0.f) {
+        g = fminf(g, a.limit);
+        u = fminf(fmaxf(u, -a.limit), a.limit);
+    }
+    const float s = FAST ? __fdividef(g, 1.f + __expf(-a.alpha * g)) : g / (1.f + expf(-a.alpha * g));
+    return s * (u + a.shift);
+}
+
 __device__ __forceinline__ float ns_warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -265,18 +265,13 @@ NS_API int ns_residual_add(float* resid, const void* branch, int n_rows, int hid
 }
 
 // ---------------------------------------------------------------------------------------
-// SwiGLU gate on the packed [gate | up] projection:
+// SwiGLU gate on the packed [gate | up] projection, and gated units of the same form (NsGate, common.cuh):
 //   out[n, j] = silu(gu[n, j]) * gu[n, inter + j],  silu(a) = a / (1 + exp(-a)),  in float
 // ---------------------------------------------------------------------------------------
-// silu(g) * u.  The float kernels use the accurate exponential and division; the bfloat16 ones the
-// hardware approximations (about 2 ulp in float, far below the rounding of the result).
-template <typename T>
-__device__ __forceinline__ float silu_mul(float g, float u) { return (g / (1.f + expf(-g))) * u; }
-template <>
-__device__ __forceinline__ float silu_mul<__nv_bfloat16>(float g, float u) { return __fdividef(g, 1.f + __expf(-g)) * u; }
+// The float kernels use the accurate exponential and division; the bfloat16 ones the hardware approximations.
 
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, long long ldg, T* __restrict__ out, long long ldo, int inter, int block, size_t total) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, long long ldg, T* __restrict__ out, long long ldo, int inter, int block, size_t total, NsGate act) {
     ns_pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one before it reads
     ns_pdl_wait();               // everything below sees the previous kernel's results
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -287,11 +282,11 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, long long ldg, T* __rest
     const size_t gi = block ? (size_t)(j / block) * 2 * block + j % block : (size_t)j;
     const float g = ns_ld(gu, n * ldg + gi);
     const float u = ns_ld(gu, n * ldg + gi + (block ? block : inter));
-    ns_st(out, n * ldo + j, silu_mul<T>(g, u));
+    ns_st(out, n * ldo + j, ns_gate_mul<sizeof(T) == 2>(act, g, u));
 }
 
 template <typename T>
-__global__ void swiglu_vec_kernel(const T* __restrict__ gu, long long ldg, T* __restrict__ out, long long ldo, int inter, int block, size_t total8) {
+__global__ void swiglu_vec_kernel(const T* __restrict__ gu, long long ldg, T* __restrict__ out, long long ldo, int inter, int block, size_t total8, NsGate act) {
     ns_pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one before it reads
     ns_pdl_wait();               // everything below sees the previous kernel's results
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -304,15 +299,16 @@ __global__ void swiglu_vec_kernel(const T* __restrict__ gu, long long ldg, T* __
     ld8(gu + n * ldg + gi, g);
     ld8(gu + n * ldg + gi + (block ? block : inter), u);
 #pragma unroll
-    for (int k = 0; k < 8; ++k) y[k] = silu_mul<T>(g[k], u[k]);
+    for (int k = 0; k < 8; ++k) y[k] = ns_gate_mul<sizeof(T) == 2>(act, g[k], u[k]);
     st8(out + n * ldo + j, y);
 }
 
 // out[n, j] = silu(g) * u with g, u = gate_up[n, j], gate_up[n, inter + j] (block == 0), or, when gate and up
 // alternate in runs of `block` features (a multiple of 8 that divides inter), gate_up[n, (j / block) * 2 * block +
-// j % block] and the element `block` further.  Rows of gate_up start ldg elements apart, rows of out ldo.
-NS_API int ns_swiglu_rows(const void* gate_up, long long ldg, void* out, long long ldo, int n_rows, int inter, int block, int dtype,
-                          cudaStream_t stream) {
+// j % block] and the element `block` further.  Rows of gate_up start ldg elements apart, rows of out ldo.  alpha, shift, limit: NsGate.
+NS_API int ns_gate_mul_rows(const void* gate_up, long long ldg, void* out, long long ldo, int n_rows, int inter, int block, float alpha, float shift,
+                            float limit, int dtype, cudaStream_t stream) {
+    const NsGate act{alpha, shift, limit};
     const size_t total = (size_t)n_rows * inter;
     if (total == 0) return NS_OK;
     if (block < 0 || (block && (block % 8 || inter % block)))
@@ -323,18 +319,24 @@ NS_API int ns_swiglu_rows(const void* gate_up, long long ldg, void* out, long lo
         const size_t total8 = total / 8;
         const unsigned vblocks = (unsigned)((total8 + 255) / 256);
         if (dtype == NS_F32)
-            NS_LAUNCH((swiglu_vec_kernel<float>), vblocks, 256, 0, stream, (const float*)gate_up, ldg, (float*)out, ldo, inter, block, total8);
+            NS_LAUNCH((swiglu_vec_kernel<float>), vblocks, 256, 0, stream, (const float*)gate_up, ldg, (float*)out, ldo, inter, block, total8, act);
         else
-            NS_LAUNCH((swiglu_vec_kernel<__nv_bfloat16>), vblocks, 256, 0, stream, (const __nv_bfloat16*)gate_up, ldg, (__nv_bfloat16*)out, ldo, inter, block, total8);
+            NS_LAUNCH((swiglu_vec_kernel<__nv_bfloat16>), vblocks, 256, 0, stream, (const __nv_bfloat16*)gate_up, ldg, (__nv_bfloat16*)out, ldo, inter, block, total8, act);
     } else {
         const unsigned blocks = (unsigned)((total + 255) / 256);
         if (dtype == NS_F32)
-            NS_LAUNCH((swiglu_kernel<float>), blocks, 256, 0, stream, (const float*)gate_up, ldg, (float*)out, ldo, inter, block, total);
+            NS_LAUNCH((swiglu_kernel<float>), blocks, 256, 0, stream, (const float*)gate_up, ldg, (float*)out, ldo, inter, block, total, act);
         else
-            NS_LAUNCH((swiglu_kernel<__nv_bfloat16>), blocks, 256, 0, stream, (const __nv_bfloat16*)gate_up, ldg, (__nv_bfloat16*)out, ldo, inter, block, total);
+            NS_LAUNCH((swiglu_kernel<__nv_bfloat16>), blocks, 256, 0, stream, (const __nv_bfloat16*)gate_up, ldg, (__nv_bfloat16*)out, ldo, inter, block, total, act);
     }
     NS_CHECK_LAUNCH("ns_swiglu");
     return NS_OK;
+}
+
+// silu(gate) * up
+NS_API int ns_swiglu_rows(const void* gate_up, long long ldg, void* out, long long ldo, int n_rows, int inter, int block, int dtype,
+                          cudaStream_t stream) {
+    return ns_gate_mul_rows(gate_up, ldg, out, ldo, n_rows, inter, block, 1.f, 0.f, 0.f, dtype, stream);
 }
 
 // the same over contiguous rows
@@ -529,4 +531,110 @@ NS_API int ns_add_dyt(float* resid, const void* a, const void* b, const float* g
     if (dtype == NS_F32) return launch_add_dyt<float>(resid, a, b, gain, bias, alpha, out, rows, n_rows, hidden, write_resid, stream);
     if (dtype == NS_BF16) return launch_add_dyt<__nv_bfloat16>(resid, a, b, gain, bias, alpha, out, rows, n_rows, hidden, write_resid, stream);
     NS_FAIL(NS_ERR_ARGUMENT, "ns_add_dyt: unknown dtype %d", dtype);
+}
+
+// ---------------------------------------------------------------------------------------
+// The same norm on what a sublayer returns, joined to the stream, and the next sublayer's norm after it, in one pass:
+//   y = a + b + sum_k weights[row, k] * ys[row_of[row, k]]      each optional; the last term is a routed sum (see moe.cu)
+//   x = resid + tanh(post.alpha y) post.gain + post.bias        written back unless rows are selected
+//   out = tanh(alpha x) gain + bias                              skipped without `out`
+// All in float; y is never rounded.  One thread takes eight neighbouring features where the rows start on 16 bytes.
+// ---------------------------------------------------------------------------------------
+namespace {
+
+struct TanhNorm { const float *gain, *bias, *alpha; };
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+dyt_join_kernel(float* __restrict__ resid, const T* __restrict__ a, const T* __restrict__ b, const T* __restrict__ ys,
+                const int* __restrict__ row_of, const float* __restrict__ weights, int top, const TanhNorm post, const TanhNorm next,
+                T* __restrict__ out, const int* __restrict__ rows, int hidden, int write_resid) {
+    ns_pdl_launch_dependents();
+    const int e0 = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+    ns_pdl_wait();
+    if (e0 >= hidden) return;
+    const int r = blockIdx.x;
+    const size_t row = rows ? rows[r] : r, src = row * hidden + e0;
+    float y[VEC], t[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) y[i] = 0.f;
+    auto load = [&](const auto* p, float (&v)[VEC]) {
+        if constexpr (VEC == 8) ld8(p, v);
+        else v[0] = ns_ld(p, 0);
+    };
+    auto store = [&](auto* p, const float (&v)[VEC]) {
+        if constexpr (VEC == 8) st8(p, v);
+        else ns_st(p, 0, v[0]);
+    };
+    if (ys) {
+        for (int k = 0; k < top; ++k) {
+            const int at = row_of[row * top + k];
+            const float w = weights[row * top + k];
+            load(ys + (size_t)at * hidden + e0, t);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) y[i] = fmaf(w, t[i], y[i]);
+        }
+    }
+    if (a) {
+        load(a + src, t);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y[i] += t[i];
+    }
+    if (b) {
+        load(b + src, t);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y[i] += t[i];
+    }
+    auto norm = [&](const TanhNorm& n, float (&v)[VEC]) {
+        float g[VEC];
+        const float al = *n.alpha;
+        load(n.gain + e0, g);
+        if (n.bias) load(n.bias + e0, t);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = fmaf(tanhf(al * v[i]), g[i], n.bias ? t[i] : 0.f);
+    };
+    norm(post, y);
+    load(resid + src, t);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) y[i] += t[i];
+    if (write_resid) store(resid + src, y);
+    if (!out) return;
+    norm(next, y);
+    store(out + (size_t)r * hidden + e0, y);
+}
+
+template <typename T>
+int launch_dyt_join(float* resid, const void* a, const void* b, const void* ys, const int* row_of, const float* weights, int top,
+                    const TanhNorm& post, const TanhNorm& next, void* out, const int* rows, int n_rows, int hidden, int write_resid,
+                    cudaStream_t stream) {
+    const uintptr_t all = (uintptr_t)resid | (uintptr_t)a | (uintptr_t)b | (uintptr_t)ys | (uintptr_t)post.gain | (uintptr_t)post.bias |
+                          (uintptr_t)next.gain | (uintptr_t)next.bias | (uintptr_t)out;
+    const bool vec = hidden % 8 == 0 && all % 16 == 0;
+    const int per = vec ? 8 : 1;
+    const int threads = hidden / per >= 256 ? 256 : hidden / per > 64 ? 128 : 64;
+    const unsigned bx = (unsigned)((hidden + threads * per - 1) / (threads * per));
+    if (vec)
+        NS_LAUNCH((dyt_join_kernel<T, 8>), dim3(n_rows, bx), threads, 0, stream, resid, (const T*)a, (const T*)b, (const T*)ys, row_of, weights,
+                  top, post, next, (T*)out, rows, hidden, write_resid);
+    else
+        NS_LAUNCH((dyt_join_kernel<T, 1>), dim3(n_rows, bx), threads, 0, stream, resid, (const T*)a, (const T*)b, (const T*)ys, row_of, weights,
+                  top, post, next, (T*)out, rows, hidden, write_resid);
+    NS_CHECK_LAUNCH("ns_dyt_join");
+    return NS_OK;
+}
+
+}  // namespace
+
+// a, b [n, hidden] and ys [pairs, hidden] in the compute type (row_of, weights [n, top] with ys; every row_of entry >= 0); out may be null.
+NS_API int ns_dyt_join(float* resid, const void* a, const void* b, const void* ys, const int* row_of, const float* weights, int top,
+                       const float* post_gain, const float* post_bias, const float* post_alpha, const float* gain, const float* bias,
+                       const float* alpha, void* out, const int* rows, int n_rows, int hidden, int write_resid, int dtype, cudaStream_t stream) {
+    if (n_rows <= 0) return NS_OK;
+    if (hidden <= 0 || !post_gain || !post_alpha || (out && (!gain || !alpha))) NS_FAIL(NS_ERR_ARGUMENT, "ns_dyt_join: hidden=%d, gains and alphas are needed", hidden);
+    if (ys && (!row_of || !weights || top < 1)) NS_FAIL(NS_ERR_ARGUMENT, "ns_dyt_join: a routed sum needs its rows and weights");
+    if (rows && write_resid) NS_FAIL(NS_ERR_ARGUMENT, "ns_dyt_join: a row selection cannot write the stream back");
+    const TanhNorm post{post_gain, post_bias, post_alpha}, next{gain, bias, alpha};
+    if (dtype == NS_F32) return launch_dyt_join<float>(resid, a, b, ys, row_of, weights, top, post, next, out, rows, n_rows, hidden, write_resid, stream);
+    if (dtype == NS_BF16) return launch_dyt_join<__nv_bfloat16>(resid, a, b, ys, row_of, weights, top, post, next, out, rows, n_rows, hidden, write_resid, stream);
+    NS_FAIL(NS_ERR_ARGUMENT, "ns_dyt_join: unknown dtype %d", dtype);
 }

@@ -48,7 +48,8 @@ constexpr int kMaxSplits = 8;
 
 // What the epilogue does besides storing the product (all pointers null: nothing).
 struct GemmEpilogue {
-    int gated;                    // silu(gate) * up on alternating runs of 64 features
+    int gated;                    // the gated unit on alternating runs of 64 gate and 64 up features
+    NsGate act;
     // scale: out rows *= rsqrt(sum_p row_partials[token, p] / hidden + eps)
     const float* row_partials;    // [tokens, n_partials]
     int n_partials;
@@ -63,6 +64,11 @@ struct GemmEpilogue {
     // complete as it is (no partials, and the product that reads it applies no scale)
     const float* sink_bias;       // [features] or null
     const float* sink_alpha;      // one float in device memory; null: the RMS form above
+    // ... and, with post_alpha given, the product itself passes such a norm before it joins the stream:
+    // resid += tanh(post_alpha * product) * post_gain + post_bias
+    const float* post_gain;
+    const float* post_bias;
+    const float* post_alpha;
     // rope: the product is an attention layer's packed [q | k | v] projection.  q and k are rotated by the
     // token's position (pairs (j, j + head_dim / 2)); q goes to `out`, k and v to the token's slot of the cache
     // [page, kv head, offset, head_dim].  Tiles of 128 features hold whole heads (head_dim 32, 64 or 128).
@@ -456,6 +462,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                     acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
                 }
                 if (kNorm && sink) {
+                    if (ep.post_alpha) {
+                        const float pa = __ldg(ep.post_alpha);
+                        float pg[4], pb[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                        for (int c = 0; c < 4; ++c) {
+                            pg[c] = __ldg(ep.post_gain + n0 + i + c);
+                            if (ep.post_bias) pb[c] = __ldg(ep.post_bias + n0 + i + c);
+                        }
+                        acc = make_float4(fmaf(tanhf(pa * acc.x), pg[0], pb[0]), fmaf(tanhf(pa * acc.y), pg[1], pb[1]),
+                                          fmaf(tanhf(pa * acc.z), pg[2], pb[2]), fmaf(tanhf(pa * acc.w), pg[3], pb[3]));
+                    }
                     res.x += acc.x; res.y += acc.y; res.z += acc.z; res.w += acc.w;
                     *reinterpret_cast<float4*>(ep.sink_resid + so) = res;
                     if (sink_tanh) {
@@ -525,10 +542,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                     const float inv = inv_s[j];
                     gs.x *= inv; gs.y *= inv; us.x *= inv; us.y *= inv;
                 }
-                // silu(gate) * up; the hardware exponential and division (about 2 ulp in float) are far below the
-                // rounding of the result
-                const float r0 = __fdividef(gs.x, 1.f + __expf(-gs.x)) * us.x;
-                const float r1 = __fdividef(gs.y, 1.f + __expf(-gs.y)) * us.y;
+                const float r0 = ns_gate_mul<true>(ep.act, gs.x, us.x), r1 = ns_gate_mul<true>(ep.act, gs.y, us.y);
                 OutT* dst = out + (size_t)(tok0 + j) * ldo + o0 + i;
                 if (2 * (o0 + i + 1) < N_feat && (reinterpret_cast<uintptr_t>(dst) % (2 * sizeof(OutT))) == 0) {
                     store_out2(dst, r0, r1);
@@ -649,12 +663,18 @@ NS_API int ns_gemm_bf16_tc(const void* x, const void* w, void* out, int M_tok, i
 
 // The gated feed-forward's first half in one kernel: w[N_feat, K] holds, for every run of 64 outputs, 64 gate
 // rows followed by the 64 matching up rows (N_feat a multiple of 128);
-// out[M_tok, N_feat / 2] = silu(x * gate^T) * (x * up^T), the sums and the activation in fp32.
-NS_API int ns_gemm_bf16_tc_gated(const void* x, const void* w, void* out, int M_tok, int N_feat, int K, int ldx, int ldw,
-                                 int ldo, int out_f32, int splits, int* error_flag, cudaStream_t stream) {
+// out[M_tok, N_feat / 2] = silu(x * gate^T) * (x * up^T), the sums and the activation in fp32; alpha, shift, limit: NsGate ({1, 0, 0} is that).
+NS_API int ns_gemm_bf16_tc_unit(const void* x, const void* w, void* out, int M_tok, int N_feat, int K, int ldx, int ldw,
+                                int ldo, int out_f32, int splits, float alpha, float shift, float limit, int* error_flag, cudaStream_t stream) {
     GemmEpilogue ep = {};
     ep.gated = 1;
+    ep.act = {alpha, shift, limit};
     return gemm_tc_host(x, w, out, M_tok, N_feat, K, ldx, ldw, ldo, out_f32, splits, ep, error_flag, stream);
+}
+
+NS_API int ns_gemm_bf16_tc_gated(const void* x, const void* w, void* out, int M_tok, int N_feat, int K, int ldx, int ldw,
+                                 int ldo, int out_f32, int splits, int* error_flag, cudaStream_t stream) {
+    return ns_gemm_bf16_tc_unit(x, w, out, M_tok, N_feat, K, ldx, ldw, ldo, out_f32, splits, 1.f, 0.f, 0.f, error_flag, stream);
 }
 
 // The same products with the norm epilogues (64 tokens at most).
@@ -669,6 +689,7 @@ NS_API int ns_gemm_bf16_tc_norm(const void* x, const void* w, void* out, int M_t
                                 float* sink_partials, int sink_ld, int* error_flag, cudaStream_t stream) {
     GemmEpilogue ep = {};
     ep.gated = gated;
+    ep.act = {1.f, 0.f, 0.f};
     ep.row_partials = row_partials;
     ep.n_partials = n_partials;
     ep.inv_hidden = hidden > 0 ? 1.f / (float)hidden : 0.f;
@@ -683,16 +704,22 @@ NS_API int ns_gemm_bf16_tc_norm(const void* x, const void* w, void* out, int M_t
 
 // A product whose output joins the residual stream and is followed by a norm that takes no statistics (64 tokens at most):
 // resid [M_tok, sink_ld] += product; sink_x [M_tok, sink_ld] = bf16(tanh(alpha * resid) * gain + bias).  `alpha` points at one
-// float in device memory; `bias` may be null.
+// float in device memory; `bias` may be null.  With post_gain and post_alpha (post_bias may be null) the product passes a norm of that
+// kind of its own first: resid += tanh(post_alpha * product) * post_gain + post_bias.
 NS_API int ns_gemm_bf16_tc_dyt(const void* x, const void* w, int M_tok, int N_feat, int K, int ldx, int ldw, int splits,
                                float* sink_resid, const float* sink_gain, const float* sink_bias, const float* sink_alpha,
+                               const float* post_gain, const float* post_bias, const float* post_alpha,
                                void* sink_x, int sink_ld, int* error_flag, cudaStream_t stream) {
+    if (!post_alpha != !post_gain) NS_FAIL(NS_ERR_ARGUMENT, "ns_gemm_bf16_tc_dyt: a norm of the product takes a gain and alpha");
     if (!sink_resid || !sink_gain || !sink_alpha || !sink_x) NS_FAIL(NS_ERR_ARGUMENT, "ns_gemm_bf16_tc_dyt: the stream, the gain, alpha and the output are needed");
     GemmEpilogue ep = {};
     ep.sink_resid = sink_resid;
     ep.sink_gain = sink_gain;
     ep.sink_bias = sink_bias;
     ep.sink_alpha = sink_alpha;
+    ep.post_gain = post_gain;
+    ep.post_bias = post_bias;
+    ep.post_alpha = post_alpha;
     ep.sink_x = (__nv_bfloat16*)sink_x;
     ep.sink_ld = sink_ld;
     return gemm_tc_host(x, w, nullptr, M_tok, N_feat, K, ldx, ldw, 0, 0, splits, ep, error_flag, stream);

@@ -2,11 +2,12 @@
 // the experts' products for steps of a few tokens.
 //
 //   ns_cast_f32        rows of the compute type as float (the router's input: its logits are a float product)
-//   ns_router_logits   the router's float product (the largest steps and routers: ns_cast_f32 and the float GEMM)
+//   ns_router_logits   the router's float product with an optional bias (the largest steps and routers: ns_cast_f32 and the float GEMM)
 //   ns_moe_route       scores = sigmoid(logits) (or softmax); consecutive experts form `groups` groups of equal size, ranked by
 //                      the top-2 sum of their scores; all but the `keep` highest-ranked groups are barred; then the `top`
 //                      highest-scoring experts that are not barred; weights = score / (sum of the chosen + 1e-20) * scale,
-//                      or score * scale.  An optional correction per expert is added to the scores that choose (groups
+//                      or score * scale; or the logits rank and choose, and the weights are their softmax over the chosen alone,
+//                      times scale.  An optional correction per expert is added to the scores that choose (groups
 //                      and experts) and not to the weights.  Ties go to the lower index.
 //   ns_moe_plan        counts per expert, their running offsets, and for every (token, choice) its row in the
 //                      order that has each expert's tokens side by side; a choice beyond the experts that have weights (an
@@ -35,12 +36,12 @@ __global__ void cast_f32_kernel(const T* __restrict__ x, long long ldx, float* _
 
 constexpr int kMaxExperts = 1024;
 
-// logits[n, e] = x[n] . w[e] in float: a block takes TOK tokens (their rows in shared memory) and eight experts, a warp per expert,
+// logits[n, e] = x[n] . w[e] (+ bias[e]) in float: a block takes TOK tokens (their rows in shared memory) and eight experts, a warp per expert,
 // so a row of w is read once for TOK tokens.  The sum over a row runs in the same order whatever TOK is.
 template <typename T, int TOK>
 __global__ void __launch_bounds__(256)
-router_logits_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, float* __restrict__ logits, int n_tokens, int E,
-                     int K) {
+router_logits_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                     float* __restrict__ logits, int n_tokens, int E, int K) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     extern __shared__ __align__(16) float xrow[];  // [TOK][K4]
@@ -87,7 +88,7 @@ router_logits_kernel(const T* __restrict__ x, long long ldx, const float* __rest
     }
 #pragma unroll
     for (int t = 0; t < TOK; ++t) {
-        const float v = ns_warp_sum(a[t]);
+        const float v = ns_warp_sum(a[t]) + (bias ? bias[e] : 0.f);
         if (lane == 0 && t < cnt) logits[(size_t)(n0 + t) * E + e] = v;
     }
 }
@@ -95,7 +96,7 @@ router_logits_kernel(const T* __restrict__ x, long long ldx, const float* __rest
 struct RouteRule {
     int E, groups, keep, top;
     float scale;
-    int softmax;
+    int softmax;  // 0: sigmoid scores, 1: a softmax over all, 2: a softmax over the chosen alone (the logits choose)
     const float* correction;
     int renormalize;
 };
@@ -116,12 +117,14 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, const R
             sc[e] = v;
             sum += v;
         }
-        sum = ns_warp_sum(sum);
-        for (int e = lane; e < E; e += 32) sc[e] /= sum;
+        if (r.softmax == 1) {
+            sum = ns_warp_sum(sum);
+            for (int e = lane; e < E; e += 32) sc[e] /= sum;
+        }
     } else {
         for (int e = lane; e < E; e += 32) sc[e] = 1.f / (1.f + expf(-z[e]));
     }
-    for (int e = lane; e < E; e += 32) cs[e] = sc[e] + (r.correction ? r.correction[e] : 0.f);
+    for (int e = lane; e < E; e += 32) cs[e] = (r.softmax == 2 ? z[e] : sc[e]) + (r.correction ? r.correction[e] : 0.f);
     __syncwarp();
     const float taken = -INFINITY;  // a taken or barred entry
     if (groups > 1) {
@@ -180,7 +183,8 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, const R
         if (lane == 0) cs[bi] = taken;
         __syncwarp();
     }
-    const float f = r.renormalize ? r.scale / (total + 1e-20f) : r.scale;
+    // (a softmax over the chosen: the largest logit is among them, so the total is 1 or more)
+    const float f = r.renormalize || r.softmax == 2 ? r.scale / (total + 1e-20f) : r.scale;
     if (lane < top && lane < 32) {
         ids[lane] = mine_id;
         weights[lane] = mine * f;
@@ -349,11 +353,11 @@ __device__ __forceinline__ float dot_row(const T* __restrict__ w, const float* _
     return ns_warp_sum(a);
 }
 
-// act[pair, j] = silu(gate_e[j] . x) * (up_e[j] . x); grid (pairs, feature chunks), a warp per feature
+// act[pair, j] = silu(gate_e[j] . x) * (up_e[j] . x), or another unit of that form; grid (pairs, feature chunks), a warp per feature
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_gate_up_rows_kernel(const T* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ w_gate,
-                        const T* __restrict__ w_up, T* __restrict__ act, int E, int top, int width, int ff, int per_block) {
+                        const T* __restrict__ w_up, T* __restrict__ act, int E, int top, int width, int ff, int per_block, NsGate unit) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     extern __shared__ float xs[];
@@ -369,7 +373,7 @@ moe_gate_up_rows_kernel(const T* __restrict__ x, const int* __restrict__ ids, co
         const size_t off = ((size_t)e * ff + j) * width;
         const float g = dot_row(w_gate + off, xs, width, lane, vec);
         const float u = dot_row(w_up + off, xs, width, lane, vec);
-        if (lane == 0) ns_st(act, (size_t)pair * ff + j, g / (1.f + expf(-g)) * u);
+        if (lane == 0) ns_st(act, (size_t)pair * ff + j, ns_gate_mul<false>(unit, g, u));
     }
 }
 
@@ -473,8 +477,8 @@ NS_API int ns_cast_f32(const void* x, long long ldx, float* out, int n_rows, int
     return NS_OK;
 }
 
-// x [n, K] (row stride ldx) in the compute type, w [E, K] float, logits [n, E] float
-NS_API int ns_router_logits(const void* x, long long ldx, const float* w, float* logits, int n_tokens, int E, int K, int dtype,
+// x [n, K] (row stride ldx) in the compute type, w [E, K] and bias [E] (or null) float, logits [n, E] float
+NS_API int ns_router_logits(const void* x, long long ldx, const float* w, const float* bias, float* logits, int n_tokens, int E, int K, int dtype,
                             cudaStream_t stream) {
     if (n_tokens <= 0) return NS_OK;
     const size_t row = (size_t)(K + 3) / 4 * 4 * sizeof(float);
@@ -488,7 +492,7 @@ NS_API int ns_router_logits(const void* x, long long ldx, const float* w, float*
 #define NS_ROUTER(T, TK)                                                                                                              \
     {                                                                                                                                 \
         if (smem > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(router_logits_kernel<T, TK>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
-        NS_LAUNCH((router_logits_kernel<T, TK>), grid, 256, smem, stream, (const T*)x, ldx, w, logits, n_tokens, E, K);               \
+        NS_LAUNCH((router_logits_kernel<T, TK>), grid, 256, smem, stream, (const T*)x, ldx, w, bias, logits, n_tokens, E, K);         \
     }
 #define NS_ROUTER_T(T) { if (tok == 1) NS_ROUTER(T, 1) else if (tok == 2) NS_ROUTER(T, 2) else if (tok == 4) NS_ROUTER(T, 4) else NS_ROUTER(T, 8) }
     if (dtype == NS_F32) NS_ROUTER_T(float)
@@ -582,10 +586,11 @@ NS_API int ns_moe_combine(const void* ys, const int* row_of, const float* weight
 }
 
 // x [n, width]; ids, weights [n, top]; w_gate, w_up [E, ff, width]; w_down [E, width, ff]; act [n * top, ff] scratch;
-// out [n, width]; ids from n_experts on return their input
+// out [n, width]; ids from n_experts on return their input; alpha, shift, limit: NsGate
 NS_API int ns_moe_expert_rows(const void* x, const int* ids, const float* weights, const void* w_gate, const void* w_up,
                               const void* w_down, void* act, void* out, int n_experts, int n_tokens, int top, int width,
-                              int ff, int dtype, cudaStream_t stream) {
+                              int ff, float alpha, float shift, float limit, int dtype, cudaStream_t stream) {
+    const NsGate unit{alpha, shift, limit};
     if (n_tokens <= 0) return NS_OK;
     const size_t smem_a = (size_t)width * sizeof(float), smem_b = (size_t)top * ff * sizeof(float);
     if (smem_a > 200 * 1024 || smem_b > 200 * 1024)
@@ -597,7 +602,7 @@ NS_API int ns_moe_expert_rows(const void* x, const int* ids, const float* weight
         if (smem_a > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(moe_gate_up_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
         if (smem_b > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(moe_down_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));    \
         NS_LAUNCH((moe_gate_up_rows_kernel<T>), grid_a, 256, smem_a, stream, (const T*)x, ids, (const T*)w_gate, (const T*)w_up,      \
-                  (T*)act, n_experts, top, width, ff, per_a);                                                                            \
+                  (T*)act, n_experts, top, width, ff, per_a, unit);                                                                          \
         NS_CHECK_LAUNCH("ns_moe_expert_rows");                                                                                \
         NS_LAUNCH((moe_down_rows_kernel<T>), grid_b, 256, smem_b, stream, (const T*)act, ids, weights, (const T*)w_down, (const T*)x, (T*)out,     \
                   n_experts, top, width, ff, per_b);                                                                                     \

@@ -6,6 +6,7 @@
 // two m16n8k16 row tiles) with its slice of the expert's weights, which stream through shared memory in chunks of 64
 // along k, double-buffered with cp.async.  Two products:
 //   gated   act[row, f] = silu(x[token(row)] . gate_e[f]) * (x[token(row)] . up_e[f])      64 features a block, A rows gathered
+//           (or another gated unit of that form: NsGate)
 //   plain   y[row, i]   = act[row] . down_e[i]                                                128 features a block
 // Each weight is read once per 32 rows of its expert, so a decode step of many requests reads every chosen expert once
 // instead of once per (token, choice).  bfloat16, k a multiple of 8.
@@ -20,7 +21,7 @@ template <bool GATED, int MT>
 __global__ void __launch_bounds__(128)
 moe_grouped_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const int* __restrict__ pair_of, int top,
                    const int* __restrict__ offsets, const __nv_bfloat16* __restrict__ w_a, const __nv_bfloat16* __restrict__ w_b,
-                   __nv_bfloat16* __restrict__ out, long long ldo, int F, int K) {
+                   __nv_bfloat16* __restrict__ out, long long ldo, int F, int K, NsGate act) {
     ns_pdl_launch_dependents();
     ns_pdl_wait();
     constexpr int kTileM = 16 * MT;
@@ -123,7 +124,7 @@ moe_grouped_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const int
                         const int f = f0 + 16 * warp + 8 * j + (lane & 3) * 2;
                         const float g0 = acc[mt][j][half * 2], g1 = acc[mt][j][half * 2 + 1];
                         const float u0 = acc[mt][j + 2][half * 2], u1 = acc[mt][j + 2][half * 2 + 1];
-                        const float v0 = g0 / (1.f + __expf(-g0)) * u0, v1 = g1 / (1.f + __expf(-g1)) * u1;
+                        const float v0 = ns_gate_mul<true>(act, g0, u0), v1 = ns_gate_mul<true>(act, g1, u1);
                         if (f + 1 < F) *reinterpret_cast<uint32_t*>(orow + f) = ns_pack_bf16(v0, v1);
                         else if (f < F) orow[f] = __float2bfloat16_rn(v0);
                     }
@@ -147,7 +148,8 @@ moe_grouped_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const int
 // rows_per_expert: the step's pairs over the experts (the host's guess of how many rows an expert holds).
 NS_API int ns_moe_grouped(const void* x, const int* pair_of, const int* offsets, const void* w_gate, const void* w_up,
                           const void* w_down, void* act, void* ys, int n_experts, int top, int width, int ff, int rows_per_expert,
-                          cudaStream_t stream) {
+                          float alpha, float shift, float limit, cudaStream_t stream) {
+    const NsGate act_kind{alpha, shift, limit};
     if (width % 8 || ff % 8) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_moe_grouped: width %d and expert width %d must be multiples of 8", width, ff);
     if ((((uintptr_t)x | (uintptr_t)w_gate | (uintptr_t)w_up | (uintptr_t)w_down | (uintptr_t)act) % 16) || ((uintptr_t)ys % 4))
         NS_FAIL(NS_ERR_ARGUMENT, "ns_moe_grouped: operands must start on 16 bytes");
@@ -162,10 +164,10 @@ NS_API int ns_moe_grouped(const void* x, const int* pair_of, const int* offsets,
             NS_CUDA(cudaFuncSetAttribute(moe_grouped_kernel<false, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));     \
         }                                                                                                                           \
         NS_LAUNCH((moe_grouped_kernel<true, MT>), grid_a, 128, smem, stream, (const __nv_bfloat16*)x, (long long)width, pair_of, top,  \
-                  offsets, (const __nv_bfloat16*)w_gate, (const __nv_bfloat16*)w_up, (__nv_bfloat16*)act, (long long)ff, ff, width);   \
+                  offsets, (const __nv_bfloat16*)w_gate, (const __nv_bfloat16*)w_up, (__nv_bfloat16*)act, (long long)ff, ff, width, act_kind); \
         NS_CHECK_LAUNCH("ns_moe_grouped");                                                                                          \
         NS_LAUNCH((moe_grouped_kernel<false, MT>), grid_b, 128, smem, stream, (const __nv_bfloat16*)act, (long long)ff, pair_of, top, \
-                  offsets, (const __nv_bfloat16*)w_down, (const __nv_bfloat16*)nullptr, (__nv_bfloat16*)ys, (long long)width, width, ff); \
+                  offsets, (const __nv_bfloat16*)w_down, (const __nv_bfloat16*)nullptr, (__nv_bfloat16*)ys, (long long)width, width, ff, act_kind); \
         NS_CHECK_LAUNCH("ns_moe_grouped");                                                                                          \
     }
     if (wide) NS_GROUPED(4) else NS_GROUPED(2)

@@ -3,7 +3,8 @@
 // ns_moe_plan has laid the (token, choice) pairs out so that every expert's pairs are neighbours and ns_moe_gather has brought
 // their rows of x into that order: expert e owns rows offsets[e] .. offsets[e + 1] of xs, read on the device.  Two products,
 // one kernel: the experts' packed gate/up projection (runs of 64 gate features and the 64 matching up features alternate, so a
-// tile of 128 weight rows holds both halves of 64 outputs) with silu(gate) * up in the epilogue, and the down projection.
+// tile of 128 weight rows holds both halves of 64 outputs) with silu(gate) * up, or another unit of that form (NsGate), in the
+// epilogue, and the down projection.
 //
 // The layout of a product is gemm_tcgen05.cu's: 128 weight rows are the M side of tcgen05.mma, BN rows of xs its N side; one lane
 // of warp 0 loads tiles of 64 along k with TMA (128-byte swizzle) into a ring of stages, one lane of warp 1 issues the products
@@ -33,7 +34,7 @@ template <int BN>
 __global__ void __launch_bounds__(kThreads, Cfg<BN>::kMinBlocks)
 moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                       __nv_bfloat16* __restrict__ out, long long ldo, const int* __restrict__ offsets, int E, int rows_w, int k_blocks,
-                      int gated, int* __restrict__ error_flag) {
+                      int gated, NsGate act, int* __restrict__ error_flag) {
     using C = Cfg<BN>;
     extern __shared__ unsigned char smem_dyn[];
     const uint32_t base = (smem_u32(smem_dyn) + 1023u) & ~1023u;
@@ -178,7 +179,7 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
 #pragma unroll
             for (int k = 0; k < 8; k += 4) *reinterpret_cast<float4*>(u + k) = *reinterpret_cast<const float4*>(src + 64 + k);
 #pragma unroll
-            for (int k = 0; k < 8; ++k) v[k] = __fdividef(v[k], 1.f + __expf(-v[k])) * u[k];
+            for (int k = 0; k < 8; ++k) v[k] = ns_gate_mul<true>(act, v[k], u[k]);
             st8(out + (size_t)(row0 + j) * ldo + n0 / 2 + p, v);
         } else if (n0 + p < rows_w) {  // (rows beyond the expert's belong to the next one)
             st8(out + (size_t)(row0 + j) * ldo + n0 + p, v);
@@ -188,7 +189,7 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
 
 template <int BN>
 int launch_grouped(const void* x, const void* w, void* out, long long ldo, const int* offsets, int E, int n_pairs, int rows_w, int K,
-                   int gated, int* error_flag, cudaStream_t stream) {
+                   int gated, NsGate act, int* error_flag, cudaStream_t stream) {
     using C = Cfg<BN>;
     static bool configured = false;
     if (!configured) {
@@ -201,7 +202,7 @@ int launch_grouped(const void* x, const void* w, void* out, long long ldo, const
     const int most = min(n_pairs, n_pairs / BN + E);  // tiles that n_pairs rows of E experts can make
     if (most > 65535) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_moe_grouped_tc: %d pairs over %d experts exceed the grid", n_pairs, E);
     NS_LAUNCH((moe_grouped_tc_kernel<BN>), dim3((rows_w + BM - 1) / BM, most), kThreads, C::kSmemBytes, stream, mw, mx, (__nv_bfloat16*)out,
-              ldo, offsets, E, rows_w, (K + BK - 1) / BK, gated, error_flag);
+              ldo, offsets, E, rows_w, (K + BK - 1) / BK, gated, act, error_flag);
     NS_CHECK_LAUNCH("ns_moe_grouped_tc");
     return NS_OK;
 }
@@ -210,9 +211,10 @@ int launch_grouped(const void* x, const void* w, void* out, long long ldo, const
 
 // xs [n_pairs, width]: the pairs' rows in the plan's order; offsets [E + 1] of that plan; w_gate_up [E, 2 * ff, width] (runs of 64 gate and
 // 64 up rows alternate); w_down [E, width, ff]; act [n_pairs, ff] and ys [n_pairs, width] in the plan's order; everything bfloat16,
-// width a multiple of 8, ff of 64.  tile: 32, 128 or 256 rows of xs to a block.  error_flag: a device int that a timed-out wait sets.
+// width a multiple of 8, ff of 64; alpha, shift, limit: NsGate.  tile: 32, 128 or 256 rows of xs to a block.  error_flag: a device int that a timed-out wait sets.
 NS_API int ns_moe_grouped_tc(const void* xs, const int* offsets, const void* w_gate_up, const void* w_down, void* act, void* ys,
-                             int n_experts, int n_pairs, int width, int ff, int tile, int* error_flag, cudaStream_t stream) {
+                             int n_experts, int n_pairs, int width, int ff, int tile, float alpha, float shift, float limit, int* error_flag,
+                             cudaStream_t stream) {
     if (n_pairs <= 0) return NS_OK;
     if (width % 8 || ff % 64 || n_experts < 1) NS_FAIL(NS_ERR_UNSUPPORTED, "ns_moe_grouped_tc: width %d (a multiple of 8), expert width %d (of 64)", width, ff);
     if (((uintptr_t)xs | (uintptr_t)w_gate_up | (uintptr_t)w_down | (uintptr_t)act | (uintptr_t)ys) % 16)
@@ -220,7 +222,7 @@ NS_API int ns_moe_grouped_tc(const void* xs, const int* offsets, const void* w_g
     if (tile != 32 && tile != 128 && tile != 256) NS_FAIL(NS_ERR_ARGUMENT, "ns_moe_grouped_tc: tiles of %d rows", tile);
     auto run = [&](const void* x, const void* w, void* out, int rows_w, int K, int gated) {
         auto* launch = tile == 256 ? launch_grouped<256> : tile == 128 ? launch_grouped<128> : launch_grouped<32>;
-        return launch(x, w, out, gated ? rows_w / 2 : rows_w, offsets, n_experts, n_pairs, rows_w, K, gated, error_flag, stream);
+        return launch(x, w, out, gated ? rows_w / 2 : rows_w, offsets, n_experts, n_pairs, rows_w, K, gated, NsGate{alpha, shift, limit}, error_flag, stream);
     };
     if (const int rc = run(xs, w_gate_up, act, 2 * ff, width, 1)) return rc;
     return run(act, w_down, ys, width, ff, 0);

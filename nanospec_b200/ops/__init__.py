@@ -109,13 +109,34 @@ def residual_add(resid: torch.Tensor, branch: torch.Tensor) -> torch.Tensor:
     return resid
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0) -> torch.Tensor:
-    """out[n, j] = silu(gate_up[n, j]) * gate_up[n, I + j]; with `block` > 0 gate and up alternate in
+@dataclass(frozen=True)
+class GatedUnit:
+    """A gated feed-forward's activation: with the gate g held below `limit` and the up part u within +-`limit` (0: as they are),
+    g * sigmoid(alpha * g) * (u + shift).  The default is silu(g) * u."""
+
+    alpha: float = 1.0
+    shift: float = 0.0
+    limit: float = 0.0
+
+    @property
+    def args(self) -> tuple[float, float, float]:
+        return float(self.alpha), float(self.shift), float(self.limit)
+
+
+SILU = GatedUnit()
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0, unit: GatedUnit = SILU) -> torch.Tensor:
+    """out[n, j] = silu(gate_up[n, j]) * gate_up[n, I + j] (or another `unit` of the two); with `block` > 0 gate and up alternate in
     runs of `block` features instead (gate j at (j // block) * 2 * block + j % block, up `block` further)."""
     _cuda(gate_up, out)
     n, inter = out.shape
     if gate_up.shape != (n, 2 * inter) or gate_up.dtype != out.dtype or gate_up.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("swiglu: gate_up must be [N, 2I] and out [N, I], same dtype, rows with unit inner stride")
+    if unit != SILU:
+        lib.call("ns_gate_mul_rows", gate_up.data_ptr(), gate_up.stride(0), out.data_ptr(), out.stride(0), n, inter, int(block), *unit.args,
+                 dtype_code(out.dtype), _stream())
+        return out
     if not (gate_up.is_contiguous() and out.is_contiguous()):  # column ranges of wider buffers
         lib.call("ns_swiglu_rows", gate_up.data_ptr(), gate_up.stride(0), out.data_ptr(), out.stride(0), n, inter, int(block),
                  dtype_code(out.dtype), _stream())
@@ -271,15 +292,26 @@ class RowScaled:
 
 
 @dataclass
+class TanhNorm:
+    """The tensors of a norm without statistics, tanh(alpha * x) * gain + bias: float32, `alpha` one number on the device."""
+
+    gain: torch.Tensor
+    bias: torch.Tensor | None
+    alpha: torch.Tensor
+
+
+@dataclass
 class TanhSink:
     """Where a product's output goes when the residual sum and a norm WITHOUT statistics that follow are folded into its epilogue:
-    `resid` [N, H] float32 is updated in place and tanh(alpha * resid) * gain + bias comes back complete, as a `Normed`."""
+    `resid` [N, H] float32 is updated in place and tanh(alpha * resid) * gain + bias comes back complete, as a `Normed`.
+    `post`: the product itself passes a norm of this kind before it joins the stream."""
 
     resid: torch.Tensor
     gain: torch.Tensor
     bias: torch.Tensor | None
     alpha: torch.Tensor  # one float32 on the device
     workspace: object
+    post: TanhNorm | None = None
 
 
 @dataclass
@@ -358,7 +390,9 @@ def linear(x, w: torch.Tensor, out: torch.Tensor, sink: NormSink | None = None):
             N = w.shape[0]
             normed = sink.workspace.get("sink_x", M, N, torch.bfloat16)
             lib.call("ns_gemm_bf16_tc_dyt", x.data_ptr(), w.data_ptr(), M, N, K, x.stride(0), w.stride(0), gemm_splits(M, N, K),
-                     sink.resid.data_ptr(), sink.gain.data_ptr(), _ptr(sink.bias), sink.alpha.data_ptr(), normed.data_ptr(), N,
+                     sink.resid.data_ptr(), sink.gain.data_ptr(), _ptr(sink.bias), sink.alpha.data_ptr(),
+                     *((_ptr(sink.post.gain), _ptr(sink.post.bias), _ptr(sink.post.alpha)) if sink.post is not None else (None, None, None)),
+                     normed.data_ptr(), N,
                      _tc(x.device).error.data_ptr(), _stream())
             return Normed(normed, sink.gain)
         sink = None  # the step does not fit: the plain product, and the caller's norm runs as a kernel of its own
@@ -447,15 +481,15 @@ def linear_rope(x, w: torch.Tensor, out: torch.Tensor, positions: torch.Tensor, 
 GATE_BLOCK = 64  # gate and up rows alternate in runs of this many in a packed projection that the fused kernel takes
 
 
-def gated_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor, block: int) -> torch.Tensor:
-    """out[n, j] = silu(x @ gate_j) * (x @ up_j) for a packed projection w [2I, K]: [gate | up] when
+def gated_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor, block: int, unit: GatedUnit = SILU) -> torch.Tensor:
+    """out[n, j] = silu(x @ gate_j) * (x @ up_j) (or another `unit` of the two) for a packed projection w [2I, K]: [gate | up] when
     `block` is 0, runs of `block` gate rows followed by the matching up rows otherwise.  A decode step
     in bfloat16 with block == GATE_BLOCK is one tcgen05 kernel whose epilogue applies the activation;
     everything else is the product into `scratch` [N, 2I] and the swiglu kernel.  `x` may be a `RowScaled`."""
     if isinstance(x, RowScaled):
-        if block == GATE_BLOCK and out.dtype == torch.bfloat16:
+        if block == GATE_BLOCK and out.dtype == torch.bfloat16 and unit == SILU:
             return _linear_norm(x, w, out, True, None)
-        return swiglu(_linear_norm(x, w, scratch, False, None), out, block)
+        return swiglu(_linear_norm(x, w, scratch, False, None), out, block, unit)
     _cuda(x, w, out, scratch)
     M, K = x.shape
     if x.dtype == torch.bfloat16 and block == GATE_BLOCK and USE_TENSOR_CORE_GEMM and w.shape[0] % 128 == 0 \
@@ -464,24 +498,25 @@ def gated_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch: t
                                                      or w.data_ptr() % 16 or x.stride(1) != 1 or w.stride(1) != 1):
         if w.shape[1] != K or out.shape != (M, w.shape[0] // 2) or out.stride(1) != 1:
             raise KernelError(f"gated_linear: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)} do not agree")
-        lib.call("ns_gemm_bf16_tc_gated", x.data_ptr(), w.data_ptr(), out.data_ptr(), M, w.shape[0], K, x.stride(0),
-                 w.stride(0), out.stride(0), 0, gemm_splits(M, w.shape[0], K), _tc(x.device).error.data_ptr(), _stream())
+        lib.call("ns_gemm_bf16_tc_gated" if unit == SILU else "ns_gemm_bf16_tc_unit", x.data_ptr(), w.data_ptr(), out.data_ptr(), M,
+                 w.shape[0], K, x.stride(0), w.stride(0), out.stride(0), 0, gemm_splits(M, w.shape[0], K), *(() if unit == SILU else unit.args), _tc(x.device).error.data_ptr(), _stream())
         return out
-    return swiglu(linear(x, w, scratch), out, block)
+    return swiglu(linear(x, w, scratch), out, block, unit)
 
 
 def attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                       token_req: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, nq: int, nkv: int,
                       head_dim: int, page_size: int, scale: float | None = None, window: int = 0,
                       keep_first: int = 0, v_dim: int | None = None, chunk: int = 0, softcap: float = 0.0,
-                      sink: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
+                      sink: torch.Tensor | None = None, gate: torch.Tensor | None = None, feature_gate: bool = False,
+                      out_scale: float = 1.0) -> torch.Tensor:
     """q: [N, >= nq*head_dim] rows (a view into the packed projection is fine, unit inner
     stride); out: [N, nq*v_dim] (`v_dim`: the values' head size when it differs from the keys').  `keep_first`: the
     first so many keys of a request stay visible behind the window.  `chunk` > 0: a query sees only the keys of its own
-    chunk of that many positions; `softcap` > 0: scaled scores pass through softcap * tanh(s / softcap).  `sink` and
-    `gate`: see `attention`.  See csrc/attention_generic.cu for the masking rule."""
+    chunk of that many positions; `softcap` > 0: scaled scores pass through softcap * tanh(s / softcap).  `sink`,
+    `gate`, `feature_gate` and `out_scale`: see `attention`.  See csrc/attention_generic.cu for the masking rule."""
     _cuda(q, k_cache, v_cache, block_table, token_req, positions, out, sink, gate)
-    _check_sink_gate(sink, gate, nq, n_rows=out.shape[0], dtype=q.dtype)
+    _check_sink_gate(sink, gate, nq, n_rows=out.shape[0], dtype=q.dtype, gates=nq * int(v_dim or head_dim) if feature_gate else nq)
     _i32(positions, "positions"), _i32(token_req, "token_req")
     n = out.shape[0]
     if q.stride(1) != 1 or out.stride(1) != 1 or q.shape[0] != n or q.dtype != out.dtype:
@@ -494,15 +529,16 @@ def attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
              block_table.data_ptr(), block_table.stride(0), token_req.data_ptr(), positions.data_ptr(),
              out.data_ptr(), out.stride(0), n, nq, nkv, head_dim, int(v_dim or head_dim), page_size, float(scale), int(window),
              int(keep_first), int(chunk), float(softcap), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0,
-             dtype_code(q.dtype), _stream())
+             int(bool(feature_gate)), float(out_scale), dtype_code(q.dtype), _stream())
     return out
 
 
-def _check_sink_gate(sink: torch.Tensor | None, gate: torch.Tensor | None, nq: int, n_rows: int, dtype: torch.dtype) -> None:
+def _check_sink_gate(sink: torch.Tensor | None, gate: torch.Tensor | None, nq: int, n_rows: int, dtype: torch.dtype,
+                     gates: int) -> None:
     if sink is not None and (sink.dtype != torch.float32 or sink.numel() != nq or not sink.is_contiguous()):
         raise KernelError("attention: the sink is one contiguous float32 number per query head")
-    if gate is not None and (gate.dtype != dtype or gate.dim() != 2 or gate.shape[0] != n_rows or gate.shape[1] < nq or gate.stride(1) != 1):
-        raise KernelError("attention: the gate is one number per token and query head, in the activations' dtype, unit inner stride")
+    if gate is not None and (gate.dtype != dtype or gate.dim() != 2 or gate.shape[0] != n_rows or gate.shape[1] < gates or gate.stride(1) != 1):
+        raise KernelError("attention: the gate is one number per token and query head (or output feature), in the activations' dtype, unit inner stride")
 
 
 def sample_rows(logits: torch.Tensor, temperature: torch.Tensor, top_k: torch.Tensor, top_p: torch.Tensor,
@@ -556,10 +592,18 @@ def _target_blocks() -> int:
 
 
 def _tensor_core_attention(dtype: torch.dtype, head_dim: int, v_dim: int | None = None) -> bool:
-    """Keys and values of one width: multiples of 16 up to 128; of two widths: multiples of 8, the larger at most 128."""
+    """Keys and values of one width: multiples of 16 up to 128; of two widths: multiples of 8, keys up to 128 and values up to 512
+    (in slices of up to 128)."""
     if v_dim is None or v_dim == head_dim:
         return dtype == torch.bfloat16 and head_dim % 16 == 0 and 16 <= head_dim <= 128
-    return dtype == torch.bfloat16 and head_dim % 8 == 0 and v_dim % 8 == 0 and 8 <= min(head_dim, v_dim) and max(head_dim, v_dim) <= 128
+    return dtype == torch.bfloat16 and head_dim % 8 == 0 and v_dim % 8 == 0 and 8 <= min(head_dim, v_dim) and head_dim <= 128 and v_dim <= 512
+
+
+def _value_slices(head_dim: int, v_dim: int) -> tuple[int, int]:
+    """Slices of a value's features in the m16n8k16 kernels, and the columns of the instance that runs (csrc/attention_common.cuh)."""
+    count = -(-v_dim // 128)
+    width = -(-(-(-v_dim // count)) // 8) * 8
+    return count, -(-max(head_dim, width) // 16) * 16
 
 
 USE_CLUSTER_DECODE = True
@@ -582,7 +626,7 @@ def attention_decode(qkv: torch.Tensor, lane, ctx, out: torch.Tensor, nq: int, n
                      window: int, rows: torch.Tensor | None, n_rows: int, max_kv_len: int | None,
                      work: torch.Tensor | None = None, work_slots: int = 0, keep_first: int = 0, wide_weights: bool = False,
                      chunk: int = 0, softcap: float = 0.0, v_dim: int | None = None, sink: torch.Tensor | None = None,
-                     gate: torch.Tensor | None = None) -> None:
+                     gate: torch.Tensor | None = None, feature_gate: bool = False, out_scale: float = 1.0) -> None:
     """Split-KV decode attention for the requests that bring one token.  Head sizes 64 and 128 with
     pages of 8 to 64 tokens: TMA loads and a thread-block cluster per request and kv head
     (csrc/attention_decode_tma.cu); everything else: cp.async loads and a merge through global
@@ -600,7 +644,7 @@ def attention_decode(qkv: torch.Tensor, lane, ctx, out: torch.Tensor, nq: int, n
     # pages in key order and knows one mask)
     if USE_CLUSTER_DECODE and head_dim in (64, 128) and lane.page_size in (8, 16, 32, 64) and qkv.stride(0) % 2 == 0 \
             and not keep_first and not wide_weights and not chunk and not softcap and v_dim == head_dim \
-            and sink is None and gate is None:
+            and sink is None and gate is None and out_scale == 1.0:
         n_splits = _cluster_decode_splits(n_rows * nkv * head_tiles, max_kv_len)
         if work is not None and window == 0:
             ws = ctx.workspace
@@ -618,7 +662,8 @@ def attention_decode(qkv: torch.Tensor, lane, ctx, out: torch.Tensor, nq: int, n
                  nkv, head_dim, lane.page_size, float(scale), int(window), n_splits, _tc(qkv.device).error.data_ptr(),
                  None, None, None, _stream())
         return
-    n_splits = max(1, min(16, -(-_target_blocks() // (n_rows * nkv * head_tiles))))
+    slices, instance = _value_slices(head_dim, v_dim)
+    n_splits = max(1, min(16, -(-_target_blocks() // (n_rows * nkv * head_tiles * slices))))
     if max_kv_len is not None:
         # long contexts split further (measured: 4 splits are best at 4,096 keys even for 64 requests),
         # and a split keeps at least two tiles of keys
@@ -629,15 +674,15 @@ def attention_decode(qkv: torch.Tensor, lane, ctx, out: torch.Tensor, nq: int, n
         if chunk > 0:
             n_splits = max(1, min(n_splits, -(-min(max_kv_len, chunk) // 128)))
     ws = ctx.workspace
-    part_o = ws.get("attn_part_o", n_rows * nq * n_splits, -(-max(head_dim, v_dim) // 16) * 16, torch.float32)
-    part_ml = ws.get("attn_part_ml", n_rows * nq * n_splits, 2, torch.float32)
-    counters = ws.get("attn_counters", n_rows * nkv * head_tiles, 1, torch.int32, zero=True)
+    part_o = ws.get("attn_part_o", n_rows * nq * slices * n_splits, instance, torch.float32)
+    part_ml = ws.get("attn_part_ml", n_rows * nq * slices * n_splits, 2, torch.float32)
+    counters = ws.get("attn_counters", n_rows * nkv * head_tiles * slices, 1, torch.int32, zero=True)
     lib.call("ns_attention_decode_kept", qkv.data_ptr(), qkv.stride(0), lane.k.data_ptr(), lane.v.data_ptr(),
              lane.block_table.data_ptr(), lane.block_table.stride(0), ctx.token_req.data_ptr(), ctx.positions.data_ptr(),
              ctx.qo_indptr.data_ptr(), out.data_ptr(), out.stride(0), part_o.data_ptr(), part_ml.data_ptr(),
              counters.data_ptr(), _ptr(rows), n_rows, nq, nkv, head_dim, lane.page_size, float(scale), int(window),
              int(keep_first), int(bool(wide_weights)), int(chunk), float(softcap), n_splits, int(v_dim), _ptr(sink), _ptr(gate),
-             gate.stride(0) if gate is not None else 0, _stream())
+             gate.stride(0) if gate is not None else 0, int(bool(feature_gate)), float(out_scale), _stream())
 
 
 PREFILL_TWO_HEADS = "auto"  # "always" / "never": tests run both kernels whatever the size of the grid
@@ -646,14 +691,15 @@ PREFILL_TWO_HEADS = "auto"  # "always" / "never": tests run both kernels whateve
 def attention_prefill(qkv: torch.Tensor, lane, ctx, out: torch.Tensor, nq: int, nkv: int, head_dim: int, scale: float,
                       window: int, tiles: torch.Tensor, tiles_tc: torch.Tensor | None = None, keep_first: int = 0,
                       wide_weights: bool = False, chunk: int = 0, softcap: float = 0.0, v_dim: int | None = None,
-                      sink: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> None:
+                      sink: torch.Tensor | None = None, gate: torch.Tensor | None = None, feature_gate: bool = False,
+                      out_scale: float = 1.0) -> None:
     """Tensor-core attention for portions of prompts.  `tiles`: int32 [n, 2] of (request, offset
     among its tokens of this step).  Head sizes 64 and 128 with pages of 8 to 64 tokens and no window run
     on tcgen05 (csrc/attention_prefill_tc.cu); everything else on m16n8k16 (csrc/attention_prefill.cu), also values of
     another width than the keys (`v_dim`, both multiples of 8)."""
     v_dim = head_dim if v_dim is None else v_dim
     if USE_TCGEN05_ATTENTION and tiles_tc is not None and head_dim in (64, 128) and window == 0 and not wide_weights \
-            and not chunk and not softcap and v_dim == head_dim and sink is None and gate is None \
+            and not chunk and not softcap and v_dim == head_dim and sink is None and gate is None and out_scale == 1.0 \
             and lane.page_size in (8, 16, 32, 64) and qkv.stride(0) % 8 == 0 and out.stride(0) % 8 == 0:
         # heads of 64: two query heads of a kv head to a block (four softmax warps per sub-partition keep the exponential
         # unit busier and the keys are read once for both) - once one head to a block would give more blocks than SMs
@@ -669,7 +715,7 @@ def attention_prefill(qkv: torch.Tensor, lane, ctx, out: torch.Tensor, nq: int, 
              lane.block_table.data_ptr(), lane.block_table.stride(0), ctx.positions.data_ptr(), ctx.qo_indptr.data_ptr(),
              tiles.data_ptr(), tiles.shape[0], out.data_ptr(), out.stride(0), nq, nkv, head_dim, lane.page_size,
              float(scale), int(window), int(keep_first) if window else 0, int(bool(wide_weights)), int(chunk), float(softcap), int(v_dim),
-             _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, _stream())
+             _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, int(bool(feature_gate)), float(out_scale), _stream())
 
 
 def _attention_plan(ctx) -> dict:
@@ -706,7 +752,8 @@ def _attention_plan(ctx) -> dict:
 
 def attention(qkv: torch.Tensor, lane, ctx, out: torch.Tensor, nq: int, nkv: int, head_dim: int, scale: float,
               window: int = 0, keep_first: int = 0, v_dim: int | None = None, wide_weights: bool = False, chunk: int = 0,
-              softcap: float = 0.0, sink: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
+              softcap: float = 0.0, sink: torch.Tensor | None = None, gate: torch.Tensor | None = None, feature_gate: bool = False,
+              out_scale: float = 1.0) -> torch.Tensor:
     """Attention of the step's queries (the first nq*head_dim columns of `qkv`) over `lane`.
 
     bfloat16 with a head size that the tensor-core kernels take: the decode kernel for requests
@@ -717,15 +764,18 @@ def attention(qkv: torch.Tensor, lane, ctx, out: torch.Tensor, nq: int, nkv: int
     the m16n8k16 kernels); `v_dim`: values of another width than the keys (the same kernels, widths in multiples of 8).
     `sink` (float32 [nq]): the softmax's denominator also holds exp(sink[h]), a term that has no key and no value and counts once
     (zeros: "one added to the denominator"); `gate` ([N, >= nq] in the activations' dtype, a column range of the packed projection
-    is fine): head h's output is multiplied by sigmoid(gate[n, h]).  Both run in the exact and the m16n8k16 kernels.  float32, and head
+    is fine): head h's output is multiplied by sigmoid(gate[n, h]), or, with `feature_gate` ([N, >= nq * v_dim]), every output feature
+    by the sigmoid of its own; `out_scale` multiplies the output before it is rounded.  They run in the exact and the m16n8k16 kernels.  float32, and head
     sizes those kernels refuse: the exact kernel, one warp per (token, head)."""
     v_dim = head_dim if v_dim is None else v_dim
     keep_first = keep_first if window else 0
-    if not _tensor_core_attention(qkv.dtype, head_dim, v_dim) or nq // nkv > 64 or (v_dim != head_dim and (nq * head_dim) % 8):
+    if not _tensor_core_attention(qkv.dtype, head_dim, v_dim) or nq // nkv > 64 or (v_dim != head_dim and (nq * head_dim) % 8) \
+            or (feature_gate and (gate.stride(0) % 2 or gate.data_ptr() % 4)):
         return attention_generic(qkv, lane.k, lane.v, lane.block_table, ctx.token_req, ctx.positions, out, nq, nkv,
-                                 head_dim, lane.page_size, scale, window, keep_first if window else 0, v_dim, chunk, softcap, sink, gate)
+                                 head_dim, lane.page_size, scale, window, keep_first if window else 0, v_dim, chunk, softcap, sink, gate,
+                                 feature_gate, out_scale)
     _cuda(qkv, out, lane.k, lane.v, lane.block_table, sink, gate)
-    _check_sink_gate(sink, gate, nq, n_rows=out.shape[0], dtype=qkv.dtype)
+    _check_sink_gate(sink, gate, nq, n_rows=out.shape[0], dtype=qkv.dtype, gates=nq * v_dim if feature_gate else nq)
     if out.stride(1) != 1 or qkv.stride(1) != 1 or lane.k.dtype != qkv.dtype:
         raise KernelError("attention: row-major bfloat16 operands and a bfloat16 cache are needed")
     plan = _attention_plan(ctx)
@@ -739,18 +789,22 @@ def attention(qkv: torch.Tensor, lane, ctx, out: torch.Tensor, nq: int, nkv: int
         fork, join = _side_events(qkv.device)
         fork.record(main)
         side.wait_event(fork)
-        attention_prefill(qkv, lane, ctx, out, nq, nkv, head_dim, scale, window, plan["tiles"], plan.get("tiles_tc"), keep_first, wide_weights, chunk, softcap, v_dim, sink, gate)
+        attention_prefill(qkv, lane, ctx, out, nq, nkv, head_dim, scale, window, plan["tiles"], plan.get("tiles_tc"), keep_first, wide_weights, chunk, softcap, v_dim, sink, gate,
+                              feature_gate, out_scale)
         with torch.cuda.stream(side):
             attention_decode(qkv, lane, ctx, out, nq, nkv, head_dim, scale, window, plan["decode_rows"], plan["n_decode"],
-                             plan["max_kv_len"], plan.get("work"), plan.get("work_slots", 0), keep_first, wide_weights, chunk, softcap, v_dim, sink, gate)
+                             plan["max_kv_len"], plan.get("work"), plan.get("work_slots", 0), keep_first, wide_weights, chunk, softcap, v_dim, sink, gate,
+                              feature_gate, out_scale)
             join.record(side)
         main.wait_event(join)
         return out
     if plan["n_decode"]:
         attention_decode(qkv, lane, ctx, out, nq, nkv, head_dim, scale, window, plan["decode_rows"], plan["n_decode"],
-                         plan["max_kv_len"], plan.get("work"), plan.get("work_slots", 0), keep_first, wide_weights, chunk, softcap, v_dim, sink, gate)
+                         plan["max_kv_len"], plan.get("work"), plan.get("work_slots", 0), keep_first, wide_weights, chunk, softcap, v_dim, sink, gate,
+                              feature_gate, out_scale)
     if plan["tiles"] is not None:
-        attention_prefill(qkv, lane, ctx, out, nq, nkv, head_dim, scale, window, plan["tiles"], plan.get("tiles_tc"), keep_first, wide_weights, chunk, softcap, v_dim, sink, gate)
+        attention_prefill(qkv, lane, ctx, out, nq, nkv, head_dim, scale, window, plan["tiles"], plan.get("tiles_tc"), keep_first, wide_weights, chunk, softcap, v_dim, sink, gate,
+                              feature_gate, out_scale)
     return out
 
 
@@ -1205,8 +1259,8 @@ def cast_f32(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
 ROUTER_DIRECT_MAX = 1 << 31
 
 
-def router_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch=None) -> torch.Tensor:
-    """out [N, E] float32 = x @ w^T with float32 products and sums, x in the compute type, w [E, K] float32:
+def router_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch=None, bias: torch.Tensor | None = None) -> torch.Tensor:
+    """out [N, E] float32 = x @ w^T (+ bias, float32 [E]) with float32 products and sums, x in the compute type, w [E, K] float32:
     one kernel, a warp per expert and a few tokens; very many tokens and a large router: x as float32 (into `scratch(...)`'s buffer) and the float32 GEMM."""
     _cuda(x, w, out)
     n, K = x.shape
@@ -1214,16 +1268,23 @@ def router_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch=N
     if w.dtype != torch.float32 or out.dtype != torch.float32 or out.shape != (n, E) or not (w.is_contiguous() and out.is_contiguous()) \
             or x.stride(1) != 1 or w.shape[1] != K:
         raise KernelError("router_logits: float32 router [E, K] and logits [N, E], contiguous; x rows with unit inner stride")
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != E or not bias.is_contiguous()):
+        raise KernelError("router_logits: one contiguous float32 bias per output")
     if n * E * K <= ROUTER_DIRECT_MAX or n <= 64:
-        lib.call("ns_router_logits", x.data_ptr(), x.stride(0), w.data_ptr(), out.data_ptr(), n, E, K, dtype_code(x.dtype), _stream())
+        lib.call("ns_router_logits", x.data_ptr(), x.stride(0), w.data_ptr(), _ptr(bias), out.data_ptr(), n, E, K, dtype_code(x.dtype), _stream())
         return out
     x32 = x if x.dtype == torch.float32 else cast_f32(x, scratch(n, K))
-    return linear(x32, w, out)
+    linear(x32, w, out)
+    return out if bias is None else add_bias(out, bias)
+
+
+ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_CHOSEN = 0, 1, 2
 
 
 def moe_route(logits: torch.Tensor, groups: int, keep: int, top: int, scale: float, ids: torch.Tensor, weights: torch.Tensor,
-              softmax: bool = False, correction: torch.Tensor | None = None, renormalize: bool = True) -> None:
-    """Per row of float32 logits [N, E]: the chosen experts (int32 [N, top], largest score first) and their weights
+              softmax: int = 0, correction: torch.Tensor | None = None, renormalize: bool = True) -> None:
+    """`softmax`: ROUTE_SIGMOID, ROUTE_SOFTMAX (over all outputs) or ROUTE_CHOSEN (the logits choose, a softmax over the chosen).
+    Per row of float32 logits [N, E]: the chosen experts (int32 [N, top], largest score first) and their weights
     (float32 [N, top]); see csrc/moe.cu for the rule.  `correction` [E] float32 is added to the scores that choose, not to the
     weights; `renormalize`: the weights are divided by the sum of the chosen scores before they are scaled."""
     _cuda(logits, ids, weights, correction)
@@ -1233,11 +1294,11 @@ def moe_route(logits: torch.Tensor, groups: int, keep: int, top: int, scale: flo
     if logits.dtype != torch.float32 or not logits.is_contiguous() or ids.dtype != torch.int32 or weights.dtype != torch.float32 \
             or ids.shape != (n, top) or weights.shape != (n, top) or not (ids.is_contiguous() and weights.is_contiguous()):
         raise KernelError("moe_route: float32 logits [N, E], int32 ids and float32 weights [N, top], contiguous")
-    lib.call("ns_moe_route", logits.data_ptr(), n, E, int(groups), int(keep), int(top), float(scale), int(bool(softmax)),
+    lib.call("ns_moe_route", logits.data_ptr(), n, E, int(groups), int(keep), int(top), float(scale), int(softmax),
              _ptr(correction), int(bool(renormalize)), ids.data_ptr(), weights.data_ptr(), _stream())
 
 
-def moe_route_plan(logits: torch.Tensor, groups: int, keep: int, top: int, scale: float, ids: torch.Tensor, weights: torch.Tensor, softmax: bool,
+def moe_route_plan(logits: torch.Tensor, groups: int, keep: int, top: int, scale: float, ids: torch.Tensor, weights: torch.Tensor, softmax: int,
                    correction: torch.Tensor | None, renormalize: bool, n_experts: int, offsets: torch.Tensor, row_of: torch.Tensor,
                    pair_of: torch.Tensor) -> None:
     """`moe_route` and `moe_plan` in one launch of one block (`route_plan_ok`)."""
@@ -1250,7 +1311,7 @@ def moe_route_plan(logits: torch.Tensor, groups: int, keep: int, top: int, scale
             or offsets.numel() != n_experts + 1 \
             or (correction is not None and (correction.dtype != torch.float32 or correction.numel() != E or not correction.is_contiguous())):
         raise KernelError("moe_route_plan: operands as moe_route and moe_plan take them")
-    lib.call("ns_moe_route_plan", logits.data_ptr(), n, E, int(groups), int(keep), int(top), float(scale), int(bool(softmax)), _ptr(correction),
+    lib.call("ns_moe_route_plan", logits.data_ptr(), n, E, int(groups), int(keep), int(top), float(scale), int(softmax), _ptr(correction),
              int(bool(renormalize)), ids.data_ptr(), weights.data_ptr(), int(n_experts), offsets.data_ptr(), row_of.data_ptr(),
              pair_of.data_ptr(), _stream())
 
@@ -1276,9 +1337,9 @@ def moe_grouped_ok(x: torch.Tensor, width: int, ff: int) -> bool:
 
 
 def moe_grouped(x: torch.Tensor, pair_of: torch.Tensor, offsets: torch.Tensor, w_gate: torch.Tensor, w_up: torch.Tensor,
-                w_down: torch.Tensor, act: torch.Tensor, ys: torch.Tensor, top: int) -> torch.Tensor:
+                w_down: torch.Tensor, act: torch.Tensor, ys: torch.Tensor, top: int, unit: GatedUnit = SILU) -> torch.Tensor:
     """Every expert over its rows of the plan, on the tensor cores, the counts read on the device (csrc/moe_tc.cu):
-    act [pairs, ff] = silu(x . gate) * (x . up), ys [pairs, width] = act . down, both in the plan's row order."""
+    act [pairs, ff] = silu(x . gate) * (x . up) (or another `unit`), ys [pairs, width] = act . down, both in the plan's row order."""
     _cuda(x, pair_of, offsets, w_gate, w_up, w_down, act, ys)
     n, width = x.shape
     E, ff = w_gate.shape[0], w_gate.shape[1]
@@ -1286,17 +1347,18 @@ def moe_grouped(x: torch.Tensor, pair_of: torch.Tensor, offsets: torch.Tensor, w
             or act.shape != (n * top, ff) or ys.shape != (n * top, width) or w_down.shape != (E, width, ff) or w_up.shape != w_gate.shape:
         raise KernelError("moe_grouped: contiguous bfloat16 operands of the sizes the experts have")
     lib.call("ns_moe_grouped", x.data_ptr(), pair_of.data_ptr(), offsets.data_ptr(), w_gate.data_ptr(), w_up.data_ptr(),
-             w_down.data_ptr(), act.data_ptr(), ys.data_ptr(), E, int(top), width, ff, (n * int(top)) // E, _stream())
+             w_down.data_ptr(), act.data_ptr(), ys.data_ptr(), E, int(top), width, ff, (n * int(top)) // E, *unit.args, _stream())
     return ys
 
 
 MOE_TILE: int | None = None  # rows of a tile in `moe_grouped_tc` (None: by the rows an expert holds on average)
 
 
-def moe_grouped_tc(xs: torch.Tensor, offsets: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, act: torch.Tensor, ys: torch.Tensor) -> torch.Tensor:
+def moe_grouped_tc(xs: torch.Tensor, offsets: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, act: torch.Tensor, ys: torch.Tensor,
+                   unit: GatedUnit = SILU) -> torch.Tensor:
     """Every expert over its rows of the plan as tcgen05 products whose tiles are found from the offsets on the device
     (csrc/moe_tcgen05.cu): xs [pairs, width] in the plan's order (`moe_gather`), w_gate_up [E, 2 ff, width] with gate and up rows alternating in
-    runs of GATE_BLOCK, act [pairs, ff] = silu(gate) * up, ys [pairs, width] = act . down."""
+    runs of GATE_BLOCK, act [pairs, ff] = silu(gate) * up (or another `unit`), ys [pairs, width] = act . down."""
     _cuda(xs, offsets, w_gate_up, w_down, act, ys)
     _i32(offsets, "offsets")
     n, width = xs.shape
@@ -1306,7 +1368,7 @@ def moe_grouped_tc(xs: torch.Tensor, offsets: torch.Tensor, w_gate_up: torch.Ten
         raise KernelError("moe_grouped_tc: contiguous bfloat16 operands of the sizes the experts have")
     tile = MOE_TILE or (256 if n >= 300 * E else 128 if n > 24 * E else 32)
     lib.call("ns_moe_grouped_tc", xs.data_ptr(), offsets.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), act.data_ptr(), ys.data_ptr(),
-             E, n, width, ff, tile, _tc(xs.device).error.data_ptr(), _stream())
+             E, n, width, ff, tile, *unit.args, _tc(xs.device).error.data_ptr(), _stream())
     return ys
 
 
@@ -1346,7 +1408,7 @@ def moe_combine(ys: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor, o
 
 
 def moe_expert_rows(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate: torch.Tensor, w_up: torch.Tensor,
-                    w_down: torch.Tensor, act: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+                    w_down: torch.Tensor, act: torch.Tensor, out: torch.Tensor, unit: GatedUnit = SILU) -> torch.Tensor:
     """The chosen experts of a few tokens without a host round trip: w_gate, w_up [E, ff, width], w_down [E, width, ff]; ids
     from E on return their input."""
     _cuda(x, ids, weights, w_gate, w_up, w_down, act, out)
@@ -1356,7 +1418,7 @@ def moe_expert_rows(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w
             or out.shape != (n, width) or w_down.shape[1:] != (width, ff) or len({x.dtype, w_gate.dtype, w_up.dtype, w_down.dtype, act.dtype, out.dtype}) != 1:
         raise KernelError("moe_expert_rows: contiguous operands of one dtype and the sizes the experts have")
     lib.call("ns_moe_expert_rows", x.data_ptr(), ids.data_ptr(), weights.data_ptr(), w_gate.data_ptr(), w_up.data_ptr(),
-             w_down.data_ptr(), act.data_ptr(), out.data_ptr(), w_gate.shape[0], n, top, width, ff, dtype_code(x.dtype), _stream())
+             w_down.data_ptr(), act.data_ptr(), out.data_ptr(), w_gate.shape[0], n, top, width, ff, *unit.args, dtype_code(x.dtype), _stream())
     return out
 
 
@@ -1441,6 +1503,58 @@ def add_dyt(resid: torch.Tensor, branches, gain: torch.Tensor, bias: torch.Tenso
     b = branches[1] if len(branches) > 1 else None
     lib.call("ns_add_dyt", resid.data_ptr(), _ptr(a), _ptr(b), gain.data_ptr(), _ptr(bias), alpha.data_ptr(), out.data_ptr(), _ptr(rows),
              n_rows, hidden, int(rows is None), dtype_code(out.dtype), _stream())
+    return out
+
+
+@dataclass
+class RoutedSum:
+    """A routed feed-forward's output before it is added up: token n's is sum_k weights[n, k] * ys[rows[n, k]] (every row >= 0), plus
+    `rest` [N, H] (None: nothing), as the kernels that take it sum them in float32."""
+
+    ys: torch.Tensor
+    rows: torch.Tensor
+    weights: torch.Tensor
+    rest: torch.Tensor | None = None
+
+
+def dyt_join(resid: torch.Tensor, branch, post: TanhNorm, next: TanhNorm | None = None, out: torch.Tensor | None = None,
+             rows: torch.Tensor | None = None) -> torch.Tensor | None:
+    """resid += tanh(post.alpha * y) * post.gain + post.bias with y = `branch` - a tensor, a pair of them, or a `RoutedSum` -
+    and, with `next` and `out`, out = tanh(next.alpha * resid) * next.gain + next.bias: one pass, float32 throughout
+    (csrc/elementwise.cu).  With `rows`, output row j reads input row rows[j] and the stream is left unchanged."""
+    hidden = resid.shape[1]
+    routed = branch if isinstance(branch, RoutedSum) else None
+    plain = [t for t in ((routed.rest,) if routed is not None else branch if isinstance(branch, (tuple, list)) else (branch,)) if t is not None]
+    if len(plain) > 2 or (routed is None and not plain) or (next is None) != (out is None) or (rows is not None and out is None):
+        raise KernelError("dyt_join: one or two branches or a routed sum; the next norm and its output go together")
+    _cuda(resid, out, rows, *plain)
+    _i32(rows, "rows")
+    if resid.dtype != torch.float32 or not resid.is_contiguous():
+        raise KernelError("dyt_join: the residual stream is contiguous float32")
+    dt = routed.ys.dtype if routed is not None else plain[0].dtype
+    for t in plain:
+        if t.dtype != dt or t.shape != resid.shape or not t.is_contiguous():
+            raise KernelError("dyt_join: branches have the stream's shape and one dtype")
+    for n in (post, next):
+        if n is not None and (any(t.dtype != torch.float32 or not t.is_contiguous() or t.numel() != hidden for t in (n.gain, n.bias) if t is not None)
+                              or n.alpha.dtype != torch.float32 or n.alpha.numel() != 1):
+            raise KernelError("dyt_join: float32 gains and biases of the stream's width and one float32 alpha")
+    n_rows = resid.shape[0] if rows is None else rows.numel()
+    if out is not None and (out.shape != (n_rows, hidden) or out.dtype != dt or not out.is_contiguous()):
+        raise KernelError("dyt_join: out must be contiguous [rows, hidden] of the branches' dtype")
+    top = 0
+    if routed is not None:
+        top = routed.rows.shape[1]
+        _cuda(routed.ys, routed.rows, routed.weights)
+        _i32(routed.rows, "rows of the routed sum")
+        if routed.rows.shape != (resid.shape[0], top) or routed.weights.shape != routed.rows.shape or routed.weights.dtype != torch.float32 \
+                or not routed.weights.is_contiguous() or routed.ys.shape[1] != hidden or not routed.ys.is_contiguous():
+            raise KernelError("dyt_join: rows and weights [N, top] and ys [pairs, hidden], contiguous")
+    lib.call("ns_dyt_join", resid.data_ptr(), _ptr(plain[0] if plain else None), _ptr(plain[1] if len(plain) > 1 else None),
+             *((_ptr(routed.ys), _ptr(routed.rows), _ptr(routed.weights)) if routed is not None else (None, None, None)), top,
+             post.gain.data_ptr(), _ptr(post.bias), post.alpha.data_ptr(),
+             *((_ptr(next.gain), _ptr(next.bias), _ptr(next.alpha)) if next is not None else (None, None, None)), _ptr(out), _ptr(rows),
+             n_rows, hidden, int(rows is None), dtype_code(dt), _stream())
     return out
 
 

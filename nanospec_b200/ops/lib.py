@@ -28,6 +28,7 @@ _SIGNATURES: dict[str, list] = {
     "ns_residual_add": [_P, _P, _I, _I, _I, _P],
     "ns_swiglu": [_P, _P, _I, _I, _I, _I, _P],
     "ns_swiglu_rows": [_P, _L, _P, _L, _I, _I, _I, _I, _P],
+    "ns_gate_mul_rows": [_P, _L, _P, _L, _I, _I, _I, _F, _F, _F, _I, _P],
     "ns_gemm_f32": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "ns_rope_kv_write": [_P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "ns_attention_generic": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _I, _P],
@@ -45,7 +46,7 @@ _SIGNATURES: dict[str, list] = {
     "ns_attention_decode": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
     "ns_attention_decode_tma": [_P, _I, _P, _P, _L, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P, _P, _P],
     "ns_gemm_bf16_tc_norm": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _F, _P, _P, _P, _P, _I, _P, _P],
-    "ns_gemm_bf16_tc_dyt": [_P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _I, _P, _P],
+    "ns_gemm_bf16_tc_dyt": [_P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _P],
     "ns_rope_token_kernel_from": [_I],
     "ns_gemm_bf16_tc_rope": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _F, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I,
                              _P, _P],
@@ -54,13 +55,15 @@ _SIGNATURES: dict[str, list] = {
     "ns_attention_decode_stages": [_I],
     "ns_gemm_bf16_tc": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "ns_gemm_bf16_tc_gated": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "ns_gemm_bf16_tc_unit": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
     "ns_attention_prefill_tc": [_P, _I, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P],
     "ns_wait_probe": [_P, _L, _P, _P],
     "ns_attention_decode_kept": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _F, _I, _I,
-                                 _P, _P, _I, _P],
-    "ns_attention_prefill_kept": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _F, _I, _P, _P, _I, _P],
-    "ns_attention_generic_sink": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _P, _I, _I, _P],
+                                 _P, _P, _I, _I, _F, _P],
+    "ns_attention_prefill_kept": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _F, _I, _P, _P, _I, _I, _F, _P],
+    "ns_attention_generic_sink": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _P, _I, _I, _F, _I, _P],
     "ns_add_dyt": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
+    "ns_dyt_join": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
     "ns_head_prepare_store": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _I, _P, _F, _I, _I, _P, _P, _I, _F, _F, _F, _P, _I, _P, _L, _P, _P,
                               _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "ns_conv_tail": [_P, _I, _P, _L, _L, _P, _P, _I, _I, _I, _I, _P],
@@ -72,16 +75,16 @@ _SIGNATURES: dict[str, list] = {
     "ns_attention_latent": [_P, _L, _L, _P, _L, _L, _P, _P, _I, _P, _P, _P, _P, _L, _P, _L, _L, _I, _I, _I, _I, _I, _F, _I, _I, _P],
     "ns_attention_latent_tc": [_P, _L, _L, _P, _L, _L, _P, _P, _I, _P, _P, _P, _P, _L, _P, _L, _L, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
     "ns_cast_f32": [_P, _L, _P, _I, _I, _I, _P],
-    "ns_router_logits": [_P, _L, _P, _P, _I, _I, _I, _I, _P],
+    "ns_router_logits": [_P, _L, _P, _P, _P, _I, _I, _I, _I, _P],
     "ns_moe_route": [_P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P, _P],
     "ns_moe_route_plan": [_P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P, _I, _P, _P, _P, _P],
     "ns_moe_plan": [_P, _I, _I, _P, _P, _P, _P],
-    "ns_moe_grouped": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
-    "ns_moe_grouped_tc": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
+    "ns_moe_grouped": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P],
+    "ns_moe_grouped_tc": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
     "ns_moe_pad_rows": [_P, _P, _P, _I, _I, _P],
     "ns_moe_gather": [_P, _P, _P, _I, _I, _I, _I, _P],
     "ns_moe_combine": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
-    "ns_moe_expert_rows": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "ns_moe_expert_rows": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _I, _P],
     "ns_activation": [_P, _P, _L, _I, _P, _I, _P],
     "ns_activation_rows": [_P, _L, _P, _L, _I, _I, _I, _P, _I, _P],
     "ns_norm_add": [_P, _P, _P, _P, _P, _I, _I, _F, _I, _P],

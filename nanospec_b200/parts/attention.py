@@ -45,6 +45,9 @@ class GQAAttention(Part):
                  `writes=False` on that lane), with queries, mask and output projection of its own
     sink         "zero": the softmax's denominator holds one more term, exp(0) = 1, that has no key and no value; "learned": that term
                  is exp(sink[h]) with a float32 tensor of one number per head (name "sink"); default none
+    feature_gate True: a projection `g` of heads * v_dim rows; every feature of the concatenated heads is multiplied by the sigmoid of its
+                 own gate before `o` (in the attention kernels' epilogue, before the output is rounded)
+    out_scale    the concatenated heads are multiplied by this number there as well (default 1)
     names        the tensors' names after the part's prefix, keys "q", "k", "v", "o", "q_norm", "k_norm"
                  (default the Hugging Face ones).
     The next five act on one head at a time and run in one kernel between the projection and the attention (`ops.head_prepare_store`);
@@ -89,6 +92,11 @@ class GQAAttention(Part):
         self.head_norm = dict(p["head_norm"]) if p.get("head_norm") else None
         self.q_temp = dict(p["q_temp"]) if p.get("q_temp") else None
         self.head_gate = bool(p.get("head_gate"))
+        self.feature_gate = bool(p.get("feature_gate"))
+        self.out_scale = float(p.get("out_scale", 1.0))
+        if self.head_gate and self.feature_gate:
+            raise ValueError("gqa_attention: one gate per head or one per feature, not both")
+        self.gates = self.heads if self.head_gate else 0  # columns of the gates' projection
         self.v_from_k = bool(p.get("v_from_k"))
         self.taps = int(p.get("conv") or 0)
         self.per_head = bool(self.head_norm or self.q_temp or self.head_gate or self.v_from_k or self.taps)
@@ -112,11 +120,13 @@ class GQAAttention(Part):
         self.kv_size = self.kv_heads * self.head_dim
         self.v_size = self.kv_heads * self.v_dim
         self.o_in = self.heads * self.v_dim
+        if self.feature_gate:
+            self.gates = self.o_in
         # what the llama-shaped fast paths (a projection with the rotation in its epilogue) do not know of
         self.general = self.v_dim != self.head_dim or self.qk_norm is not None or self.has_bias or not self.own_kv \
-            or self.v_norm is not None
-        # the packed projection's columns on the per-head path: [q | k | v (unless the keys double as values) | g (the heads' gates)]
-        self.channels = self.q_size + self.kv_size + (0 if self.v_from_k else self.v_size)
+            or self.v_norm is not None or self.feature_gate or self.out_scale != 1.0
+        # the packed projection's columns before the gates': [q | k | v (unless the keys double as values)], q alone without own_kv
+        self.channels = self.q_size + (self.kv_size + (0 if self.v_from_k else self.v_size) if self.own_kv else 0)
         self.sink: torch.Tensor | None = None
         self.conv_taps: torch.Tensor | None = None
         self.qkv_bias: torch.Tensor | None = None
@@ -139,8 +149,8 @@ class GQAAttention(Part):
         if self.head_norm and self.head_norm.get("gain"):
             specs[n["q_norm"]] = WeightSpec((self.head_dim,), rule="float32", init="gain")
             specs[n["k_norm"]] = WeightSpec((self.head_dim,), rule="float32", init="gain")
-        if self.head_gate:
-            specs[n["g"]] = WeightSpec((self.heads, self.hidden))
+        if self.gates:
+            specs[n["g"]] = WeightSpec((self.gates, self.hidden))
         if self.sink_kind == "learned":
             specs[n["sink"]] = WeightSpec((self.heads,), rule="float32", init="normal", std=1.0)
         if self.taps:
@@ -161,7 +171,7 @@ class GQAAttention(Part):
         n = self.names
         kinds = (("q", "k") if self.v_from_k else ("q", "k", "v")) if self.own_kv else ("q",)
         # one packed projection [q | k | v]: one matrix product instead of three
-        self.w_qkv = torch.cat([tensors[n[k]] for k in kinds + (("g",) if self.head_gate else ())], dim=0).contiguous()
+        self.w_qkv = torch.cat([tensors[n[k]] for k in kinds + (("g",) if self.gates else ())], dim=0).contiguous()
         if (self.per_head or self.general) and self.w_qkv.shape[0] % 8:  # rows of the product start on 16 bytes in bfloat16
             pad = torch.zeros((-self.w_qkv.shape[0] % 8, self.hidden), dtype=self.w_qkv.dtype, device=self.w_qkv.device)
             self.w_qkv = torch.cat([self.w_qkv, pad], dim=0).contiguous()
@@ -246,7 +256,12 @@ class GQAAttention(Part):
                                        v_dim=self.v_dim, q_gain=self.q_gain, k_gain=self.k_gain,
                                        eps=float(qn["eps"]) if qn else 0.0, **extra)
         ops.attention(qkv, lane, ctx, attn, self.heads, self.kv_heads, self.head_dim, self.scale, self.window,
-                      self.keep_first, self.v_dim, self.wide_weights, self.chunk, self.softcap, sink=self.sink)
+                      self.keep_first, self.v_dim, self.wide_weights, self.chunk, self.softcap, sink=self.sink, gate=self._gate(qkv),
+                      feature_gate=self.feature_gate, out_scale=self.out_scale)
+
+    def _gate(self, proj: torch.Tensor) -> torch.Tensor | None:
+        """The gates' columns of the packed projection."""
+        return proj[:, self.channels: self.channels + self.gates] if self.gates else None
 
     def _forward_per_head(self, x, ctx: StepContext, lane: LaneView, writes: bool):
         """Projection, the per-head steps and the attention (`forward_projected`), output projection."""
@@ -295,6 +310,6 @@ class GQAAttention(Part):
             q_gain=self.q_gain, k_gain=self.k_gain, eps=float(hn["eps"]) if hn else 0.0,
             q_temp=(float(self.q_temp["coef"]), float(self.q_temp["every"])) if self.q_temp else None,
             taps=self.conv_taps, v_from_k=self.v_from_k, write_kv=writes)
-        gate = proj[:, self.channels: self.channels + self.heads] if self.head_gate else None
         ops.attention(qkv, lane, ctx, attn, self.heads, self.kv_heads, self.head_dim, self.scale, self.window, self.keep_first,
-                      self.v_dim, self.wide_weights, self.chunk, self.softcap, sink=self.sink, gate=gate)
+                      self.v_dim, self.wide_weights, self.chunk, self.softcap, sink=self.sink, gate=self._gate(proj),
+                      feature_gate=self.feature_gate, out_scale=self.out_scale)

@@ -39,6 +39,12 @@ that norm is elementwise (`elementwise_sink`): a decode layer is then five kerne
 there as in "prenorm" when nothing but the packed input product reads it (`input_norm_sink`).
 A feed-forward that is only partly a pair of products (routed experts beside a shared one) offers `join_stream(h, ctx, resid)`, which
 adds that part to the float32 stream itself, and `forward_rest(h, ctx)` (or its projections) for what is left, None if nothing is.
+
+"sandwich" norms what a sublayer reads AND what it returns: x = x + norm(mixer(norm(x))); x = x + norm(feed_forward(norm(x))).  The norm on a
+branch, the sum into the stream and the norm that the next sublayer reads are one kernel where both norms are elementwise ("dyt"): the
+block leaves a `PostNormed` pending and the next norm takes it; a routed feed-forward hands its branch over unsummed
+(`forward_unsummed`), so that kernel adds the experts up as well.  In a step of up to 64 tokens a mixer whose last product can feed a
+sink has all of that in its epilogue.  Other norms that offer `join` (an RMS norm) join the stream in a kernel of their own.
 """
 
 from __future__ import annotations
@@ -50,6 +56,7 @@ import torch
 from .. import ops
 from ..config.recipe import LayerSpec
 from .context import LaneView, StepContext
+from .norm import PostNormed
 from .registry import build_part, register_part
 
 
@@ -317,4 +324,69 @@ class ParallelBlock:
         """The model's end: the final norm takes what is pending."""
         if isinstance(pending, tuple) and int(getattr(norm, "takes_branches", 1)) < 2:
             pending = self._settle(resid, pending)
+        return norm.add_norm(resid, pending, ctx, rows=rows, out_name=out_name)
+
+
+@register_part("block", "sandwich")
+class SandwichBlock:
+    slots = ("norm_mixer", "mixer", "post_mixer", "norm_feed_forward", "feed_forward", "post_feed_forward")
+    takes_follow = True
+
+    def __init__(self, layer: LayerSpec, dtype: torch.dtype, device: torch.device) -> None:
+        self.layer = layer
+        self.mixer = build_part("mixer", layer.mixer, dtype, device)
+        self.feed_forward = build_part("feed_forward", layer.feed_forward, dtype, device) if layer.feed_forward is not None else None
+        self.norm_mixer, self.post_mixer = (build_part("norm", layer.norm, dtype, device) for _ in range(2))
+        self.norm_feed_forward = self.post_feed_forward = None
+        if self.feed_forward is not None:
+            self.norm_feed_forward, self.post_feed_forward = (build_part("norm", layer.norm, dtype, device) for _ in range(2))
+        if not callable(getattr(self.post_mixer, "join", None)):
+            raise ValueError("the sandwich arrangement norms what a sublayer returns: a norm part with `join` is needed")
+
+    def parts(self) -> dict:
+        return {s: getattr(self, s) for s in self.slots if getattr(self, s) is not None}
+
+    @staticmethod
+    def _elementwise(norm) -> bool:
+        return callable(getattr(norm, "elementwise_sink", None))
+
+    def _leave(self, resid: torch.Tensor, branch, post, reader):
+        """A sublayer's branch: pending for `reader`'s kernel (the norm that comes next), or joined to the stream now."""
+        if isinstance(branch, ops.Normed):  # the product's epilogue has done all of it
+            return branch
+        if self._elementwise(post) and self._elementwise(reader):
+            return PostNormed(branch, post)
+        post.join(resid, branch)
+        return None
+
+    def forward(self, resid: torch.Tensor, pending, ctx: StepContext, lane: LaneView, writes: bool = True, follow=None):
+        n = ctx.n_tokens
+        # what the block that runs next reads first (the model's end reads with a norm of this kind: `close`)
+        after = getattr(follow, "norm_mixer", None) if isinstance(follow, SandwichBlock) else self.norm_mixer if follow is None else None
+        h = self.norm_mixer.add_norm(resid, pending, ctx)
+        reader = self.norm_feed_forward if self.feed_forward is not None else after
+        sink = None
+        if (self.feed_forward is not None or follow is not None) and self._elementwise(reader) and self._elementwise(self.post_mixer) \
+                and _can(self.mixer, "feeds_norm_sink", n):
+            sink = reader.elementwise_sink(resid, ctx, post=self.post_mixer)
+        y = self.mixer.forward(h, ctx, lane, writes, **({"sink": sink} if sink is not None else {}))
+        pending = self._leave(resid, y, self.post_mixer, reader)
+        if self.feed_forward is None:
+            return resid, pending
+        h = self.norm_feed_forward.add_norm(resid, pending, ctx)
+        f, sink = self.feed_forward, None
+        if getattr(f, "gives_unsummed", False) and self._elementwise(self.post_feed_forward):
+            y = f.forward_unsummed(h, ctx)
+        else:
+            if follow is not None and self._elementwise(after) and self._elementwise(self.post_feed_forward) and _can(f, "feeds_norm_sink", n):
+                sink = after.elementwise_sink(resid, ctx, post=self.post_feed_forward)
+            y = f.forward(h, ctx, **({"sink": sink} if sink is not None else {}))
+        return resid, self._leave(resid, y, self.post_feed_forward, after)
+
+    def close(self, resid: torch.Tensor, pending, norm, ctx: StepContext, rows: torch.Tensor | None = None,
+              out_name: str = "final_normed") -> torch.Tensor:
+        """The model's end: the final norm takes what is pending."""
+        if isinstance(pending, PostNormed) and not self._elementwise(norm):
+            pending.settle(resid)
+            pending = None
         return norm.add_norm(resid, pending, ctx, rows=rows, out_name=out_name)

@@ -1,7 +1,8 @@
 """A feed-forward of routed experts: every token runs `top` of `experts` small gated feed-forwards and adds their outputs
 up with weights from a router.
 
-    z = W_router h   (a float32 product in every mode)          s = sigmoid(z)   ("score": "softmax" for a softmax over z)
+    z = W_router h   (a float32 product in every mode)          s = sigmoid(z)   ("score": "softmax" for a softmax over z;
+                                                                                 "chosen": z itself chooses, s = softmax over the chosen)
     experts e * per .. (e + 1) * per - 1 form group e (`groups` of them, per = experts / groups); group score = top-2 sum of its s
     (its one s when per is 1); the `keep` groups of highest score stay eligible, the rest are barred (groups <= 1: none barred)
     the `top` eligible experts of largest s are chosen; weight_k = s_k / (sum of the chosen s + 1e-20) * scale
@@ -11,7 +12,9 @@ and, all optional:
     correction   a float32 number per expert that is added to the scores that choose (groups and experts), not to the weights
     renormalize  False: weight_k = s_k * scale
     identity     the last so many outputs of the router stand for experts without tensors whose output is h itself
-    shared       {"intermediate": f}: one more gated feed-forward that every token runs, added with weight 1
+    bias         a float32 number per router output, added to z
+    unit         the gated unit's constants {alpha, shift, limit} (`ops.GatedUnit`; default silu(gate) * up)
+    shared       {"intermediate": f, "unit": ...}: one more gated feed-forward that every token runs, added with weight 1
 
 Several routes, the same numbers up to rounding.  In bfloat16 the (token, choice) pairs are laid out by expert on the device
 (`ops.moe_plan`; up to 128 tokens the choice and the plan are one launch, `ops.moe_route_plan`), and where the experts' width is a multiple
@@ -25,12 +28,15 @@ read the counts on the host and run the framework's products per expert.  `ops.m
 choice (float32 sums, one rounding).
 
 params: hidden, experts (those with tensors), top, intermediate (an expert's width), groups, keep, scale, score, correction (bool),
-renormalize (default True), identity (default 0), shared, names (optional: "router", "correction"; the experts' tensors are e<k>.gate,
+renormalize (default True), identity (default 0), bias (bool), unit, shared, names (optional: "router", "correction", "bias" - default the
+router's + ".b"; the experts' tensors are e<k>.gate,
 e<k>.up, e<k>.down, the shared one's shared.gate, shared.up, shared.down).
 
 An arrangement that runs its sublayers side by side may take the part in two: `join_stream(h, ctx, resid)` adds the routed experts'
 sum to the float32 stream (no rounding in between), and the rest - the shared expert - offers its projections like any
 feed-forward (`packs_projections`; `input_weight` None when there is no shared expert), or runs alone (`forward_rest`).
+An arrangement that norms what the part returns may take it unsummed: `forward_unsummed(h, ctx)` runs the shared expert on a second stream
+beside the routed ones and returns an `ops.RoutedSum` (or a plain pair of branches), which the norm's kernel adds up in float32.
 """
 
 from __future__ import annotations
@@ -62,9 +68,11 @@ class RoutedExperts(Part):
         self.hidden, self.experts, self.top, self.inter = int(p["hidden"]), int(p["experts"]), int(p["top"]), int(p["intermediate"])
         self.groups, self.keep = int(p.get("groups") or 1), int(p.get("keep") or 1)
         self.scale = float(p.get("scale") if p.get("scale") is not None else 1.0)
-        self.softmax = p.get("score", "sigmoid") == "softmax"
-        if p.get("score", "sigmoid") not in ("sigmoid", "softmax"):
-            raise ValueError(f"routed_experts: unknown score {p.get('score')!r}")
+        scores = {"sigmoid": ops.ROUTE_SIGMOID, "softmax": ops.ROUTE_SOFTMAX, "chosen": ops.ROUTE_CHOSEN}
+        if p.get("score", "sigmoid") not in scores:
+            raise ValueError(f"routed_experts: unknown score {p.get('score')!r} (known: {', '.join(scores)})")
+        self.softmax = scores[p.get("score", "sigmoid")]
+        self.unit = ops.GatedUnit(**dict(p.get("unit") or {}))
         self.identity = int(p.get("identity") or 0)
         self.choices = self.experts + self.identity  # the router's outputs
         self.renormalize = bool(p.get("renormalize", True))
@@ -73,11 +81,13 @@ class RoutedExperts(Part):
             raise ValueError(f"routed_experts: {self.top} of {self.choices} experts in {self.groups} groups of which {self.keep} stay")
         names = dict(p.get("names") or {})
         self.n_router, self.n_correction = names.get("router", "router"), names.get("correction", "correction")
-        self.has_correction = bool(p.get("correction"))
+        self.n_bias = names.get("bias", self.n_router + ".b")
+        self.has_correction, self.has_bias = bool(p.get("correction")), bool(p.get("bias"))
+        self.router_bias: torch.Tensor | None = None
         self.correction: torch.Tensor | None = None
         shared = p.get("shared")
         self.shared = None if shared is None else build_part("feed_forward", PartSpec("swiglu", {
-            "hidden": self.hidden, "intermediate": int(shared["intermediate"]),
+            "hidden": self.hidden, "intermediate": int(shared["intermediate"]), "unit": shared.get("unit"),
             "names": {k: f"shared.{k}" for k in ("gate", "up", "down")}}), dtype, device)
         self.tcgen05 = USE_TCGEN05 and dtype == torch.bfloat16 and self.hidden % 8 == 0 and self.inter % ops.GATE_BLOCK == 0
         self.w_router = self.w_gate = self.w_up = self.w_down = self.w_gate_up = None
@@ -87,6 +97,8 @@ class RoutedExperts(Part):
         specs = {self.n_router: WeightSpec((self.choices, self.hidden), rule="float32", init="normal", std=0.1)}
         if self.has_correction:
             specs[self.n_correction] = WeightSpec((self.choices,), rule="float32", init="normal", std=0.01)
+        if self.has_bias:
+            specs[self.n_bias] = WeightSpec((self.choices,), rule="float32", init="normal", std=0.1)
         if self.shared is not None:
             specs.update(self.shared.weight_specs())
         for e in range(self.experts):
@@ -100,6 +112,8 @@ class RoutedExperts(Part):
         self.w_router = tensors[self.n_router].contiguous()
         if self.has_correction:
             self.correction = tensors[self.n_correction].contiguous()
+        if self.has_bias:
+            self.router_bias = tensors[self.n_bias].contiguous()
         if self.shared is not None:
             self.shared.bind({n: tensors[n] for n in self.shared.weight_specs()})
         self.w_gate = torch.stack([tensors[f"e{e}.gate"] for e in range(E)]).contiguous()   # [E, ff, width]
@@ -118,7 +132,7 @@ class RoutedExperts(Part):
 
     def _logits(self, x, ctx: StepContext) -> torch.Tensor:
         return ops.router_logits(x, self.w_router, ctx.buffer("router_logits", self.choices, torch.float32),
-                                 scratch=lambda rows, cols: ctx.buffer("router_in", cols, torch.float32, rows=rows))
+                                 scratch=lambda rows, cols: ctx.buffer("router_in", cols, torch.float32, rows=rows), bias=self.router_bias)
 
     def route(self, x, ctx: StepContext) -> tuple[torch.Tensor, torch.Tensor]:
         """(chosen experts int32 [N, top], their weights float32 [N, top])"""
@@ -143,6 +157,29 @@ class RoutedExperts(Part):
     def forward_rest(self, x, ctx: StepContext):
         """What `join_stream` leaves: the shared expert's output, or None without one."""
         return None if self.shared is None else self.shared.forward(x, ctx)
+
+    @property
+    def gives_unsummed(self) -> bool:
+        """Whether `forward_unsummed` may be asked for: every choice has a row of its own (no expert returns its input)."""
+        return self.identity == 0
+
+    def forward_unsummed(self, x, ctx: StepContext):
+        """The part's output as an `ops.RoutedSum`, or as the branches (routed, shared) where the routed sum is made on the way."""
+        rest = None
+        side = ops.side_lane(x.device, "shared_expert") if self.shared is not None else None
+        if side is not None:
+            side.fork()
+            with side.stream():
+                rest = self.shared.forward(x, ctx, out_name="branch_shared")
+        elif self.shared is not None:
+            rest = self.shared.forward(x, ctx, out_name="branch_shared")
+        y = self._routed(x, ctx, ctx.buffer("branch", self.hidden), None, summed=False)
+        if side is not None:
+            side.join()
+        if isinstance(y, ops.RoutedSum):
+            y.rest = rest
+            return y
+        return (y, rest) if rest is not None else y
 
     # ---- optional: the shared expert's products inside larger ones of an arrangement (see `GQAAttention.packs_projections`) ------
     packs_projections = True
@@ -173,7 +210,10 @@ class RoutedExperts(Part):
         ops.moe_plan(ids, self.experts, offsets, row_of, pair_of)
         return weights
 
-    def _grouped(self, x, ids, weights, offsets, row_of, out, ctx: StepContext, resid):
+    def _finish(self, ys, row_of, weights, out, x, resid, summed: bool):
+        return ops.moe_combine(ys, row_of, weights, out, self.top, x=x, resid=resid) if summed else ops.RoutedSum(ys, row_of, weights)
+
+    def _grouped(self, x, ids, weights, offsets, row_of, out, ctx: StepContext, resid, summed: bool = True):
         n = x.shape[0]
         pair_of = ctx.buffer("expert_pairs", self.top, torch.int32)
         if ids is None:
@@ -182,11 +222,12 @@ class RoutedExperts(Part):
             ops.moe_plan(ids, self.experts, offsets, row_of, pair_of)
         act = ctx.buffer("expert_act", self.inter, rows=n * self.top)
         ys = ctx.buffer("expert_out", self.hidden, rows=n * self.top)
-        ops.moe_grouped(x, pair_of, offsets, self.w_gate, self.w_up, self.w_down, act, ys, self.top)
-        return ops.moe_combine(ys, row_of, weights, out, self.top, x=x, resid=resid)
+        ops.moe_grouped(x, pair_of, offsets, self.w_gate, self.w_up, self.w_down, act, ys, self.top, self.unit)
+        return self._finish(ys, row_of, weights, out, x, resid, summed)
 
-    def _routed(self, x, ctx: StepContext, out: torch.Tensor, resid: torch.Tensor | None):
-        """The routed experts' sum in `out`, or added to the float32 `resid` when that is given; returns where it went."""
+    def _routed(self, x, ctx: StepContext, out: torch.Tensor, resid: torch.Tensor | None, summed: bool = True):
+        """The routed experts' sum in `out`, or added to the float32 `resid` when that is given; returns where it went.  `summed` False: the
+        sum is left to the caller (`ops.RoutedSum`) where the route taken leaves a row per choice."""
         n = x.shape[0]
         captured = bool(ctx.extras.get("graph")) or torch.cuda.is_current_stream_capturing()
         offsets = ctx.buffer("expert_offsets", 1, torch.int32, rows=self.experts + 1).view(-1)
@@ -195,15 +236,15 @@ class RoutedExperts(Part):
             weights = self._choose_and_plan(x, ctx, offsets, row_of)
             xs = ops.moe_gather(x, row_of, ctx.buffer("expert_in", self.hidden, rows=n * self.top), self.top)
             ys = ctx.buffer("expert_out", self.hidden, rows=n * self.top)
-            ops.moe_grouped_tc(xs, offsets, self.w_gate_up, self.w_down, ctx.buffer("expert_act", self.inter, rows=n * self.top), ys)
-            return ops.moe_combine(ys, row_of, weights, out, self.top, x=x, resid=resid)
+            ops.moe_grouped_tc(xs, offsets, self.w_gate_up, self.w_down, ctx.buffer("expert_act", self.inter, rows=n * self.top), ys, self.unit)
+            return self._finish(ys, row_of, weights, out, x, resid, summed)
         grouped_ok = ops.moe_grouped_ok(x, self.hidden, self.inter)
         if grouped_ok and (GROUPED_MAX is None or n <= GROUPED_MAX or captured):
-            return self._grouped(x, None, None, offsets, row_of, out, ctx, resid)
+            return self._grouped(x, None, None, offsets, row_of, out, ctx, resid, summed)
         ids, weights = self.route(x, ctx)
         if n <= ROWS_MAX or captured:
             act = ctx.buffer("expert_act", self.inter, rows=n * self.top)
-            ops.moe_expert_rows(x, ids, weights, self.w_gate, self.w_up, self.w_down, act, out)
+            ops.moe_expert_rows(x, ids, weights, self.w_gate, self.w_up, self.w_down, act, out, self.unit)
             return out if resid is None else ops.residual_add(resid, out)
         ops.moe_plan(ids, self.experts, offsets, row_of)
         bounds = offsets.tolist()  # the one host round trip of the step's experts
@@ -212,15 +253,15 @@ class RoutedExperts(Part):
             cap = max(64, -(-max(b - a for a, b in zip(bounds, bounds[1:])) // 64) * 64)
             rows = self.experts * cap
             if rows > PAD_WASTE_MAX * n * self.top:  # the tokens crowd a few experts: no layout of equal shares for them
-                return self._grouped(x, ids, weights, offsets, row_of, out, ctx, resid)
+                return self._grouped(x, ids, weights, offsets, row_of, out, ctx, resid, summed)
             ops.moe_pad_rows(ids, offsets, row_of, cap)
             xs = ops.moe_gather(x, row_of, ctx.buffer("expert_in", self.hidden, rows=rows), self.top)
             gu = ctx.buffer("expert_gate_up", 2 * self.inter, rows=rows)
             torch.bmm(xs.view(self.experts, cap, self.hidden), self.w_gate_up.transpose(1, 2), out=gu.view(self.experts, cap, 2 * self.inter))
-            act = ops.swiglu(gu, ctx.buffer("expert_act", self.inter, rows=rows), self.gate_block)
+            act = ops.swiglu(gu, ctx.buffer("expert_act", self.inter, rows=rows), self.gate_block, self.unit)
             ys = ctx.buffer("expert_out", self.hidden, rows=rows)
             torch.bmm(act.view(self.experts, cap, self.inter), self.w_down.transpose(1, 2), out=ys.view(self.experts, cap, self.hidden))
-            return ops.moe_combine(ys, row_of, weights, out, self.top, x=x, resid=resid)
+            return self._finish(ys, row_of, weights, out, x, resid, summed)
         xs = ops.moe_gather(x, row_of, ctx.buffer("expert_in", self.hidden, rows=n * self.top), self.top)
         ys = ctx.buffer("expert_out", self.hidden, rows=n * self.top)
         act = ctx.buffer("expert_act", self.inter, rows=n * self.top)
@@ -228,6 +269,6 @@ class RoutedExperts(Part):
         for e in range(self.experts):
             lo, hi = bounds[e], bounds[e + 1]
             if hi > lo:
-                ops.gated_linear(xs[lo:hi], self.w_gate_up[e], act[lo:hi], scratch[lo:hi], self.gate_block)
+                ops.gated_linear(xs[lo:hi], self.w_gate_up[e], act[lo:hi], scratch[lo:hi], self.gate_block, self.unit)
                 ops.linear(act[lo:hi], self.w_down[e], ys[lo:hi])
-        return ops.moe_combine(ys, row_of, weights, out, self.top, x=x, resid=resid)
+        return self._finish(ys, row_of, weights, out, x, resid, summed)

@@ -21,7 +21,8 @@ from .registry import register_part
 @register_part("feed_forward", "swiglu")
 class SwiGLU(Part):
     """params: hidden, intermediate, names (optional: the tensors' names after the part's prefix, keys "gate", "up",
-    "down"; default the Hugging Face ones).  `forward` takes `out_name`, the step buffer that receives the result."""
+    "down"; default the Hugging Face ones), unit (optional: the gated unit's constants {alpha, shift, limit}, see
+    `ops.GatedUnit`; default silu(gate) * up).  `forward` takes `out_name`, the step buffer that receives the result."""
 
     names_output = True
 
@@ -33,6 +34,7 @@ class SwiGLU(Part):
         self.n_gate = names.get("gate", "gate_proj.weight")
         self.n_up = names.get("up", "up_proj.weight")
         self.n_down = names.get("down", "down_proj.weight")
+        self.unit = ops.GatedUnit(**dict(spec.params.get("unit") or {}))
         self.w_gate_up: torch.Tensor | None = None
         self.w_down: torch.Tensor | None = None
         self.gate_block = 0
@@ -63,7 +65,7 @@ class SwiGLU(Part):
 
     def forward(self, x, ctx: StepContext, sink: ops.NormSink | None = None, out_name: str = "branch"):
         act = ops.gated_linear(x, self.w_gate_up, ctx.buffer("ffn_act", self.inter), ctx.buffer("gate_up", 2 * self.inter),
-                               self.gate_block)
+                               self.gate_block, self.unit)
         return ops.linear(act, self.w_down, ctx.buffer(out_name, self.hidden), sink=sink)
 
     # ---- optional: an arrangement that runs the two products inside larger ones of its own (see `GQAAttention.packs_projections`)
@@ -84,7 +86,7 @@ class SwiGLU(Part):
 
     def forward_projected(self, u: torch.Tensor, ctx: StepContext, act: torch.Tensor) -> None:
         """`u` [N, 2 * intermediate] (rows may lie in a wider buffer): the gated activation into `act` (likewise)."""
-        ops.swiglu(u, act, self.gate_block)
+        ops.swiglu(u, act, self.gate_block, self.unit)
 
 
 @register_part("feed_forward", "dense_act")

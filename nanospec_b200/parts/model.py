@@ -11,6 +11,7 @@ from .. import ops
 from ..config.recipe import ModelRecipe
 from .base import CacheNeed, StateNeed, WeightSpec
 from .context import StepContext
+from .norm import PostNormed
 from .registry import build_block, build_part
 
 
@@ -85,7 +86,10 @@ class DecoderModel:
                 if pending is not None:
                     if isinstance(pending, ops.RowScaled):
                         raise RuntimeError("a branch folded into a norm cannot precede a run that adds the input")
-                    ops.residual_add(resid, pending)
+                    if isinstance(pending, PostNormed):
+                        pending.settle(resid)
+                    else:
+                        ops.residual_add(resid, pending)
                     pending = None
                 ops.residual_add(resid, first)
             # the block that runs next: its first norm may be folded into this block's last product

@@ -14,9 +14,12 @@ Interface of a norm part:
                                         before it into its epilogue; `add_norm` hands the product's
                                         `ops.RowScaled` result on unchanged.  A norm without `sink`
                                         is never folded.
+    join(resid, branch)                 (optional) the norm on what a sublayer returns: resid += norm(branch)
 """
 
 from __future__ import annotations
+
+from dataclasses import dataclass
 
 import torch
 
@@ -52,6 +55,9 @@ class RMSNorm(Part):
     def sink(self, resid: torch.Tensor, ctx: StepContext) -> ops.NormSink:
         return ops.NormSink(resid, self.gain, self.eps, ctx.workspace)
 
+    def join(self, resid: torch.Tensor, branch: torch.Tensor) -> None:
+        ops.norm_add(resid, branch, self.gain, self.eps)
+
     def add_norm(self, resid: torch.Tensor, pending, ctx: StepContext,
                  rows: torch.Tensor | None = None, out_name: str = "normed"):
         if isinstance(pending, ops.RowScaled):
@@ -72,6 +78,7 @@ class LayerNorm(RMSNorm):
     bias_name (the bias's name after the norm's prefix; default None: no bias)."""
 
     sink = None  # hasattr(norm, "sink") is what the blocks ask; None says it cannot be folded
+    join = None  # (the kernel that norms a branch into the stream takes no mean)
     centered = True
 
     def __init__(self, spec, dtype, device) -> None:
@@ -99,6 +106,17 @@ class LayerNorm(RMSNorm):
         if self.bias is not None:  # the kernel of the streams, on one stream: the residual sum, the norm and its bias
             return ops.stream_mix_norm(resid, 1, pending, None, None, None, self.gain, self.bias, self.eps, True, out, rows=rows)
         return ops.add_layernorm(resid, pending, self.gain, self.eps, out, rows=rows)
+
+
+@dataclass
+class PostNormed:
+    """A pending branch with a norm of its own: the stream still lacks norm(branch).  `branch`: a tensor, a pair, an `ops.RoutedSum`."""
+
+    branch: object
+    norm: "DynamicTanh"
+
+    def settle(self, resid: torch.Tensor) -> None:
+        self.norm.join(resid, self.branch)
 
 
 @register_part("norm", "dyt")
@@ -134,10 +152,18 @@ class DynamicTanh(Part):
         self.bias = tensors[self.bias_name].contiguous()
         self.alpha = tensors[self.alpha_name].reshape(1).contiguous()
 
-    def elementwise_sink(self, resid: torch.Tensor, ctx: StepContext) -> ops.TanhSink:
+    def tensors(self) -> ops.TanhNorm:
+        return ops.TanhNorm(self.gain, self.bias, self.alpha)
+
+    def join(self, resid: torch.Tensor, branch) -> None:
+        """resid += this norm of a branch (a tensor, a pair of them, or an `ops.RoutedSum`)."""
+        ops.dyt_join(resid, branch, self.tensors())
+
+    def elementwise_sink(self, resid: torch.Tensor, ctx: StepContext, post: "DynamicTanh | None" = None) -> ops.TanhSink:
         """What a product needs to fold this norm and the residual sum before it into its epilogue (`ops.linear(..., sink=)`): the
-        norm is elementwise, so the product's epilogue leaves its result complete (`ops.Normed`), which `add_norm` hands on."""
-        return ops.TanhSink(resid, self.gain, self.bias, self.alpha, ctx.workspace)
+        norm is elementwise, so the product's epilogue leaves its result complete (`ops.Normed`), which `add_norm` hands on.
+        `post`: a norm of this kind on the product itself, before it joins the stream."""
+        return ops.TanhSink(resid, self.gain, self.bias, self.alpha, ctx.workspace, None if post is None else post.tensors())
 
     def add_norm(self, resid: torch.Tensor, pending, ctx: StepContext,
                  rows: torch.Tensor | None = None, out_name: str = "normed"):
@@ -148,6 +174,9 @@ class DynamicTanh(Part):
             if pending.gain is not self.gain or rows is not None:
                 raise ValueError("a Normed reached a norm it was not made for")
             return pending.x
+        if isinstance(pending, PostNormed):
+            n = resid.shape[0] if rows is None else rows.numel()
+            return ops.dyt_join(resid, pending.branch, pending.norm.tensors(), self.tensors(), ctx.buffer(out_name, self.hidden, rows=n), rows=rows)
         branches = pending if isinstance(pending, (tuple, list)) else (pending,)
         n = resid.shape[0] if rows is None else rows.numel()
         out = ctx.buffer(out_name, self.hidden, rows=n)

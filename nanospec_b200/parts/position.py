@@ -76,7 +76,7 @@ class RotaryEncoding(Part):
 def rotary_frequencies(dims: int, base: float, scaling: dict | None) -> tuple[torch.Tensor, float]:
     """Frequencies of the dims / 2 rotated pairs (float32 on the CPU) and the factor on cos and sin.
 
-    Without scaling f_i = base^(-2i / dims).  With the YaRN block (`factor`, `original`, `fast`, `slow`): a pair
+    Without scaling f_i = base^(-2i / dims); a block of `factor` alone divides every f_i by it.  With the YaRN block (`factor`, `original`, `fast`, `slow`): a pair
     that makes `t` turns over `original` positions sits at d(t) = dims * ln(original / (2 pi t)) / (2 ln base);
     pairs up to floor(d(fast)) keep f_i, pairs from ceil(d(slow)) on turn `factor` times slower, and a linear
     ramp joins them; cos and sin are multiplied by 0.1 * ln(factor) + 1.
@@ -85,7 +85,10 @@ def rotary_frequencies(dims: int, base: float, scaling: dict | None) -> tuple[to
     f = float(base) ** (-2.0 * i / dims)
     if not scaling:
         return f.to(torch.float32), 1.0
-    factor, original = float(scaling["factor"]), float(scaling["original"])
+    factor = float(scaling["factor"])
+    if set(scaling) == {"factor"}:
+        return (f / factor).to(torch.float32), 1.0
+    original = float(scaling["original"])
     if "low" in scaling or "high" in scaling:
         # the wavelength bands (`factor`, `low`, `high`, `original`): with wavelength l = 2 pi / f, a pair with
         # l < original / high keeps f, one with l > original / low turns `factor` times slower, and between the two
@@ -110,7 +113,7 @@ class Rotary(Part):
     """Rotation of the first `dims` features of every q and k head, in either pairing.
 
     params: head_dim, dims (how many features turn, even, at most head_dim), base, layout ("half": pairs
-    (i, i + dims/2); "interleaved": pairs (2i, 2i + 1)), scaling (None, the YaRN block {factor, original, fast, slow} or
+    (i, i + dims/2); "interleaved": pairs (2i, 2i + 1)), scaling (None, {factor} alone: all frequencies divided by it, the YaRN block {factor, original, fast, slow} or
     the wavelength bands {factor, original, low, high}, see `rotary_frequencies`).
     An attention mixer calls `rotate_and_store` (which can also norm the whole q and k projections first and takes
     values of another width than the keys); a mixer with a state reads `inv_freq`, `magnitude` and `interleaved`.

@@ -176,7 +176,8 @@ class GatedDeltaRule(Part):
 @register_part("mixer", "mamba2")
 class Mamba2(Part):
     """params: hidden, heads, v_dim (features of a head), state (rows of S), groups (of heads that share B and C; head h reads group
-    h // (heads / groups)), conv (taps of the short convolution), norm_groups (parts of the read-out's norm), eps, names (optional: keys
+    h // (heads / groups)), conv (taps of the short convolution), norm_groups (parts of the read-out's norm), eps, out_scale (the normed read-out is
+    multiplied by it, through the norm's gain; default 1), names (optional: keys
     "in", "conv", "conv_bias", "dt_bias", "A_log", "D", "norm", "o"; default those words, the bias "conv.b")."""
 
     DEFAULT_NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "A_log": "A_log", "D": "D", "norm": "norm", "o": "o"}
@@ -187,6 +188,7 @@ class Mamba2(Part):
         self.hidden, self.heads, self.v_dim = int(p["hidden"]), int(p["heads"]), int(p["v_dim"])
         self.state_dim, self.groups, self.taps = int(p["state"]), int(p["groups"]), int(p["conv"])
         self.norm_groups, self.eps = int(p["norm_groups"]), float(p["eps"])
+        self.out_scale = float(p.get("out_scale", 1.0))
         self.inner = self.heads * self.v_dim
         if self.heads % self.groups or self.taps < 1 or self.inner % self.norm_groups:
             raise ValueError(f"mamba2: {self.heads} heads in {self.groups} groups, {self.taps} taps, {self.inner} features in {self.norm_groups} parts")
@@ -217,6 +219,8 @@ class Mamba2(Part):
         self.conv_taps = tensors[n["conv"]].t().contiguous()                 # one row per tap, as the kernel reads them
         self.conv_bias, self.dt_bias = tensors[n["conv_bias"]].contiguous(), tensors[n["dt_bias"]].contiguous()
         self.a_log, self.skip, self.gain = (tensors[n[k]].contiguous() for k in ("A_log", "D", "norm"))
+        if self.out_scale != 1.0:
+            self.gain = self.gain * self.out_scale
 
     def cache_need(self) -> CacheNeed | None:
         return None
