@@ -36,7 +36,9 @@ sink in the denominator - windowed with kept first keys, gated heads and keys as
 convolution) beside Dezolorn layers of windowed attention.  `--design rasezen`: Rasezen models (one RMS norm a layer whose output the
 mixer and the feed-forward both read; windowed attention or the Mamba-2 state space, a dense xielu feed-forward or routed experts with
 identity experts and a shared one) beside Dezolorn layers of windowed attention and the gated delta rule, and Sorizen layers of routed
-experts; `like` as for Debuvik.
+experts; `like` as for Debuvik.  `--design tafesun`: Tafesun models (a dynamic tanh on what every sublayer reads and returns; attention with a
+gate per feature and the Mamba-2 state space side by side on one input; routed experts with clamped units) beside Rasezen models of the same
+sublayers one after another.
 """
 
 from __future__ import annotations
@@ -1193,6 +1195,137 @@ def run_design_rasezen(args) -> dict:
     }
 
 
+# ---- Tafesun beside Rasezen layers of the same parts one after another (--design tafesun) ------------------------------------
+
+TAFESUN_SIZES = {
+    # width; attention heads / kv heads / key size / value size; state heads / features / rows / groups; experts (count, chosen, width),
+    # the shared expert's width; layers (the sibling has two for each: attention alone, state space and experts)
+    "w2048": dict(width=2048, heads=32, kv_heads=8, dim=64, vdim=128, s_heads=64, s_vdim=64, s_state=128, s_groups=8, experts=32, top=4, eff=1024,
+                  shared=2048, layers=4),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=256, s_heads=128, s_vdim=64, s_state=128, s_groups=8, experts=32, top=4, eff=2048,
+                  shared=4096, layers=2),
+}
+TAFESUN_CONV = 4
+
+
+def tafesun_config(kind: str, sz: dict) -> dict:
+    """The model, and its sibling at equal width, heads, state size, experts and count of every sublayer (its values are at most 128 wide)."""
+    d = sz["dim"]
+    base = {"vocab": DESIGN_VOCAB, "width": sz["width"], "norm": {"eps": 1e-6}}
+    left = {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": d, "vdim": sz["vdim"], "scale": d ** -0.5, "rot": {"dims": d, "base": 1000000.0}}
+    right = {"heads": sz["s_heads"], "vdim": sz["s_vdim"], "state": sz["s_state"], "groups": sz["s_groups"], "conv": TAFESUN_CONV, "norm_groups": sz["s_groups"]}
+    if kind == "tafesun":
+        left["rot"]["scaling"] = {"factor": 2.0}
+        mlp = {"kind": "moe", "expert": {"ff": sz["eff"], "limit": 7.0}, "router": {"experts": sz["experts"], "top": sz["top"]},
+               "shared": {"ff": sz["shared"], "limit": 7.0}}
+        layer = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 1.0, "right_scale": 0.5}, "mlp": mlp}
+        return {"architecture": "Tafesun", **base, "logit_scale": 0.5, "layers": [layer] * sz["layers"]}
+    moe = {"kind": "moe", "expert": {"ff": sz["eff"]}, "shared": {"ff": sz["shared"]},
+           "router": {"experts": sz["experts"], "identity": 0, "top": sz["top"], "scale": 2.0}}
+    attention = {"type": "attention", "mixer": {**left, "vdim": min(sz["vdim"], 128), "mask": {"size": 1 << 16}}, "mlp": None}
+    return {"architecture": "Rasezen", **base, "layers": [attention, {"type": "mamba2", "mixer": right, "mlp": moe}] * sz["layers"]}
+
+
+def tafesun_bounds(kind: str, sz: dict, tokens: int, batch: int, context: int, pk: dict) -> dict[str, float]:
+    """Seconds that every kernel of one step needs at least, over all its calls (see kernel_bounds)."""
+    N = tokens or batch
+    W, L, H, nkv, d = sz["width"], sz["layers"], sz["heads"], sz["kv_heads"], sz["dim"]
+    dv = sz["vdim"] if kind == "tafesun" else min(sz["vdim"], 128)
+    sh, sg, sn, sv = sz["s_heads"], sz["s_groups"], sz["s_state"], sz["s_vdim"]
+    E, top, eff = sz["experts"], sz["top"], sz["eff"]
+    bw, tc, cc = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12, FP32_TFLOPS_NOMINAL * 1e12
+    pairs = sum(p + 1 for p in range(tokens)) if tokens else batch * (context + 1)
+    chan = sh * sv + 2 * sg * sn
+    operands = (2 * sg * sn + sh * (sv + 2)) * 4.0 + sh * sv * 4.0
+    out = {"ns_qk_norm_rope_store": L * 2.0 * N * ((H + nkv) * d * 2 + nkv * (d + 2 * dv)) / bw,
+           "ns_ssm_prepare": L * N * (chan * 2 + (chan + 2 * sh) * 4.0) / bw,
+           "ns_ssm_gate_norm": L * N * sh * sv * 12.0 / bw,
+           "ns_router_logits": L * (2.0 * N * W + 4.0 * E * W) / bw,
+           "ns_embed": N * W * 6.0 / bw}
+    if tokens:
+        out["ns_attention_prefill_kept"] = L * 2.0 * H * (d + dv) * pairs / tc
+        out["ns_ssm_chunked"] = L * 5.0 * tokens * sh * sn * sv / cc
+        out["ns_moe_grouped_tc"] = L * 6.0 * N * top * eff * W / tc
+        out["ns_moe_gather"] = L * 4.0 * N * top * W / bw
+    else:
+        out["ns_attention_decode_kept"] = L * 2.0 * pairs * nkv * (d + dv) / bw
+        out["ns_linear_scan"] = L * batch * (8.0 * sh * sn * sv + operands) / bw
+        out["ns_moe_grouped_tc"] = L * min(E, batch * top) * 6.0 * eff * W / bw
+    if kind == "rasezen":
+        out["ns_add_rmsnorm"] = (2 if tokens else 1) * L * 12.0 * N * W / bw
+        out["ns_swiglu_rows"] = L * 6.0 * N * sz["shared"] / bw
+        out["ns_moe_combine"] = L * N * W * (2.0 * top + 8.0) / bw
+        return out
+    # after a mixer (in the product's epilogue in a step of up to 64 tokens): the stream read and written, a branch, a norm's output; after
+    # the experts: their rows beside the shared one's (the last of these is at the wanted rows only)
+    out["ns_dyt_join"] = ((L if tokens else 0) * 12.0 + (L - 1) * (12.0 + 2.0 * top)) * N * W / bw
+    out["ns_add_dyt"] = 6.0 * N * W / bw
+    out["ns_gate_mul_rows"] = L * 6.0 * N * sz["shared"] / bw
+    return out
+
+
+TAFESUN_LIKE = {**{k: k for k in ("ns_qk_norm_rope_store", "ns_ssm_prepare", "ns_ssm_gate_norm", "ns_router_logits", "ns_attention_prefill_kept", "ns_ssm_chunked",
+                                  "ns_moe_grouped_tc", "ns_moe_gather", "ns_attention_decode_kept", "ns_linear_scan")},
+                "ns_dyt_join": "ns_add_rmsnorm", "ns_add_dyt": "ns_add_rmsnorm", "ns_gate_mul_rows": "ns_swiglu_rows"}
+
+
+def run_design_tafesun(args) -> dict:
+    import torch
+
+    from nanospec_b200 import random_model
+
+    pk, pk_src = peaks()
+    out_sizes, headline = {}, None
+    for name, sz in TAFESUN_SIZES.items():
+        row = {}
+        for kind in ("tafesun", "rasezen"):
+            model = random_model(tafesun_config(kind, sz), seed=1, device="cuda", dtype=torch.bfloat16)
+            pages_per_req = -(-(CONTEXT + args.repeats * args.steps + args.warmup + 64) // PAGE)
+            eng = design_engine(model, 64, max(64 * pages_per_req, -(-PREFILL_TOKENS // PAGE) + 8) + 8)
+            rec = {"parameters": sum(math.prod(s.shape) for s in model.weight_specs().values() if s.alias is None)}
+            for b in (8, 64):
+                pt = time_decode(eng, b, args.steps, args.warmup, args.repeats)
+                rec[f"decode_b{b}_tok_s"] = round(b * 1000.0 / pt["ms"], 1)
+                rec[f"decode_b{b}_ms"] = round(pt["ms"], 4)
+                rec[f"decode_b{b}_clocks"] = {"sm_mhz": pt["clocks"].get("sm_mhz"), "reasons": pt["clocks"].get("reasons")}
+                if b == 8 and kind == "tafesun" and name == "w4096":
+                    headline = pt
+            pre_ms, pre_clocks = time_prefill(eng, warmup=3, iters=5)
+            rec["prefill_tok_s"] = round(PREFILL_TOKENS * 1000.0 / pre_ms, 1)
+            rec["prefill_ms"] = round(pre_ms, 3)
+            rec["prefill_clocks"] = {"sm_mhz": pre_clocks.get("sm_mhz"), "reasons": pre_clocks.get("reasons")}
+            del eng
+            torch.cuda.empty_cache()
+            kernels = {}
+            for what, tokens, batch in (("prefill", PREFILL_TOKENS, 0), ("decode_b64", 0, 64)):
+                timed = time_kernels(model, tokens, batch, CONTEXT)
+                bounds = tafesun_bounds(kind, sz, tokens, batch, CONTEXT, pk)
+                kernels[what] = {k: {"calls": n, "ms": round(ms, 4), "bound_ms": round(bounds[k] * 1e3, 4) if k in bounds else None,
+                                     "frac": round(bounds[k] * 1e3 / ms, 4) if k in bounds and ms > 0 else None}
+                                 for k, (n, ms) in sorted(timed.items(), key=lambda kv: -kv[1][1])}
+            rec["kernels"] = kernels
+            row[kind] = rec
+            del model
+            torch.cuda.empty_cache()
+        # every kernel's fraction of its bound over that of the sibling's kernel that does the like work (below 0.5: twice as far)
+        row["like"] = {what: {k: round(v["frac"] / row["rasezen"]["kernels"][what][TAFESUN_LIKE[k]]["frac"], 2)
+                              for k, v in row["tafesun"]["kernels"][what].items()
+                              if k in TAFESUN_LIKE and v["frac"] and row["rasezen"]["kernels"][what].get(TAFESUN_LIKE[k], {}).get("frac")}
+                       for what in ("prefill", "decode_b64")}
+        out_sizes[name] = row
+    return {
+        "metric": "decode tok/s (Tafesun, width 4,096, 2 layers, batch 8, 1,024-token context)", "value": out_sizes["w4096"]["tafesun"]["decode_b8_tok_s"],
+        "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "ms_per_step": out_sizes["w4096"]["tafesun"]["decode_b8_ms"],
+        "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+        "data": "synthetic: seeded uniform random token ids, random weights",
+        "config": {"design": "tafesun beside rasezen (attention layers, and state-space layers with experts)", "sizes": TAFESUN_SIZES,
+                   "vocab": DESIGN_VOCAB, "conv": TAFESUN_CONV, "seq_len": CONTEXT, "prefill_tokens": PREFILL_TOKENS,
+                   "page": PAGE, "cuda_graphs": True, "peaks": pk_src, "fp32_tflops_nominal": round(FP32_TFLOPS_NOMINAL, 1),
+                   "l2": "the weights of every step are larger than L2"},
+        "gpu_launches": headline["launches"], "clocks": headline["clocks"], "sizes": out_sizes,
+    }
+
+
 def run_reference(args) -> dict:
     from baseline import reference_arm
 
@@ -1209,7 +1342,7 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=SHAPE["num_hidden_layers"])
     ap.add_argument("--no-workloads", action="store_true", help="leave out the 3B continuous-batching and 1B mixed workloads")
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    ap.add_argument("--design", choices=["dezolorn", "sorizen", "debuvik", "fubolix", "rasezen"], help="measure this design beside its closest sibling of equal size instead")
+    ap.add_argument("--design", choices=["dezolorn", "sorizen", "debuvik", "fubolix", "rasezen", "tafesun"], help="measure this design beside its closest sibling of equal size instead")
     args = ap.parse_args()
     args.warmup = max(3, args.warmup)
     args.repeats = max(1, args.repeats)
@@ -1217,7 +1350,7 @@ def main() -> int:
         if int(os.environ.get("RANK", "0")) == 0:
             print(f"bench.py measures a single-GPU engine; --gpus {args.gpus} is not supported")
         return 2
-    out = run_reference(args) if args.impl == "reference" else run_design_fubolix(args) if args.design == "fubolix" else run_design_rasezen(args) if args.design == "rasezen" else run_design_sorizen(args) if args.design == "sorizen" else run_design_debuvik(args) if args.design == "debuvik" else run_design(args) if args.design else run_ours(args)
+    out = run_reference(args) if args.impl == "reference" else run_design_fubolix(args) if args.design == "fubolix" else run_design_rasezen(args) if args.design == "rasezen" else run_design_tafesun(args) if args.design == "tafesun" else run_design_sorizen(args) if args.design == "sorizen" else run_design_debuvik(args) if args.design == "debuvik" else run_design(args) if args.design else run_ours(args)
     print(json.dumps(out), flush=True)
     return 0
 
