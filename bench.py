@@ -1269,6 +1269,20 @@ TAFESUN_LIKE = {**{k: k for k in ("ns_qk_norm_rope_store", "ns_ssm_prepare", "ns
                 "ns_dyt_join": "ns_add_rmsnorm", "ns_add_dyt": "ns_add_rmsnorm", "ns_gate_mul_rows": "ns_swiglu_rows"}
 
 
+def spread_norms(model) -> None:
+    """Dynamic-tanh norms of a random model without their biases and with a large alpha: the random streams are small against random biases,
+    and with these every token would look alike to the routers and choose the same experts."""
+    import torch
+
+    from nanospec_b200.weights import update_weights
+
+    specs = model.weight_specs()
+    state = {}
+    for name in [n[: -len(".alpha")] for n in specs if n.endswith(".alpha")]:
+        state |= {name: torch.ones(specs[name].shape), name + ".b": torch.zeros(specs[name].shape), name + ".alpha": torch.tensor(50.0)}
+    update_weights(model, state)
+
+
 def run_design_tafesun(args) -> dict:
     import torch
 
@@ -1280,6 +1294,8 @@ def run_design_tafesun(args) -> dict:
         row = {}
         for kind in ("tafesun", "rasezen"):
             model = random_model(tafesun_config(kind, sz), seed=1, device="cuda", dtype=torch.bfloat16)
+            if kind == "tafesun":
+                spread_norms(model)
             pages_per_req = -(-(CONTEXT + args.repeats * args.steps + args.warmup + 64) // PAGE)
             eng = design_engine(model, 64, max(64 * pages_per_req, -(-PREFILL_TOKENS // PAGE) + 8) + 8)
             rec = {"parameters": sum(math.prod(s.shape) for s in model.weight_specs().values() if s.alias is None)}
@@ -1317,7 +1333,7 @@ def run_design_tafesun(args) -> dict:
         "metric": "decode tok/s (Tafesun, width 4,096, 2 layers, batch 8, 1,024-token context)", "value": out_sizes["w4096"]["tafesun"]["decode_b8_tok_s"],
         "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "ms_per_step": out_sizes["w4096"]["tafesun"]["decode_b8_ms"],
         "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
-        "data": "synthetic: seeded uniform random token ids, random weights",
+        "data": "synthetic: seeded uniform random token ids, random weights (norms without biases, so that tokens spread over the experts)",
         "config": {"design": "tafesun beside rasezen (attention layers, and state-space layers with experts)", "sizes": TAFESUN_SIZES,
                    "vocab": DESIGN_VOCAB, "conv": TAFESUN_CONV, "seq_len": CONTEXT, "prefill_tokens": PREFILL_TOKENS,
                    "page": PAGE, "cuda_graphs": True, "peaks": pk_src, "fp32_tflops_nominal": round(FP32_TFLOPS_NOMINAL, 1),

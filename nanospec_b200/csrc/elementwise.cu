@@ -488,14 +488,14 @@ add_dyt_kernel(float* __restrict__ resid, const T* __restrict__ a, const T* __re
         ld8(gain + e0, g);
         if (bias) ld8(bias + e0, t);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) x[i] = fmaf(tanhf(al * x[i]), g[i], bias ? t[i] : 0.f);
+        for (int i = 0; i < 8; ++i) x[i] = fmaf(ns_tanh<sizeof(T) == 2>(al * x[i]), g[i], bias ? t[i] : 0.f);
         st8(o, x);
     } else {
         float x = resid[src + e0];
         if (a) x += ns_ld(a, src + e0);
         if (b) x += ns_ld(b, src + e0);
         if (write_resid && (a || b)) resid[src + e0] = x;
-        ns_st(o, 0, fmaf(tanhf(al * x), gain[e0], bias ? bias[e0] : 0.f));
+        ns_st(o, 0, fmaf(ns_tanh<sizeof(T) == 2>(al * x), gain[e0], bias ? bias[e0] : 0.f));
     }
 }
 
@@ -591,7 +591,7 @@ dyt_join_kernel(float* __restrict__ resid, const T* __restrict__ a, const T* __r
         load(n.gain + e0, g);
         if (n.bias) load(n.bias + e0, t);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) v[i] = fmaf(tanhf(al * v[i]), g[i], n.bias ? t[i] : 0.f);
+        for (int i = 0; i < VEC; ++i) v[i] = fmaf(ns_tanh<sizeof(T) == 2>(al * v[i]), g[i], n.bias ? t[i] : 0.f);
     };
     norm(post, y);
     load(resid + src, t);

@@ -470,8 +470,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                             pg[c] = __ldg(ep.post_gain + n0 + i + c);
                             if (ep.post_bias) pb[c] = __ldg(ep.post_bias + n0 + i + c);
                         }
-                        acc = make_float4(fmaf(tanhf(pa * acc.x), pg[0], pb[0]), fmaf(tanhf(pa * acc.y), pg[1], pb[1]),
-                                          fmaf(tanhf(pa * acc.z), pg[2], pb[2]), fmaf(tanhf(pa * acc.w), pg[3], pb[3]));
+                        acc = make_float4(fmaf(ns_tanh<true>(pa * acc.x), pg[0], pb[0]), fmaf(ns_tanh<true>(pa * acc.y), pg[1], pb[1]),
+                                          fmaf(ns_tanh<true>(pa * acc.z), pg[2], pb[2]), fmaf(ns_tanh<true>(pa * acc.w), pg[3], pb[3]));
                     }
                     res.x += acc.x; res.y += acc.y; res.z += acc.z; res.w += acc.w;
                     *reinterpret_cast<float4*>(ep.sink_resid + so) = res;
@@ -482,8 +482,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                             for (int c = 0; c < 4; ++c) b[c] = __ldg(ep.sink_bias + n0 + i + c);
                         }
-                        store_out4(ep.sink_x + so, make_float4(fmaf(tanhf(al * res.x), gain[0], b[0]), fmaf(tanhf(al * res.y), gain[1], b[1]),
-                                                               fmaf(tanhf(al * res.z), gain[2], b[2]), fmaf(tanhf(al * res.w), gain[3], b[3])));
+                        store_out4(ep.sink_x + so, make_float4(fmaf(ns_tanh<true>(al * res.x), gain[0], b[0]), fmaf(ns_tanh<true>(al * res.y), gain[1], b[1]),
+                                                               fmaf(ns_tanh<true>(al * res.z), gain[2], b[2]), fmaf(ns_tanh<true>(al * res.w), gain[3], b[3])));
                     } else {
                         store_out4(ep.sink_x + so, make_float4(res.x * gain[0], res.y * gain[1], res.z * gain[2], res.w * gain[3]));
                         float* sq = sq_s + j * (BM + 1) + (i - i0);

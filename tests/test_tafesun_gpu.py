@@ -207,6 +207,21 @@ def test_the_norm_on_a_branch_and_the_norm_after_it(hidden, dtype):
         assert torch.equal(got, out[pick.long().cuda()]) and torch.equal(resid.cpu(), x)
 
 
+@pytest.mark.parametrize("dtype", [F32, BF16], ids=["float32", "bfloat16"])
+def test_tanh_over_its_range(dtype):
+    """The norm's tanh on the stream (float32 in both types): tiny arguments, both sides of where its two forms meet, saturation."""
+    from nanospec_b200 import ops
+
+    a = torch.cat([torch.logspace(-6, 3, 3000), torch.linspace(0.2, 0.3, 1000), torch.zeros(96)])
+    x = torch.cat([a, -a]).view(1, -1).contiguous()
+    norm = ops.TanhNorm(torch.ones(x.shape[1]).cuda(), None, torch.ones(1).cuda())
+    want = torch.tanh(x.to(dtype).double())
+    resid = torch.zeros_like(x).cuda()
+    ops.dyt_join(resid, x.to(dtype).cuda(), norm)
+    err = (resid.cpu().double() - want).abs()
+    assert float(err.max()) <= 4e-7 and float((err / want.abs().clamp(min=1e-30)).max()) <= 2e-6
+
+
 def test_gated_units_in_every_kernel_that_runs_them():
     """g held below the limit, u within it, g sigmoid(alpha g) (u + shift): the activation kernel (contiguous and column ranges, both
     layouts), and the tcgen05 product of a short step; a limit that few inputs reach and one that most do."""
