@@ -316,7 +316,7 @@ def test_routing_by_biased_logits(E, top, N, K):
             assert torch.equal(ids, ids2) and torch.equal(weights, w2) and int(offsets[-1]) == N * top
 
 
-@pytest.mark.parametrize("H,G,d,dv", [(4, 2, 16, 24), (4, 2, 128, 256), (2, 1, 8, 136), (6, 3, 64, 64), (2, 2, 40, 264), (34, 2, 16, 16), (3, 1, 10, 14), (2, 1, 24, 500)])
+@pytest.mark.parametrize("H,G,d,dv", [(4, 2, 16, 24), (6, 2, 128, 256), (2, 1, 8, 136), (6, 3, 64, 64), (2, 2, 40, 264), (34, 2, 16, 16), (3, 1, 10, 14), (2, 1, 24, 500)])
 @BOTH
 def test_attention_with_a_gate_per_feature_and_wide_values(H, G, d, dv, dtype):
     """Prompt portions and single tokens over scattered pages, values of any width (in slices where they are wide), the sigmoid of a gate per
